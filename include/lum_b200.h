@@ -81,7 +81,14 @@ typedef enum lum_slot {
      * logits (`SinkBuffers`), "…mlp.router.{weight,bias}" and the experts' tensors (`ExpertWeightBuffers`): gate_up
      * [n_experts * 2 * ffn, hidden] with row 2i = gate i and row 2i+1 = up i, down [n_experts * hidden, ffn], and their biases */
     LUM_S_Q_BIAS, LUM_S_K_BIAS, LUM_S_V_BIAS, LUM_S_O_BIAS, LUM_S_SINKS, LUM_S_ROUTER, LUM_S_ROUTER_BIAS,
-    LUM_S_EXP_GATE_UP, LUM_S_EXP_GATE_UP_BIAS, LUM_S_EXP_DOWN, LUM_S_EXP_DOWN_BIAS
+    LUM_S_EXP_GATE_UP, LUM_S_EXP_GATE_UP_BIAS, LUM_S_EXP_DOWN, LUM_S_EXP_DOWN_BIAS,
+    /* layers described one by one (lum_layer_desc); file labels "l<i>.norm1[.b]", "l<i>.mix.{q,k,v,o,q.norm,k.norm,vmix,temp,r1,r2}",
+     * "l<i>.mlp.{up,down,act}", "embed", "final.norm[.b]", "head".  ATTN_NORM / Q / K / V / O / UP / DOWN / Q_NORM / K_NORM / EMBED /
+     * FINAL_NORM / LM_HEAD are the slots above */
+    LUM_S_ATTN_NORM_BIAS, LUM_S_FINAL_NORM_BIAS,   /* layer norm: the added vector */
+    LUM_S_V_MIX,                                   /* [1]: share of the first mixing layer's values */
+    LUM_S_TEMP, LUM_S_DIST_R1, LUM_S_DIST_R2,      /* [heads]: score temperature; distance bias r1 * ln(1 + r2 * distance) */
+    LUM_S_ACT                                      /* [2]: the two learned numbers of xIELU */
 } lum_slot;
 
 typedef struct lum_model_desc {
@@ -120,9 +127,31 @@ typedef struct lum_model_desc {
      * kv_pool_pages: pages in the pool (0: max_batch * max_seq / kv_page_rows, enough for every sequence at full length;
      * fewer = more sequences than the memory could hold at full length each).  Not with the persistent-kernel executor. */
     int32_t kv_page_rows, kv_pool_pages;
+    /* Decoders whose layers are described one by one (lum_model_init_layers); all zero for the families above.
+     * block_kind 1: parallel sublayers — h = norm(x), x += residual_mult * (mixer(h) + ff(h)), one norm per layer.  The other fields
+     * choose the mechanisms: norm_kind 0 RMS norm, 1 layer norm with bias (rms_eps is its eps, used as given); pos_kind 0 none, 1 a
+     * sinusoidal vector added to the embedding (entry 2i: sin(p * 10000^(-2i / hidden)), 2i + 1: cos); qk_norm 2: RMS norm of q and k
+     * over the whole projection (0: none); dist_bias 1: the score is multiplied by TEMP[h] and DIST_R1[h] * ln(1 + DIST_R2[h] * distance)
+     * is taken off; logits are multiplied by logit_scale.  weight_dtype is LUM_BF16 or LUM_F32 (dense, no quantisation), linear layers
+     * have no biases, one GPU.  With LUM_F32 everything is computed in 32 bits; with LUM_BF16 matrix operands are bf16 (accumulated
+     * in f32) and norms, scores, softmax, angles and the residual stream are f32. */
+    int32_t block_kind, norm_kind, pos_kind, dist_bias;
+    float residual_mult, logit_scale;
 } lum_model_desc;
 
 int32_t lum_model_init(lum_rt* rt, const lum_model_desc* desc);
+/* No reference counterpart (its models have one layer shape each).  One layer of a model with block_kind 1: causal softmax attention with
+ * n_q_heads queries of qk_dim over n_kv_heads keys (query head h reads K/V head h / (n_q_heads / n_kv_heads)) and values of v_dim,
+ * scores times `scale`, position i seeing the last `window` positions (0: all); v_mix 1: in every such layer but the first,
+ * v = (1 - V_MIX) v + V_MIX v_first, v_first being the first such layer's values of the same token; ffn > 0: a feed-forward
+ * down(xIELU(up h)) of that width (0: none).  n_layers descriptors are read; in `desc` the fields n_q_heads, n_kv_heads, head_dim, ffn
+ * and sliding_window are ignored. */
+typedef struct lum_layer_desc {
+    int32_t n_q_heads, n_kv_heads, qk_dim, v_dim;
+    int32_t window, v_mix, ffn;
+    float scale;
+} lum_layer_desc;
+int32_t lum_model_init_layers(lum_rt* rt, const lum_model_desc* desc, const lum_layer_desc* layers);
 /* Replaces `set_data(id, data)` for weight tensors (crates/luminal_cuda/src/runtime.rs:160-165).  `data` (host or device memory) holds
  * the FULL (unsharded) tensor, `bytes` must match it; under tensor / expert parallelism this rank's part is cut out of it.
  * `dtype` = LUM_F32, LUM_F16, LUM_BF16, or LUM_Q8_0 (wire blocks of lum_llir.h, only for slots the plan holds quantised).  A float
@@ -204,7 +233,8 @@ int32_t lum_llir_describe_chunk(const uint8_t* blob, size_t size, lum_model_desc
 /* KV cache: owned by the runtime (the reference has caller-owned buffers whose raw addresses are
  * baked into op payloads, examples/llama/src/model.rs:194-223).  reset = `KVCache::reset`. */
 int32_t lum_kv_reset(lum_rt* rt);
-/* Copy rows [0, rows) of one layer's K (kind 0) or V (kind 1) cache to host as f32. */
+/* Copy rows [0, rows) of one layer's K (kind 0) or V (kind 1) cache to host as f32.  (Layers described one by one: a row is
+ * n_kv_heads vectors of qk_dim or v_dim, each padded with zeros to a multiple of 16.) */
 int32_t lum_kv_read(lum_rt* rt, int32_t layer, int32_t kind, int32_t rows, float* host_out);
 /* Rows [0, rows) of one layer's K or V cache in the cache's own element type (bf16 or f32; this rank's KV heads), to and
  * from host memory: a conversation's cache can be parked and brought back (the reference's caches are caller-owned device
@@ -239,6 +269,11 @@ int32_t lum_set_tokens(lum_rt* rt, const int32_t* ids, size_t n);
 int32_t lum_execute(lum_rt* rt);
 /* `get_f32(logits.id)` for the last row: n = vocab (or this rank's vocab shard under TP). */
 int32_t lum_get_logits(lum_rt* rt, float* host_out, size_t n);
+/* Logits of chosen rows: the NEXT lum_execute keeps those of rows rows[0..n) of its s tokens (0 <= row < s, increasing), whatever way
+ * the tokens are taken (rows of one pass or one step each); lum_get_wanted copies them out, [n][vocab].  (The reference graph
+ * computes the logits of all s rows, examples/llama/src/main.rs:109-113.)  n = 0 clears the request.  One GPU. */
+int32_t lum_want_logits(lum_rt* rt, const int32_t* rows, int32_t n);
+int32_t lum_get_wanted(lum_rt* rt, float* host_out, size_t n);
 /* The greedy sample of the last executed row — `sample()` of main.rs:137-148 (last maximum wins). */
 int32_t lum_get_token(lum_rt* rt, int32_t* token);
 

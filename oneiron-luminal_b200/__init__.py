@@ -8,11 +8,12 @@ reference's runtime interface (``luminal::op::Runtime``, src/op.rs:10-30, and th
 There is no CPU path: importing works anywhere, but creating a runtime without the built
 library or without a CUDA device raises.
 """
-from . import llir, serving, tp  # noqa: F401
+from . import build, llir, models, replay, serving, tp  # noqa: F401
 from .runtime import (  # noqa: F401
     B200Runtime,
     LumError,
     ModelDesc,
+    LayerDesc,
     Config,
     CONFIGS,
     DTYPE,

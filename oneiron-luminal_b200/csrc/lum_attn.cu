@@ -146,7 +146,9 @@ __global__ void __launch_bounds__(256) embed_row(const EmbedArgs a) {
     }
     for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < a.H; i += gridDim.x * blockDim.x) {
         const size_t o = (size_t)tok * a.H + i;
-        a.x[i] = a.kind == WK_BF16 ? bf16_bits_to_f32(((const uint16_t*)a.table)[o]) : ((const float*)a.table)[o];
+        float v = a.kind == WK_BF16 ? bf16_bits_to_f32(((const uint16_t*)a.table)[o]) : ((const float*)a.table)[o];
+        if (a.pos_freq) v += sinusoid_at(a.pos_freq, a.state->pos, i);
+        a.x[i] = v;
     }
 }
 

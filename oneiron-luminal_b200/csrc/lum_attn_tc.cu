@@ -18,6 +18,7 @@
 #include <cuda_bf16.h>
 
 #include "lum_common.cuh"
+#include "lum_dense.cuh"
 #include "lum_rows.cuh"
 
 namespace lum {
@@ -281,6 +282,268 @@ cudaError_t launch_attn_prompt_tc(const AttnRowsArgs& a, cudaStream_t st) {
     const int G = a.n_q / a.n_kv, QT = 128 / G;
     attn_prompt_tc<<<dim3(a.n_kv, (a.M + QT - 1) / QT), kAtThreads, kAtSmem, st>>>(a, G, swap);
     return cudaGetLastError();
+}
+
+// ---------------------------------------------------------------------------------------------------- band attention
+// The same tile scheme for layers with their own head sizes, a window, and a distance bias: key size dkp (a multiple of 16) and value
+// size dvp are run-time numbers, the query heads of a K/V head may be any number R <= 128 (128 / R query rows per tile), tiles of keys
+// start at the first key any row of the tile still sees.  Queries arrive scaled (score factor and temperature).  The output goes
+// straight to the operand of the next product.
+//
+// DVH: value dimensions a thread accumulates (half of the value size, rounded up to 16).
+namespace {
+struct BandSmem { int qlo, k, v, phi, plo, misc, total; };      // byte offsets; the high Q term is at 0
+__host__ __device__ inline BandSmem band_smem(int dkp, int dvp) {
+    BandSmem s;
+    s.qlo = 128 * dkp * 2;
+    s.k = 2 * s.qlo;
+    s.v = s.k + 2 * kAtKT * dkp * 2;
+    s.phi = s.v + 2 * kAtKT * dvp * 2;
+    s.plo = s.phi + kAtPBytes;
+    s.misc = s.plo + kAtPBytes;
+    s.total = s.misc + kAtMiscBytes;
+    return s;
+}
+}  // namespace
+
+template <int DVH>
+__global__ void __launch_bounds__(kAtThreads, 1) attn_band_tc(const BandArgs a) {
+    extern __shared__ __align__(128) unsigned char smem[];
+    const QkvArgs& p = a.p;
+    const int dkp = p.dkp, dvp = p.dvp, kgr = dkp / 8, vgr = dvp / 8;
+    const BandSmem L = band_smem(dkp, dvp);
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int R = p.n_q / p.n_kv, kvh = blockIdx.x, QT = 128 / R;
+    const int q0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * QT;      // later rows first: without a window they have the most keys
+    const uint32_t s_base = smem_u32(smem);
+    const uint32_t bar_s = s_base + L.misc, bar_o = bar_s + 8, tmem_slot = bar_s + 16;
+    float* x_max = (float*)(smem + L.misc + 64);
+    int* s_flag = (int*)(smem + L.misc + 64 + 1024);          // [0] largest, [2] smallest position of the CTA's rows, [1] a wait ran out
+    constexpr uint32_t kCols = DVH > 96 ? 512u : DVH > 32 ? 256u : 128u;      // S in columns 0..63, O_t from 64 on (2 DVH columns)
+
+    if (tid == 0) { mbar_init(bar_s, 1); mbar_init(bar_o, 1); mbar_fence_init(); s_flag[0] = -1; s_flag[1] = 0; s_flag[2] = 0x7fffffff; }
+    if (warp == 0) tmem_alloc(tmem_slot, kCols);
+    tc_fence_before_sync();
+    __syncthreads();
+    tc_fence_after_sync();
+    const uint32_t tmem = *(volatile uint32_t*)(smem + L.misc + 16);
+
+    const int row = (warp & 3) * 32 + lane, half = warp >> 2;
+    const int g_row = row / QT, m_row = q0 + (row - g_row * QT);
+    const bool row_ok = g_row < R && m_row < a.M;
+    int pos_row = row_ok ? a.row_pos[m_row] : -1;
+    if (pos_row >= a.max_seq) pos_row = -1;                    // flagged by the kernel that appended the row
+    {
+        int pm = pos_row, pn = pos_row >= 0 ? pos_row : 0x7fffffff;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) { pm = max(pm, __shfl_xor_sync(0xffffffffu, pm, o)); pn = min(pn, __shfl_xor_sync(0xffffffffu, pn, o)); }
+        if (lane == 0 && pm >= 0) { atomicMax(&s_flag[0], pm); atomicMin(&s_flag[2], pn); }
+    }
+    const int head = kvh * R + (row_ok ? g_row : 0);
+    const float r1 = a.r1 ? a.r1[head] : 0.0f, r2 = a.r1 ? a.r2[head] : 0.0f;
+    const bool biased = a.r1 != nullptr;
+
+    // ---- Q tile -> two bf16 operands in shared memory
+    for (int ch = tid; ch < 128 * kgr; ch += kAtThreads) {
+        const int r = ch / kgr, c = ch - r * kgr, g = r / QT, m = q0 + (r - g * QT);
+        uint4 hi = make_uint4(0u, 0u, 0u, 0u), lo = hi;
+        if (g < R && m < a.M) {
+            const float4* src = (const float4*)(a.q + ((size_t)m * p.n_q + (size_t)kvh * R + g) * dkp + c * 8);
+            const float4 v0 = src[0], v1 = src[1];
+            split2(v0.x, v0.y, &hi.x, &lo.x); split2(v0.z, v0.w, &hi.y, &lo.y);
+            split2(v1.x, v1.y, &hi.z, &lo.z); split2(v1.z, v1.w, &hi.w, &lo.w);
+        }
+        *(uint4*)(smem + c * 2048 + r * 16) = hi;
+        *(uint4*)(smem + L.qlo + c * 2048 + r * 16) = lo;
+    }
+    __syncthreads();
+    const int pos_max = s_flag[0], pos_min = s_flag[2];
+    const int first = pos_max < 0 ? 0 : (a.window > 0 && pos_min + 1 > a.window) ? pos_min + 1 - a.window : 0;     // no row sees an earlier key
+    const int t_lo = first / kAtKT, t_hi = pos_max >= 0 ? pos_max / kAtKT + 1 : t_lo;
+    const int reach = a.window > 0 ? a.window : 0x7fffffff;    // this row sees distances 0 .. reach - 1
+
+    const size_t k_row = (size_t)p.n_kv * dkp, v_row = (size_t)p.n_kv * dvp;
+    const __nv_bfloat16* kc = (const __nv_bfloat16*)a.k_cache + (size_t)kvh * dkp;
+    const __nv_bfloat16* vc = (const __nv_bfloat16*)a.v_cache + (size_t)kvh * dvp;
+    // one operand tile: 64 positions x `gr` 16-byte groups; a warp takes 8 positions x 4 groups at a time
+    auto load_part = [&](int t, size_t tile_row, uint32_t dst, const __nv_bfloat16* src, size_t row_elems, int gr) {
+        const int gq = (gr + 3) / 4;
+        for (int w = warp; w < 8 * gq; w += kAtThreads / 32) {
+            const int kb = w / gq, key = kb * 8 + (lane >> 2), c = (w - kb * gq) * 4 + (lane & 3), j = t * kAtKT + key;
+            const bool in = j <= pos_max;                      // rows never written read as zeros
+            if (c < gr) cp_async16(dst + c * 1024 + key * 16, src + (tile_row + (size_t)(in ? key : 0)) * row_elems + c * 8, in ? 16u : 0u);
+        }
+    };
+    auto load_tile = [&](int t, int buf) {
+        // the tile's 64 positions start on a multiple of 64: one sequence slot or one page (of at least 64 rows) holds them all
+        const size_t tile_row = kv_phys_row(a.pg, a.seq0, a.max_seq, t * kAtKT);
+        load_part(t, tile_row, s_base + L.k + buf * kAtKT * dkp * 2, kc, k_row, kgr);
+        load_part(t, tile_row, s_base + L.v + buf * kAtKT * dvp * 2, vc, v_row, vgr);
+        cp_async_commit();
+    };
+
+    float o_acc[DVH];
+#pragma unroll
+    for (int i = 0; i < DVH; i++) o_acc[i] = 0.0f;
+    float m_run = -INFINITY, l_run = 0.0f;
+    const uint32_t idesc_s = idesc_bf16(128, kAtKT, false), idesc_o = idesc_bf16(128, dvp, true);
+    const uint32_t lane_base = tmem + ((uint32_t)((warp & 3) * 32) << 16);
+
+    if (t_lo < t_hi) load_tile(t_lo, 0);
+    uint32_t phase = 0;
+    bool failed = false;
+#pragma unroll 1
+    for (int t = t_lo; t < t_hi; t++) {
+        const int buf = (t - t_lo) & 1;
+        if (t + 1 < t_hi) { load_tile(t + 1, buf ^ 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
+        fence_proxy_async_smem();
+        __syncthreads();
+        if (tid == 0) {
+            tc_fence_after_sync();
+            const uint32_t kb = s_base + L.k + buf * kAtKT * dkp * 2;
+            for (int term = 0; term < 2; term++) {
+                const uint32_t qb = s_base + (term ? L.qlo : 0);
+                for (int ks = 0; ks < dkp / 16; ks++)
+                    umma_bf16(tmem, umma_smem_desc(qb + ks * 2 * 2048, 2048, 128), umma_smem_desc(kb + ks * 2 * 1024, 1024, 128), idesc_s,
+                              (term | ks) ? 1u : 0u);
+            }
+            umma_commit(bar_s);
+        }
+        // distance corrections of this thread's 32 keys, while the tensor core computes the scores
+        const int j0 = t * kAtKT + half * 32;
+        float s[32];
+        if (biased) {
+#pragma unroll
+            for (int i = 0; i < 32; i++) s[i] = r1 * logf(fmaf(r2, (float)max(pos_row - (j0 + i), 0), 1.0f));      // (masked keys: any finite value)
+        } else {
+#pragma unroll
+            for (int i = 0; i < 32; i++) s[i] = 0.0f;
+        }
+        if (!mbar_wait(bar_s, phase)) failed = true;
+        tc_fence_after_sync();
+
+        // ---- softmax of this thread's row over its 32 keys of the tile
+        {
+            uint32_t v0[16], v1[16];
+            tmem_ld16(lane_base + half * 32, v0);
+            tmem_ld16(lane_base + half * 32 + 16, v1);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 16; i++) { s[i] = __uint_as_float(v0[i]) - s[i]; s[16 + i] = __uint_as_float(v1[i]) - s[16 + i]; }
+        }
+        float mx = -INFINITY;
+#pragma unroll
+        for (int i = 0; i < 32; i++) {
+            const int d = pos_row - (j0 + i);
+            s[i] = (d >= 0 && d < reach) ? s[i] : -INFINITY;
+            mx = fmaxf(mx, s[i]);
+        }
+        x_max[half * 128 + row] = mx;
+        named_sync(1, kAtThreads);
+        const float m_new = fmaxf(m_run, fmaxf(mx, x_max[(half ^ 1) * 128 + row]));
+        const float alpha = (m_new == -INFINITY) ? 1.0f : expf(m_run - m_new);
+        float psum = 0.0f;
+        uint32_t ph[16], pl[16];
+#pragma unroll
+        for (int i = 0; i < 32; i += 2) {
+            const float p0 = (s[i] == -INFINITY) ? 0.0f : expf(s[i] - m_new);
+            const float p1 = (s[i + 1] == -INFINITY) ? 0.0f : expf(s[i + 1] - m_new);
+            psum += p0 + p1;
+            split2(p0, p1, &ph[i >> 1], &pl[i >> 1]);
+        }
+        l_run = l_run * alpha + psum;
+        m_run = m_new;
+#pragma unroll
+        for (int c = 0; c < 4; c++) {
+            const int off = (half * 4 + c) * 2048 + row * 16;
+            *(uint4*)(smem + L.phi + off) = make_uint4(ph[c * 4], ph[c * 4 + 1], ph[c * 4 + 2], ph[c * 4 + 3]);
+            *(uint4*)(smem + L.plo + off) = make_uint4(pl[c * 4], pl[c * 4 + 1], pl[c * 4 + 2], pl[c * 4 + 3]);
+        }
+        fence_proxy_async_smem();
+        tc_fence_before_sync();
+        __syncthreads();
+        if (tid == 0) {
+            tc_fence_after_sync();
+            const uint32_t vb = s_base + L.v + buf * kAtKT * dvp * 2;
+#pragma unroll
+            for (int term = 0; term < 2; term++) {
+                const uint32_t pb = s_base + (term ? L.plo : L.phi);
+#pragma unroll
+                for (int ks = 0; ks < kAtKT / 16; ks++)
+                    umma_bf16(tmem + 64, umma_smem_desc(pb + ks * 2 * 2048, 2048, 128), umma_smem_desc(vb + ks * 256, 128, 1024), idesc_o,
+                              (term | ks) ? 1u : 0u);
+            }
+            umma_commit(bar_o);
+        }
+        if (!mbar_wait(bar_o, phase)) failed = true;
+        tc_fence_after_sync();
+#pragma unroll
+        for (int c = 0; c < DVH / 16; c++) {
+            uint32_t v[16];
+            tmem_ld16(lane_base + 64 + half * DVH + c * 16, v);      // (columns beyond dvp: never written, never stored)
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 16; i++) o_acc[c * 16 + i] = fmaf(o_acc[c * 16 + i], alpha, __uint_as_float(v[i]));
+        }
+        tc_fence_before_sync();
+        phase ^= 1u;
+        if (__syncthreads_or(failed ? 1 : 0)) { if (tid == 0) s_flag[1] = 1; break; }
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    if (s_flag[1] && tid == 0 && a.status) atomicOr(a.status, LUM_ST_WAIT_TMEM);
+
+    // ---- out = O / l, l = the two halves' sums, as bf16 in the operand of the next product
+    x_max[half * 128 + row] = l_run;
+    __syncthreads();
+    const float l_tot = l_run + x_max[(half ^ 1) * 128 + row];
+    if (row_ok) {
+        const float inv = l_tot > 0.0f ? 1.0f / l_tot : 0.0f;
+        const int col0 = head * p.dv, e0 = half * DVH;
+        unsigned char* out = (unsigned char*)a.out.p;
+        if ((p.dv & 7) == 0) {
+#pragma unroll
+            for (int c = 0; c < DVH / 8; c++) {
+                if (e0 + c * 8 < p.dv) {
+                    uint32_t w[4];
+#pragma unroll
+                    for (int i = 0; i < 4; i++) {
+                        const __nv_bfloat162 b = __floats2bfloat162_rn(o_acc[c * 8 + 2 * i] * inv, o_acc[c * 8 + 2 * i + 1] * inv);
+                        w[i] = *(const uint32_t*)&b;
+                    }
+                    *(uint4*)(out + row_operand_off(WK_BF16, a.out.chunks, m_row, col0 + e0 + c * 8)) = make_uint4(w[0], w[1], w[2], w[3]);
+                }
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < DVH; i++)
+                if (e0 + i < p.dv) *(__nv_bfloat16*)(out + row_operand_off(WK_BF16, a.out.chunks, m_row, col0 + e0 + i)) = __float2bfloat16_rn(o_acc[i] * inv);
+        }
+    }
+    tc_fence_before_sync();
+    __syncthreads();
+    if (warp == 0) tmem_dealloc(tmem, kCols);
+}
+
+bool band_prompt_tc_supported(const BandArgs& a) {
+    const QkvArgs& p = a.p;
+    const int R = p.n_kv > 0 ? p.n_q / p.n_kv : 0;
+    return a.kv_bf16 && a.out_kind == WK_BF16 && a.row_seq == nullptr && R >= 1 && R <= 128 && p.n_q == R * p.n_kv && p.dkp % 16 == 0 && p.dvp % 16 == 0 &&
+           p.dvp <= 256 && band_smem(p.dkp, p.dvp).total <= 226 * 1024;
+}
+
+cudaError_t launch_band_prompt_tc(const BandArgs& a, cudaStream_t st) {
+    if (!band_prompt_tc_supported(a)) return cudaErrorInvalidValue;
+    const int dvh = (a.p.dvp / 2 + 15) / 16 * 16;
+    const void* fn = dvh <= 16 ? (const void*)attn_band_tc<16> : dvh <= 32 ? (const void*)attn_band_tc<32> : dvh <= 64 ? (const void*)attn_band_tc<64>
+                     : dvh <= 96 ? (const void*)attn_band_tc<96> : (const void*)attn_band_tc<128>;
+    const int smem = band_smem(a.p.dkp, a.p.dvp).total;
+    const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
+    if (e != cudaSuccess) return e;
+    const int QT = 128 / (a.p.n_q / a.p.n_kv);
+    BandArgs b = a;
+    void* params[] = {&b};
+    return cudaLaunchKernel(fn, dim3(a.p.n_kv, (a.M + QT - 1) / QT), dim3(kAtThreads), params, (size_t)smem, st);
 }
 
 }  // namespace lum

@@ -41,50 +41,6 @@
 
 namespace lum {
 
-// The greedy sampler's last step, run by the last CTA to arrive (one-op kernels) : fold the per-CTA
-// maxima, log the token and advance the decode state.
-__device__ __forceinline__ void argmax_finish(const GemvArgs& a, ArgBest mine, int tid, int nthreads, int bar_id) {
-    __shared__ int s_last;
-    if (tid == 0) {
-        a.part_val[blockIdx.x] = mine.v;
-        a.part_idx[blockIdx.x] = mine.i;
-        __threadfence();
-        const unsigned int ticket = atomicAdd(a.counter, 1u);
-        s_last = (ticket == gridDim.x - 1) ? 1 : 0;
-    }
-    named_sync(bar_id, nthreads);
-    if (s_last && tid < 32) {
-        __threadfence();
-        const ArgBest fb = argmax_final(a.part_val, a.part_idx, (int)gridDim.x, tid);
-        const int fi = fb.i;
-        if (tid == 0) {
-            DecodeState* st = a.pair_out ? nullptr : a.state;
-            if (a.pair_out) {   // tensor parallel: publish this shard's best; the ranks' pairs are folded after an all-gather ...
-                const int pv = __float_as_int(fb.v), pi = fi >= 0 ? fi + a.row_offset : -1;
-                a.pair_out[0] = pv;
-                a.pair_out[1] = pi;
-                if (a.n_peers > 0) {   // ... or are written into every rank's memory right here, followed by "landed" words
-#pragma unroll
-                    for (int r = 0; r < kMaxPeers; r++)
-                        if (r < a.n_peers) { int* dst = (int*)a.peer_out[r]; dst[0] = pv; dst[1] = pi; }
-                    __threadfence_system();
-                    const uint32_t word = peer_word(__ldcg(a.seq), a.peer_tag);
-#pragma unroll
-                    for (int r = 0; r < kMaxPeers; r++)
-                        if (r < a.n_peers) st_release_sys(a.peer_flag[r], word);
-                }
-            }
-            if (st) {
-                const int step = st->step;
-                st->last_tok = fi;
-                if (st->log && a.tokens_out && step < st->max_steps) { a.tokens_out[step] = fi; st->step = step + 1; }
-                if (a.advance) { st->tok = fi; st->pos = st->pos + 1; }
-            }
-            *a.counter = 0u;
-        }
-    }
-}
-
 // Prologue of the plain-load kernel: bring x into shared memory as f32 (optionally RMS-normalised and
 // scaled by the gains).
 __device__ __forceinline__ void gemv_load_x(const GemvArgs& a, float* xs, int tid, int nthreads, float* scratch, int bar_id) {

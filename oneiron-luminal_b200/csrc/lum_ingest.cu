@@ -32,6 +32,7 @@
 #include <cuda_fp16.h>
 
 #include "../../include/lum_b200.h"
+#include "lum_dense.cuh"
 #include "lum_kernels.cuh"
 
 namespace lum {
@@ -387,21 +388,36 @@ static const SlotName kTopNames[] = {
     {LUM_S_EMBED, "model.embed_tokens.weight"}, {LUM_S_FINAL_NORM, "model.norm.weight"}, {LUM_S_LM_HEAD, "lm_head.weight"},
 };
 
-static std::string slot_label(int slot, int layer) {
-    for (const SlotName& s : kTopNames) if (s.slot == slot) return s.suffix;
-    for (const SlotName& s : kLayerNames) if (s.slot == slot) return "model.layers." + std::to_string(layer) + "." + s.suffix;
+// models whose layers are described one by one: "l<i>." + suffix
+static const SlotName kBlockLayerNames[] = {
+    {LUM_S_ATTN_NORM, "norm1"}, {LUM_S_ATTN_NORM_BIAS, "norm1.b"}, {LUM_S_Q, "mix.q"}, {LUM_S_K, "mix.k"}, {LUM_S_V, "mix.v"}, {LUM_S_O, "mix.o"},
+    {LUM_S_Q_NORM, "mix.q.norm"}, {LUM_S_K_NORM, "mix.k.norm"}, {LUM_S_V_MIX, "mix.vmix"}, {LUM_S_TEMP, "mix.temp"}, {LUM_S_DIST_R1, "mix.r1"},
+    {LUM_S_DIST_R2, "mix.r2"}, {LUM_S_UP, "mlp.up"}, {LUM_S_DOWN, "mlp.down"}, {LUM_S_ACT, "mlp.act"},
+};
+static const SlotName kBlockTopNames[] = {
+    {LUM_S_EMBED, "embed"}, {LUM_S_FINAL_NORM, "final.norm"}, {LUM_S_FINAL_NORM_BIAS, "final.norm.b"}, {LUM_S_LM_HEAD, "head"},
+};
+struct LabelStyle { const SlotName *top, *layer; size_t n_top, n_layer; const char* prefix; };
+static LabelStyle label_style(int style) {
+    if (style == 1) return {kBlockTopNames, kBlockLayerNames, sizeof kBlockTopNames / sizeof *kBlockTopNames, sizeof kBlockLayerNames / sizeof *kBlockLayerNames, "l"};
+    return {kTopNames, kLayerNames, sizeof kTopNames / sizeof *kTopNames, sizeof kLayerNames / sizeof *kLayerNames, "model.layers."};
+}
+
+static std::string slot_label(const LabelStyle& ls, int slot, int layer) {
+    for (size_t i = 0; i < ls.n_top; i++) if (ls.top[i].slot == slot) return ls.top[i].suffix;
+    for (size_t i = 0; i < ls.n_layer; i++) if (ls.layer[i].slot == slot) return ls.prefix + std::to_string(layer) + "." + ls.layer[i].suffix;
     return "";
 }
-static bool label_slot(const std::string& name, int* slot, int* layer) {
-    for (const SlotName& s : kTopNames) if (name == s.suffix) { *slot = s.slot; *layer = 0; return true; }
-    static const char kPre[] = "model.layers.";
-    if (name.compare(0, sizeof kPre - 1, kPre) != 0) return false;
-    size_t i = sizeof kPre - 1, d0 = i;
+static bool label_slot(const LabelStyle& ls, const std::string& name, int* slot, int* layer) {
+    for (size_t k = 0; k < ls.n_top; k++) if (name == ls.top[k].suffix) { *slot = ls.top[k].slot; *layer = 0; return true; }
+    const size_t pre = strlen(ls.prefix);
+    if (name.compare(0, pre, ls.prefix) != 0) return false;
+    size_t i = pre, d0 = i;
     int l = 0;
     while (i < name.size() && name[i] >= '0' && name[i] <= '9' && i - d0 < 6) { l = l * 10 + (name[i] - '0'); i++; }
     if (i == d0 || i >= name.size() || name[i] != '.') return false;
     const std::string rest = name.substr(i + 1);
-    for (const SlotName& s : kLayerNames) if (rest == s.suffix) { *slot = s.slot; *layer = l; return true; }
+    for (size_t k = 0; k < ls.n_layer; k++) if (rest == ls.layer[k].suffix) { *slot = ls.layer[k].slot; *layer = l; return true; }
     return false;
 }
 
@@ -433,14 +449,16 @@ static int store_weight(lum_rt* rt, int slot, int layer, const void* src, size_t
     // copies go on the runtime's own (non-blocking) stream: a legacy-stream copy from pageable memory may return before its
     // transfer has landed and would not be ordered against kernels on this stream
     void *stage = nullptr, *planes = nullptr;
-    const bool direct = !q8_src && ((dtype == LUM_F32 && t.kind == WK_F32) || (dtype == LUM_BF16 && t.kind == WK_BF16));
+    const bool direct = !q8_src && t.kc != kLayoutChunked && ((dtype == LUM_F32 && t.kind == WK_F32) || (dtype == LUM_BF16 && t.kind == WK_BF16));
     if (direct) {
         if (e == cudaSuccess) e = cudaMemcpy2DAsync(t.w, row_bytes, from, src_pitch, row_bytes, t.rows, cudaMemcpyDefault, t.stream);
     } else {
         if (e == cudaSuccess) e = cudaMalloc(&stage, t.rows * row_bytes + 64);
         if (e != cudaSuccess) return lum_internal_fail(rt, LUM_E_NOMEM, "set_weight: staging buffer");
         e = cudaMemcpy2DAsync(stage, row_bytes, from, src_pitch, row_bytes, t.rows, cudaMemcpyDefault, t.stream);
-        if (t.kind == WK_Q8) {
+        if (t.kc == kLayoutChunked) {
+            if (e == cudaSuccess) e = launch_chunked_pack(stage, dtype, t.rows, t.cols, t.w, t.kind, t.nt, t.crow0, t.stream);
+        } else if (t.kind == WK_Q8) {
             int8_t* pq = (int8_t*)t.w;
             __half* ps = t.s;
             if (t.kc) {      // -> temporary planes -> packed tile stream
@@ -485,6 +503,15 @@ static int fetch_weight(lum_rt* rt, const WeightView& t, std::vector<uint8_t>* o
         const cudaError_t es = cudaStreamSynchronize(t.stream);
         if (e == cudaSuccess) e = es;
         if (wire) cudaFree(wire);
+    } else if (t.kc == kLayoutChunked) {
+        out->resize(n * (t.kind == WK_BF16 ? 2 : 4));
+        void* rows = nullptr;
+        if (e == cudaSuccess) e = cudaMalloc(&rows, out->size() + 64);
+        if (e == cudaSuccess) e = launch_chunked_unpack(t.w, t.kind, t.nt, t.crow0, t.rows, t.cols, nullptr, rows, t.stream);
+        if (e == cudaSuccess) e = cudaMemcpyAsync(out->data(), rows, out->size(), cudaMemcpyDeviceToHost, t.stream);
+        const cudaError_t es = cudaStreamSynchronize(t.stream);
+        if (e == cudaSuccess) e = es;
+        if (rows) cudaFree(rows);
     } else {
         out->resize(n * (t.kind == WK_BF16 ? 2 : 4));
         if (e == cudaSuccess) e = cudaMemcpyAsync(out->data(), t.w, out->size(), cudaMemcpyDeviceToHost, t.stream);
@@ -595,10 +622,11 @@ int32_t lum_load_safetensors(lum_rt* rt, const char* path, int32_t* n_loaded, in
         presharded = 1;
     }
     int rc = 0, loaded = 0, ignored = 0;
+    const LabelStyle ls = label_style(lum_internal_label_style(rt));
     for (const StTensor& t : f->tensors) {
         int slot = 0, layer = 0;
         WeightView v;
-        if (!label_slot(t.name, &slot, &layer) || lum_internal_weight_view(rt, slot, layer, &v)) { ignored++; continue; }   // as the reference: labels the graph does not have are skipped
+        if (!label_slot(ls, t.name, &slot, &layer) || lum_internal_weight_view(rt, slot, layer, &v)) { ignored++; continue; }   // as the reference: labels the graph does not have are skipped
         uint32_t dt = st_dtype_code(t.dtype);
         if (dt == LUM_ST_U8) dt = LUM_Q8_0;          // U8 tensors are raw bytes (runtime.rs:148-152): here, Q8_0 wire blocks
         size_t elems = 1;
@@ -626,6 +654,7 @@ int32_t lum_save_safetensors(lum_rt* rt, const char* path) {
     if (!rt || !path || lum_internal_weight_view(rt, LUM_S_EMBED, 0, &probe)) return lum_internal_fail(rt, LUM_E_INVALID, "save_safetensors: no model or null path");
     int tp = 1, tr = 0, ep = 1, er = 0, n_layers = 0;
     n_layers = lum_internal_parallel(rt, &tp, &tr, &ep, &er);
+    const LabelStyle ls = label_style(lum_internal_label_style(rt));
     struct Item { int slot, layer; WeightView v; };
     std::vector<Item> items;
     std::vector<StOut> outs;
@@ -633,7 +662,7 @@ int32_t lum_save_safetensors(lum_rt* rt, const char* path) {
         WeightView v;
         if (lum_internal_weight_view(rt, slot, layer, &v)) return;
         StOut o;
-        o.name = slot_label(slot, layer);
+        o.name = slot_label(ls, slot, layer);
         if (v.kind == WK_Q8) { o.dtype = LUM_ST_U8; o.shape = {(int64_t)v.rows, (int64_t)(v.cols / 32 * 34)}; o.bytes = v.rows * v.cols / 32 * 34; }
         else {
             o.dtype = v.kind == WK_BF16 ? LUM_BF16 : LUM_F32;
@@ -643,8 +672,8 @@ int32_t lum_save_safetensors(lum_rt* rt, const char* path) {
         items.push_back({slot, layer, v});
         outs.push_back(o);
     };
-    for (const SlotName& s : kTopNames) add(s.slot, 0);
-    for (int l = 0; l < n_layers; l++) for (const SlotName& s : kLayerNames) add(s.slot, l);
+    for (size_t k = 0; k < ls.n_top; k++) add(ls.top[k].slot, 0);
+    for (int l = 0; l < n_layers; l++) for (size_t k = 0; k < ls.n_layer; k++) add(ls.layer[k].slot, l);
     std::map<std::string, std::string> meta;
     meta["lum.shard"] = "1";
     meta["lum.tp_size"] = std::to_string(tp); meta["lum.tp_rank"] = std::to_string(tr);

@@ -157,7 +157,14 @@ struct EmbedArgs {
     const DecodeState* state;
     uint32_t* status;
     int use_pdl;
+    const double* pos_freq;// optional [ceil(H / 2)]: sin (entry 2i) and cos (2i + 1) of position * pos_freq[i] are added
 };
+// the sinusoidal position vector's entry i (angles in f64: exact to f32 rounding at any position)
+__device__ __forceinline__ float sinusoid_at(const double* freq, int pos, int i) {
+    double s, c;
+    sincos((double)pos * freq[i >> 1], &s, &c);
+    return (float)((i & 1) ? c : s);
+}
 
 // message of the last failed stand-alone operator on this thread (read back through lum_last_error(NULL))
 void set_op_error(const char* msg);
@@ -198,6 +205,7 @@ struct WeightView {
     size_t rows, cols, kdev;             // the shard; kdev = columns of the device layout (>= cols, zero columns beyond)
     size_t row0, col0, full_rows, full_cols;
     int device; cudaStream_t stream;
+    int nt; size_t crow0;                // chunked layout (kc == kLayoutChunked, lum_dense.cuh): padded rows of the container, first row in it
 };
 cudaError_t launch_q8_dequant(const int8_t* q, const __half* s, float* out, size_t n_elems, cudaStream_t st);
 cudaError_t launch_q8_dequant_rows(const void* w, const __half* s, int K, int kc, size_t row0, size_t n_rows, float* out, cudaStream_t st, int valid_cols = 0);
@@ -208,5 +216,6 @@ cudaError_t launch_to_f32(const void* in, int kind, float* out, size_t n, cudaSt
 // Internal hand-over between the runtime (which owns the model) and the weight-ingest code; not part of the C ABI.
 struct lum_rt;
 int lum_internal_weight_view(lum_rt* rt, int slot, int layer, lum::WeightView* out);     // 0 = filled; 1 = no model / no such slot
+int lum_internal_label_style(lum_rt* rt);                                                // how the model's tensors are called in files (block_kind)
 int lum_internal_fail(lum_rt* rt, int code, const char* msg);                            // records the message, returns the code
 int lum_internal_parallel(lum_rt* rt, int* tp_size, int* tp_rank, int* ep_size, int* ep_rank);   // returns the number of layers

@@ -22,8 +22,8 @@
 namespace lum {
 
 // ---------------------------------------------------------------------------------------------------- embedding rows
-__global__ void __launch_bounds__(256) embed_rows(const void* table, int kind, int H, int vocab, const int* row_tok, float* x, int M,
-                                                  uint32_t* status) {
+__global__ void __launch_bounds__(256) embed_rows(const void* table, int kind, int H, int vocab, const int* row_tok, float* x, int ldx, int M,
+                                                  const int* row_pos, const double* pos_freq, uint32_t* status) {
     const int m = blockIdx.x;
     if (m >= M) return;
     const int tok = row_tok[m];
@@ -33,7 +33,9 @@ __global__ void __launch_bounds__(256) embed_rows(const void* table, int kind, i
     }
     for (int i = threadIdx.x; i < H; i += 256) {
         const size_t o = (size_t)tok * H + i;
-        x[(size_t)m * H + i] = kind == WK_BF16 ? bf16_bits_to_f32(((const uint16_t*)table)[o]) : ((const float*)table)[o];
+        float v = kind == WK_BF16 ? bf16_bits_to_f32(((const uint16_t*)table)[o]) : ((const float*)table)[o];
+        if (pos_freq) v += sinusoid_at(pos_freq, row_pos[m], i);
+        x[(size_t)m * ldx + i] = v;
     }
 }
 
@@ -416,7 +418,12 @@ __global__ void step_advance(int* step) { *step += 1; }
 // ---------------------------------------------------------------------------------------------------- launchers
 
 cudaError_t launch_embed_rows(const void* table, int kind, int H, int vocab, const int* row_tok, float* x, int M, uint32_t* status, cudaStream_t st) {
-    embed_rows<<<M, 256, 0, st>>>(table, kind, H, vocab, row_tok, x, M, status);
+    embed_rows<<<M, 256, 0, st>>>(table, kind, H, vocab, row_tok, x, H, M, nullptr, nullptr, status);
+    return cudaGetLastError();
+}
+cudaError_t launch_embed_rows_sinusoid(const void* table, int kind, int H, int vocab, const int* row_tok, const int* row_pos, const double* pos_freq, float* x, int ldx,
+                                       int M, uint32_t* status, cudaStream_t st) {
+    embed_rows<<<M, 256, 0, st>>>(table, kind, H, vocab, row_tok, x, ldx, M, row_pos, pos_freq, status);
     return cudaGetLastError();
 }
 

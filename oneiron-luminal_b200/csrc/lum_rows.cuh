@@ -79,6 +79,9 @@ bool gemm_supported(const GemmArgs& a);
 cudaError_t launch_rows_quantize(const RowsArgs& a, cudaStream_t st);
 cudaError_t launch_gemm(const GemmArgs& a, int sm_count, cudaStream_t st);
 cudaError_t launch_embed_rows(const void* table, int kind, int H, int vocab, const int* row_tok, float* x, int M, uint32_t* status, cudaStream_t st);
+// the same plus the sinusoidal position vector (see EmbedArgs::pos_freq; null: none), rows ldx floats apart
+cudaError_t launch_embed_rows_sinusoid(const void* table, int kind, int H, int vocab, const int* row_tok, const int* row_pos, const double* pos_freq, float* x, int ldx,
+                                       int M, uint32_t* status, cudaStream_t st);
 cudaError_t launch_rope_append_rows(const RopeRowsArgs& a, cudaStream_t st);
 cudaError_t launch_attn_rows(const AttnRowsArgs& a, cudaStream_t st);
 constexpr int kAttnRowsMaxSplits = 8;

@@ -29,6 +29,7 @@
 #include "lum_rows.cuh"
 #include "lum_moe.cuh"
 #include "lum_sample.cuh"
+#include "lum_dense.cuh"
 
 using namespace lum;
 
@@ -110,6 +111,8 @@ struct Tensor {
                                         // (a packed Q8_0 K-shard such as 14336 / 8 = 1792 -> 2048) so that it still takes the streaming kernels
     size_t row0 = 0, col0 = 0;          // shard origin in the full tensor
     size_t full_rows = 0, full_cols = 0;
+    int nt = 0;                         // chunked layout (kc == kLayoutChunked): padded rows of the container this tensor is a row range of
+    size_t crow0 = 0;                   // ... and the tensor's first row in it
     size_t bytes() const {
         const size_t n = rows * cols;
         return kind == WK_Q8 ? n + n / 16 : kind == WK_BF16 ? n * 2 : n * 4;
@@ -122,6 +125,15 @@ struct LayerW {
     Tensor router, router_b, exp_gu, exp_gu_b, exp_dn, exp_dn_b;   // routed experts (this rank's experts only)
     void* kc = nullptr;
     void* vc = nullptr;
+    size_t k_elems = 0, v_elems = 0;                          // elements of one cached row of this layer
+    // layers described one by one (block_kind 1)
+    lum_layer_desc g{};
+    int dkp = 0, dvp = 0;                                     // head sizes in the cache (padded with zeros)
+    void *w_in = nullptr, *w_o = nullptr, *w_dn = nullptr;    // containers: q | k | v | up, o, down
+    int nt_in = 0, k_off = 0, v_off = 0, act_row0 = 0;        // rows of w_in, where its parts begin (act_row0 == nt_in: no feed-forward)
+    int o_chunks = 0, dn_chunks = 0;
+    int mix = 0;                                              // 0 none, 1 the first mixing layer, 2 a later one
+    Tensor attn_norm_b, v_mix, temp, dist_r1, dist_r2, act_par;
 };
 
 }  // namespace
@@ -139,8 +151,17 @@ struct lum_rt {
     bool has_model = false;
     lum_model_desc d{};
     int nq_l = 0, nkv_l = 0, ffn_l = 0, vocab_l = 0;   // this rank's shard sizes
-    Tensor embed, final_norm, lm_head;
+    Tensor embed, final_norm, final_norm_b, lm_head;
     std::vector<LayerW> L;
+    // block_kind 1: chunks of the hidden size, residual row stride, largest sizes over the layers, first mixing layer's values, frequencies
+    int h_chunks = 0, ldx = 0, ldq = 0, q_floats = 0, attn_chunks = 0, act_chunks = 0, vf_floats = 0, head_nt = 0;
+    float* v_first = nullptr;
+    double* pos_freq = nullptr;
+    size_t qkv_floats = 0, attn_floats = 0, h_floats = 0;     // sizes of qkv, attn, h below
+    // rows whose logits the next execute keeps (lum_want_logits), and what the last one kept
+    std::vector<int32_t> want;
+    float* want_logits = nullptr; size_t want_cap = 0; int want_n = 0;
+    int* want_idx = nullptr; size_t want_idx_cap = 0;
     std::vector<void*> allocs;
 
     float *x = nullptr, *qkv = nullptr, *attn = nullptr, *h = nullptr, *logits = nullptr;
@@ -180,6 +201,8 @@ struct lum_rt {
         float *qkv = nullptr, *o = nullptr, *gu = nullptr, *down = nullptr, *logits = nullptr;   // K-split partial planes of the products
         int8_t* xq = nullptr; float* sx = nullptr;                   // quantised activation rows of the product in flight
         std::vector<int32_t> h_tok, h_pos, h_slot;
+        RowOperand in{}, att{}, act{};                               // block_kind 1: operands of the three products
+        float* v_first = nullptr;
     } rows;
     float* yarn_inv = nullptr;        // rope_style 2: inverse-frequency table [head_dim / 2] on the device
     float yarn_factor_cs = 1.0f;      // ... and the factor on cos / sin
@@ -318,6 +341,8 @@ void free_model(lum_rt* rt) {
     rt->g_batch = nullptr; rt->g_batch_n = 0; rt->batch_n = 0; rt->cur_seq = 0;
     rt->rows = lum_rt::Rows();
     rt->b_step = nullptr; rt->b_log = nullptr;
+    rt->v_first = nullptr; rt->pos_freq = nullptr;
+    rt->want.clear(); rt->want_n = 0; rt->want_logits = nullptr; rt->want_cap = 0; rt->want_idx = nullptr; rt->want_idx_cap = 0;
     rt->attn_cnt = nullptr; rt->am_cnt = nullptr; rt->d_sample = nullptr;
     rt->d_page_table = nullptr; rt->page_rows = 0; rt->h_page_table.clear(); rt->page_ref.clear(); rt->page_free.clear();
     rt->mega_ok = false; rt->mega_layers = nullptr; rt->forced_dev = nullptr; rt->gbar = nullptr; rt->abort_flag = nullptr; rt->job_ctr = nullptr; rt->step_ctr = nullptr;
@@ -333,10 +358,31 @@ Tensor* slot_tensor(lum_rt* rt, int slot, int layer) {
         case LUM_S_EMBED: return &rt->embed;
         case LUM_S_FINAL_NORM: return &rt->final_norm;
         case LUM_S_LM_HEAD: return rt->d.tied_head ? nullptr : &rt->lm_head;
+        case LUM_S_FINAL_NORM_BIAS: return rt->d.block_kind == 1 && rt->d.norm_kind == 1 ? &rt->final_norm_b : nullptr;
         default: break;
     }
     if (layer < 0 || layer >= rt->d.n_layers) return nullptr;
     LayerW& l = rt->L[(size_t)layer];
+    if (rt->d.block_kind == 1) {
+        switch (slot) {
+            case LUM_S_ATTN_NORM: return &l.attn_norm;
+            case LUM_S_ATTN_NORM_BIAS: return rt->d.norm_kind == 1 ? &l.attn_norm_b : nullptr;
+            case LUM_S_Q: return &l.q;
+            case LUM_S_K: return &l.k;
+            case LUM_S_V: return &l.v;
+            case LUM_S_O: return &l.o;
+            case LUM_S_Q_NORM: return rt->d.qk_norm ? &l.q_norm : nullptr;
+            case LUM_S_K_NORM: return rt->d.qk_norm ? &l.k_norm : nullptr;
+            case LUM_S_V_MIX: return l.mix ? &l.v_mix : nullptr;
+            case LUM_S_TEMP: return rt->d.dist_bias ? &l.temp : nullptr;
+            case LUM_S_DIST_R1: return rt->d.dist_bias ? &l.dist_r1 : nullptr;
+            case LUM_S_DIST_R2: return rt->d.dist_bias ? &l.dist_r2 : nullptr;
+            case LUM_S_UP: return l.g.ffn > 0 ? &l.up : nullptr;
+            case LUM_S_DOWN: return l.g.ffn > 0 ? &l.down : nullptr;
+            case LUM_S_ACT: return l.g.ffn > 0 ? &l.act_par : nullptr;
+            default: return nullptr;
+        }
+    }
     switch (slot) {
         case LUM_S_ATTN_NORM: return &l.attn_norm;
         case LUM_S_Q: return &l.q;
@@ -367,7 +413,7 @@ Tensor* slot_tensor(lum_rt* rt, int slot, int layer) {
 // (slots 14 and up — the gpt_oss-style tensors — have a range of their own, so the ids of the first 14 never moved)
 uint64_t tensor_id(int slot, int layer) { return slot < 14 ? (uint64_t)layer * 16u + (uint64_t)slot : (1ull << 21) + (uint64_t)layer * 32u + (uint64_t)slot; }
 int slot_layer_for_id(const lum_rt* rt, int slot, int layer) {
-    return (slot == LUM_S_EMBED || slot == LUM_S_FINAL_NORM || slot == LUM_S_LM_HEAD) ? rt->d.n_layers : layer;
+    return (slot == LUM_S_EMBED || slot == LUM_S_FINAL_NORM || slot == LUM_S_LM_HEAD || slot == LUM_S_FINAL_NORM_BIAS) ? rt->d.n_layers : layer;
 }
 
 __global__ void set_state_kernel(DecodeState* st, int pos, int tok, int log, int set_pos_tok, int reset_step) {
@@ -676,10 +722,100 @@ int issue_step(lum_rt* rt, bool with_head, bool pdl, int* n_launch) {
     return 0;
 }
 
+// ---- layers described one by one (block_kind 1) ---------------------------------------------------------------------------
+// A layer is three kernels: [norm + q, k, v, up projections + xIELU] -> [q / k norms + value mixing + cache append + attention] ->
+// [o and down projections together + residual]: both sublayers read the same normalised row, so their first products are one, and
+// their last products add into the same vector, so those are one as well.
+NormArgs block_norm(const lum_rt* rt, const Tensor& gain, const Tensor& bias) {
+    NormArgs n{};
+    n.mode = rt->d.norm_kind == 1 ? NORM_LAYER : NORM_RMS;
+    n.gain = (const float*)gain.w; n.bias = rt->d.norm_kind == 1 ? (const float*)bias.w : nullptr;
+    n.eps = rt->d.rms_eps; n.width = rt->d.hidden;
+    return n;
+}
+DenseArgs block_in(const lum_rt* rt, const LayerW& w) {
+    DenseArgs g{};
+    g.nk = 1; g.kind = kind_of(rt->d.weight_dtype); g.nt = g.n_real = w.nt_in; g.epi = DENSE_STORE; g.mult = 1.0f;
+    g.seg[0].w = w.w_in; g.seg[0].chunks = rt->h_chunks;
+    g.act_row0 = w.act_row0; g.act_par = (const float*)w.act_par.w; g.norm.mode = NORM_NONE; g.status = rt->status;
+    return g;
+}
+DenseArgs block_out(const lum_rt* rt, const LayerW& w) {
+    DenseArgs g{};
+    g.nk = w.g.ffn > 0 ? 2 : 1; g.kind = kind_of(rt->d.weight_dtype); g.nt = (int)((rt->d.hidden + 7) / 8 * 8); g.n_real = rt->d.hidden;
+    g.epi = DENSE_RESID; g.mult = rt->d.residual_mult; g.act_row0 = g.nt; g.norm.mode = NORM_NONE; g.status = rt->status;
+    g.seg[0].w = w.w_o; g.seg[0].chunks = w.o_chunks;
+    g.seg[1].w = w.w_dn; g.seg[1].chunks = w.dn_chunks;
+    return g;
+}
+DenseArgs block_head(const lum_rt* rt) {
+    DenseArgs g{};
+    g.nk = 1; g.kind = kind_of(rt->d.weight_dtype); g.nt = rt->head_nt; g.n_real = rt->d.vocab; g.mult = rt->d.logit_scale;
+    g.seg[0].w = rt->lm_head.w; g.seg[0].chunks = rt->h_chunks; g.act_row0 = g.nt; g.norm.mode = NORM_NONE; g.status = rt->status;
+    return g;
+}
+BandArgs block_band(const lum_rt* rt, const LayerW& w) {
+    const lum_model_desc& d = rt->d;
+    BandArgs t{};
+    t.p.k_off = w.k_off; t.p.v_off = w.v_off;
+    if (d.qk_norm) { t.p.q_gain = (const float*)w.q_norm.w; t.p.k_gain = (const float*)w.k_norm.w; }
+    t.p.eps = d.rms_eps; t.p.scale = w.g.scale; t.p.temp = d.dist_bias ? (const float*)w.temp.w : nullptr;
+    t.p.n_q = w.g.n_q_heads; t.p.n_kv = w.g.n_kv_heads; t.p.dk = w.g.qk_dim; t.p.dv = w.g.v_dim; t.p.dkp = w.dkp; t.p.dvp = w.dvp;
+    t.p.mix = w.mix; t.p.lambda = (const float*)w.v_mix.w; t.p.ld_vfirst = rt->vf_floats;
+    t.k_cache = w.kc; t.v_cache = w.vc; t.kv_bf16 = d.kv_dtype == LUM_BF16;
+    t.window = w.g.window; t.max_seq = d.max_seq; t.max_batch = rt->max_batch;
+    if (d.dist_bias) { t.r1 = (const float*)w.dist_r1.w; t.r2 = (const float*)w.dist_r2.w; }
+    t.status = rt->status;
+    return t;
+}
+// vocabulary projection + sample of one row of the residual stream (a decode step, or the last row of a prompt); returns launches
+int block_head_sample(lum_rt* rt, const float* x, bool pdl, int* n) {
+    DenseArgs g = block_head(rt);
+    g.epi = DENSE_ARGMAX; g.seg[0].x = x; g.y = rt->logits; g.norm = block_norm(rt, rt->final_norm, rt->final_norm_b); g.use_pdl = pdl;
+    g.am.part_val = rt->am_val; g.am.part_idx = rt->am_idx; g.am.counter = rt->am_cnt; g.am.state = rt->state;
+    g.am.tokens_out = rt->sampling ? nullptr : rt->tokens_out; g.am.advance = rt->sampling ? 0 : 1;
+    CU(rt, launch_dense_gemv(g, rt->sm_count, rt->stream)); (*n)++;
+    if (rt->sampling) {
+        SampleArgs sa{};
+        sa.logits = rt->logits; sa.row_stride = (size_t)rt->d.vocab; sa.M = 1; sa.vocab = rt->d.vocab; sa.params = rt->d_sample;
+        sa.seq0 = rt->cur_seq; sa.state = rt->state; sa.tokens_out = rt->tokens_out;
+        CU(rt, launch_sample_rows(sa, rt->stream)); (*n)++;
+    }
+    return 0;
+}
+int issue_step_blocks(lum_rt* rt, bool with_head, bool pdl, int* n_launch) {
+    const lum_model_desc& d = rt->d;
+    cudaStream_t st = rt->stream;
+    int n = 0;
+    EmbedArgs e{};
+    e.table = rt->embed.w; e.kind = rt->embed.kind; e.H = d.hidden; e.x = rt->x; e.state = rt->state; e.status = rt->status; e.pos_freq = rt->pos_freq;
+    e.use_pdl = 0;   // first kernel of the step: ordinary stream order behind the previous step
+    CU(rt, launch_embed(e, st)); n++;
+    for (const LayerW& w : rt->L) {
+        DenseArgs g = block_in(rt, w);
+        g.seg[0].x = rt->x; g.y = rt->qkv; g.act_x = rt->h; g.norm = block_norm(rt, w.attn_norm, w.attn_norm_b); g.use_pdl = pdl;
+        CU(rt, launch_dense_gemv(g, rt->sm_count, st)); n++;
+        BandArgs t = block_band(rt, w);
+        t.p.qkv = rt->qkv; t.p.v_first = rt->v_first; t.M = 1; t.state = rt->state; t.out_x = rt->attn; t.use_pdl = pdl;
+        if (rt->page_rows) t.pg = KvPages{rt->d_page_table + (size_t)rt->cur_seq * rt->pages_per_seq, rt->page_lg, rt->pages_per_seq};
+        else {
+            const size_t esz = t.kv_bf16 ? 2 : 4, row0 = (size_t)rt->cur_seq * d.max_seq;
+            t.k_cache = (char*)t.k_cache + row0 * w.k_elems * esz; t.v_cache = (char*)t.v_cache + row0 * w.v_elems * esz;
+        }
+        CU(rt, launch_band_decode(t, rt->sm_count, st)); n++;
+        DenseArgs o = block_out(rt, w);
+        o.seg[0].x = rt->attn; o.seg[1].x = rt->h; o.y = rt->x; o.use_pdl = pdl;
+        CU(rt, launch_dense_gemv(o, rt->sm_count, st)); n++;
+    }
+    if (with_head) if (int r = block_head_sample(rt, rt->x, pdl, &n)) return r;
+    if (n_launch) *n_launch = n;
+    return 0;
+}
+
 int capture_graph(lum_rt* rt, bool with_head, bool pdl, cudaGraphExec_t* out, int* n_launch) {
     cudaGraph_t g = nullptr;
     CU(rt, cudaStreamBeginCapture(rt->stream, cudaStreamCaptureModeThreadLocal));
-    int r = issue_step(rt, with_head, pdl, n_launch);
+    int r = rt->d.block_kind == 1 ? issue_step_blocks(rt, with_head, pdl, n_launch) : issue_step(rt, with_head, pdl, n_launch);
     cudaError_t e = cudaStreamEndCapture(rt->stream, &g);
     if (r) { if (g) cudaGraphDestroy(g); return r; }
     if (e != cudaSuccess) return fail(rt, LUM_E_CUDA, "cudaStreamEndCapture: %s", cudaGetErrorString(e));
@@ -710,12 +846,15 @@ int run_step(lum_rt* rt, bool with_head) {
         CU(rt, cudaGraphLaunch(with_head ? rt->g_full : rt->g_body, rt->stream));
         return 0;
     }
+    if (rt->d.block_kind == 1) return issue_step_blocks(rt, with_head, rt->cfg.use_pdl != 0, with_head ? &rt->launches_full : nullptr);
     return issue_step(rt, with_head, rt->cfg.use_pdl != 0, with_head ? &rt->launches_full : nullptr);
 }
 
 // ---- paged K/V cache ------------------------------------------------------------------------------------------------
 KvPages kv_pages(const lum_rt* rt) { return rt->page_rows ? KvPages{rt->d_page_table, rt->page_lg, rt->pages_per_seq} : KvPages{nullptr, 0, 0}; }
-size_t kv_row_bytes(const lum_rt* rt) { return (size_t)rt->nkv_l * rt->d.head_dim * (rt->d.kv_dtype == LUM_BF16 ? 2 : 4); }
+size_t kv_row_elems(const LayerW& w, int kind) { return kind ? w.v_elems : w.k_elems; }
+size_t kv_row_bytes(const lum_rt* rt, const LayerW& w, int kind) { return kv_row_elems(w, kind) * (rt->d.kv_dtype == LUM_BF16 ? 2 : 4); }
+size_t kv_rows_total(const lum_rt* rt) { return rt->page_rows ? (size_t)rt->pool_pages * rt->page_rows : (size_t)rt->d.max_batch * rt->d.max_seq; }
 
 int kv_page_upload(lum_rt* rt, int seq, int lp) {
     const size_t i = (size_t)seq * rt->pages_per_seq + lp;
@@ -738,7 +877,6 @@ int kv_page_take(lum_rt* rt, int* page) {
 // any page it shares with another sequence (a shared prefix is read-only).  Contiguous caches: nothing to do.
 int kv_ensure(lum_rt* rt, int seq, int from, int to) {
     if (!rt->page_rows || to <= from) return 0;
-    const size_t page_bytes = (size_t)rt->page_rows * kv_row_bytes(rt);
     for (int lp = from >> rt->page_lg; lp <= (to - 1) >> rt->page_lg; lp++) {
         int& e = rt->h_page_table[(size_t)seq * rt->pages_per_seq + lp];
         if (e >= 0 && rt->page_ref[(size_t)e] == 1) continue;
@@ -746,8 +884,9 @@ int kv_ensure(lum_rt* rt, int seq, int from, int to) {
         if (int r = kv_page_take(rt, &fresh)) return r;
         if (e >= 0) {      // shared: copy what it holds, then let go of it
             for (const LayerW& w : rt->L) {
-                CU(rt, cudaMemcpyAsync((char*)w.kc + fresh * page_bytes, (const char*)w.kc + e * page_bytes, page_bytes, cudaMemcpyDeviceToDevice, rt->stream));
-                CU(rt, cudaMemcpyAsync((char*)w.vc + fresh * page_bytes, (const char*)w.vc + e * page_bytes, page_bytes, cudaMemcpyDeviceToDevice, rt->stream));
+                const size_t kb = rt->page_rows * kv_row_bytes(rt, w, 0), vb = rt->page_rows * kv_row_bytes(rt, w, 1);
+                CU(rt, cudaMemcpyAsync((char*)w.kc + fresh * kb, (const char*)w.kc + e * kb, kb, cudaMemcpyDeviceToDevice, rt->stream));
+                CU(rt, cudaMemcpyAsync((char*)w.vc + fresh * vb, (const char*)w.vc + e * vb, vb, cudaMemcpyDeviceToDevice, rt->stream));
             }
             kv_page_unref(rt, e);
         }
@@ -767,7 +906,7 @@ void kv_release_seq(lum_rt* rt, int seq) {
 template <typename F>
 int kv_for_spans(lum_rt* rt, int seq, int layer, int kind, int rows, const char* who, F fn) {
     char* base = (char*)(kind ? rt->L[(size_t)layer].vc : rt->L[(size_t)layer].kc);
-    const size_t rb = kv_row_bytes(rt);
+    const size_t rb = kv_row_bytes(rt, rt->L[(size_t)layer], kind);
     if (!rt->page_rows) return fn(base + (size_t)seq * rt->d.max_seq * rb, 0, rows);
     for (int r0 = 0; r0 < rows; r0 += rt->page_rows) {
         const int e = rt->h_page_table[(size_t)seq * rt->pages_per_seq + (r0 >> rt->page_lg)];
@@ -782,6 +921,7 @@ int kv_for_spans(lum_rt* rt, int seq, int layer, int kind, int rows, const char*
 // Every linear of the model in the packed tile stream, one GPU: the tensor-core products can take the model's rows.
 bool rows_supported(const lum_rt* rt) {
     const lum_model_desc& d = rt->d;
+    if (rt->has_model && d.block_kind == 1) return true;
     if (!rt->has_model || d.weight_dtype != LUM_Q8_0 || d.tp_size > 1 || (d.head_dim != 64 && d.head_dim != 128)) return false;
     if (d.n_experts > 0 || d.proj_bias || d.attn_sinks || d.sliding_window > 0 || d.rope_style == 2) return false;     // per-token path only
     if (d.n_q_heads / d.n_kv_heads > (d.head_dim == 128 ? 4 : 8)) return false;
@@ -815,12 +955,35 @@ int ensure_rows(lum_rt* rt, int want_rows) {
     if (cap < rt->max_batch) cap = rt->max_batch;
     if (cap < want_rows) cap = want_rows;
     const lum_model_desc& d = rt->d;
-    const int H = d.hidden, hd = d.head_dim, qd = rt->nq_l * hd, kvd = rt->nkv_l * hd, W = qd + 2 * kvd, F = rt->ffn_l;
-    int kmax = H > qd ? H : qd;
-    if (F > kmax) kmax = F;
     if (int r = dev_alloc(rt, (void**)&b.tok, (size_t)cap * 4)) return r;
     if (int r = dev_alloc(rt, (void**)&b.pos, (size_t)cap * 4)) return r;
     if (int r = dev_alloc(rt, (void**)&b.seq, (size_t)cap * 4)) return r;
+    std::vector<int32_t> iota((size_t)cap);
+    for (int i = 0; i < cap; i++) iota[(size_t)i] = i;
+    CU(rt, cudaMemcpyAsync(b.seq, iota.data(), (size_t)cap * 4, cudaMemcpyHostToDevice, rt->stream));
+    if (d.block_kind == 1) {
+        const int kind = kind_of(d.weight_dtype);
+        auto zeroed = [&](void** p, size_t bytes) -> int {          // padding columns of rows and operands stay zero
+            if (int r = dev_alloc(rt, p, bytes)) return r;
+            CU(rt, cudaMemsetAsync(*p, 0, bytes, rt->stream));
+            return 0;
+        };
+        auto operand = [&](RowOperand& o, int chunks) -> int { o.chunks = chunks; return zeroed(&o.p, row_operand_bytes(kind, chunks, cap)); };
+        if (int r = zeroed((void**)&b.xr, (size_t)cap * rt->ldx * 4)) return r;
+        if (int r = dev_alloc(rt, (void**)&b.qkv, (size_t)cap * rt->ldq * 4)) return r;
+        if (int r = dev_alloc(rt, (void**)&b.q_rot, (size_t)cap * rt->q_floats * 4)) return r;
+        if (rt->vf_floats) if (int r = dev_alloc(rt, (void**)&b.v_first, (size_t)cap * rt->vf_floats * 4)) return r;
+        if (int r = operand(b.in, rt->h_chunks)) return r;
+        if (int r = operand(b.att, rt->attn_chunks)) return r;
+        if (rt->act_chunks) if (int r = operand(b.act, rt->act_chunks)) return r;
+        if (rt->max_batch > 1) if (int r = dev_alloc(rt, (void**)&b.logits, (size_t)rt->max_batch * d.vocab * 4)) return r;
+        CU(rt, cudaStreamSynchronize(rt->stream));
+        b.cap = cap;
+        return 0;
+    }
+    const int H = d.hidden, hd = d.head_dim, qd = rt->nq_l * hd, kvd = rt->nkv_l * hd, W = qd + 2 * kvd, F = rt->ffn_l;
+    int kmax = H > qd ? H : qd;
+    if (F > kmax) kmax = F;
     if (int r = dev_alloc(rt, (void**)&b.xr, (size_t)cap * H * 4)) return r;
     if (int r = dev_alloc(rt, (void**)&b.q_rot, (size_t)cap * qd * 4)) return r;
     if (int r = dev_alloc(rt, (void**)&b.attn, (size_t)cap * qd * 4)) return r;
@@ -834,11 +997,96 @@ int ensure_rows(lum_rt* rt, int want_rows) {
         if (int r = dev_alloc(rt, (void**)&b.logits, rows_parts_floats(rt, rt->vocab_l, H, rt->max_batch) * 4)) return r;
     if (int r = dev_alloc(rt, (void**)&b.xq, gemm_xq_bytes(cap, kmax))) return r;
     if (int r = dev_alloc(rt, (void**)&b.sx, gemm_sx_bytes(cap, kmax))) return r;
-    std::vector<int32_t> iota((size_t)cap);
-    for (int i = 0; i < cap; i++) iota[(size_t)i] = i;
-    CU(rt, cudaMemcpyAsync(b.seq, iota.data(), (size_t)cap * 4, cudaMemcpyHostToDevice, rt->stream));
     CU(rt, cudaStreamSynchronize(rt->stream));
     b.cap = cap;
+    return 0;
+}
+
+// The batched step's tail: a sample per row from b.logits [M][vocab] (K-split planes still to be added up when n_parts > 1), fed back on
+// the device; counts its launches.
+int batch_sample(lum_rt* rt, int M, int* d_tok, int* d_pos, const int* d_seq, int n_parts, uint64_t* launches) {
+    lum_rt::Rows& b = rt->rows;
+    const int V = rt->vocab_l;
+    ArgmaxRowsArgs x{};
+    x.logits = b.logits; x.n_parts = n_parts; x.part_stride = (size_t)M * V; x.M = M; x.vocab = V;
+    if (!rt->sampling) { x.row_tok = d_tok; x.row_pos = d_pos; x.log = rt->b_log; x.step = rt->b_step; x.max_steps = rt->d.max_new_tokens; }
+    CU(rt, launch_argmax_rows(x, rt->stream));          // with a sampler set it only adds up the partial planes
+    if (rt->sampling) {
+        SampleArgs sa{};
+        sa.logits = b.logits; sa.row_stride = (size_t)V; sa.M = M; sa.vocab = V; sa.params = rt->d_sample;
+        sa.row_seq = d_seq; sa.row_tok = d_tok; sa.row_pos = d_pos; sa.log = rt->b_log; sa.step = rt->b_step; sa.max_steps = rt->d.max_new_tokens;
+        CU(rt, launch_sample_rows(sa, rt->stream));
+        (*launches)++;
+    }
+    CU(rt, launch_step_advance(rt->b_step, rt->stream));
+    *launches += 2;
+    return 0;
+}
+
+// The wanted rows of a pass (want[w0 .. w0 + n), row indices of the call; c0: first row of the pass): logits into want_logits.
+int block_want_rows(lum_rt* rt, size_t w0, int n, int c0) {
+    lum_rt::Rows& b = rt->rows;
+    std::vector<int32_t> idx((size_t)n);
+    for (int i = 0; i < n; i++) idx[(size_t)i] = rt->want[w0 + i] - c0;
+    CU(rt, cudaMemcpyAsync(rt->want_idx, idx.data(), (size_t)n * 4, cudaMemcpyHostToDevice, rt->stream));     // pageable source: staged before the call returns
+    NormRowsArgs nr{};
+    nr.x = b.xr; nr.ldx = rt->ldx; nr.row_index = rt->want_idx; nr.M = n; nr.norm = block_norm(rt, rt->final_norm, rt->final_norm_b);
+    nr.kind = kind_of(rt->d.weight_dtype); nr.out = b.in;
+    CU(rt, launch_norm_rows(nr, rt->stream));
+    DenseArgs g = block_head(rt);
+    g.epi = DENSE_STORE; g.seg[0].a = b.in.p; g.y = rt->want_logits + w0 * rt->d.vocab; g.ldy = rt->d.vocab; g.M = n;
+    CU(rt, launch_dense_gemm(g, rt->sm_count, rt->stream));
+    rt->n_launches += 2;
+    return 0;
+}
+
+// run_rows for layers described one by one.
+int run_rows_blocks(lum_rt* rt, int M, int* d_tok, int* d_pos, const int* d_seq, int seq0, int head) {
+    const lum_model_desc& d = rt->d;
+    lum_rt::Rows& b = rt->rows;
+    cudaStream_t st = rt->stream;
+    const int kind = kind_of(d.weight_dtype);
+    uint64_t launches = 1;
+    CU(rt, launch_embed_rows_sinusoid(rt->embed.w, rt->embed.kind, d.hidden, d.vocab, d_tok, d_pos, rt->pos_freq, b.xr, rt->ldx, M, rt->status, st));
+    auto norm = [&](const Tensor& gain, const Tensor& bias) -> cudaError_t {
+        NormRowsArgs nr{};
+        nr.x = b.xr; nr.ldx = rt->ldx; nr.M = M; nr.norm = block_norm(rt, gain, bias); nr.kind = kind; nr.out = b.in;
+        launches++;
+        return launch_norm_rows(nr, st);
+    };
+    for (const LayerW& w : rt->L) {
+        CU(rt, norm(w.attn_norm, w.attn_norm_b));
+        RowOperand att = b.att, act = b.act;
+        att.chunks = w.o_chunks; act.chunks = w.dn_chunks;
+        DenseArgs g = block_in(rt, w);
+        g.seg[0].a = b.in.p; g.M = M; g.y = b.qkv; g.ldy = w.act_row0; g.act = act;
+        CU(rt, launch_dense_gemm(g, rt->sm_count, st));
+        BandArgs t = block_band(rt, w);
+        t.p.qkv = b.qkv; t.p.ld = w.act_row0; t.p.v_first = b.v_first; t.M = M; t.pg = kv_pages(rt);
+        t.row_pos = d_pos; t.row_seq = d_seq; t.seq0 = seq0; t.q_out = b.q_rot; t.q = b.q_rot; t.out_kind = kind; t.out = att;
+        CU(rt, launch_qkv_rows(t, st));
+        // many rows of one sequence (a prompt): the tensor-core kernel; few rows, rows of different sequences, f32 caches: one CTA group per row
+        static const int env_tc = [] { const char* e = getenv("LUM_ATTN_TC"); return e ? atoi(e) : 1; }();
+        if (env_tc && M >= 16 && band_prompt_tc_supported(t)) CU(rt, launch_band_prompt_tc(t, st));
+        else CU(rt, launch_band_rows(t, rt->sm_count, st));
+        DenseArgs o = block_out(rt, w);
+        o.seg[0].a = att.p; o.seg[1].a = act.p; o.M = M; o.y = b.xr; o.ldy = rt->ldx;
+        CU(rt, launch_dense_gemm(o, rt->sm_count, st));
+        launches += 4;
+    }
+    if (head == 1) {
+        int n = 0;
+        if (int r = block_head_sample(rt, b.xr + (size_t)(M - 1) * rt->ldx, false, &n)) return r;
+        launches += n;
+    } else if (head == 2) {
+        CU(rt, norm(rt->final_norm, rt->final_norm_b));
+        DenseArgs g = block_head(rt);
+        g.epi = DENSE_STORE; g.seg[0].a = b.in.p; g.y = b.logits; g.ldy = d.vocab; g.M = M;
+        CU(rt, launch_dense_gemm(g, rt->sm_count, st));
+        launches++;
+        if (int r = batch_sample(rt, M, d_tok, d_pos, d_seq, 1, &launches)) return r;
+    }
+    rt->n_launches += launches;
     return 0;
 }
 
@@ -846,6 +1094,7 @@ int ensure_rows(lum_rt* rt, int want_rows) {
 // belongs to sequence seq0.  head: 0 none (the rows only fill the cache), 1 vocabulary projection + greedy sample of the LAST row
 // into the decode state (the end of a prompt), 2 of every row into the batch state (batched decode).
 int run_rows(lum_rt* rt, int M, int* d_tok, int* d_pos, const int* d_seq, int seq0, int head) {
+    if (rt->d.block_kind == 1) return run_rows_blocks(rt, M, d_tok, d_pos, d_seq, seq0, head);
     const lum_model_desc& d = rt->d;
     lum_rt::Rows& b = rt->rows;
     const int H = d.hidden, hd = d.head_dim, qd = rt->nq_l * hd, kvd = rt->nkv_l * hd, W = qd + 2 * kvd, F = rt->ffn_l;
@@ -954,21 +1203,27 @@ int run_rows(lum_rt* rt, int M, int* d_tok, int* d_pos, const int* d_seq, int se
         GemmArgs g{};
         g.nseg = 1; g.seg[0] = {(const unsigned char*)rt->lm_head.w, V, 0};
         CU(rt, gemm(g, H, ks_v, b.logits, V));
-        ArgmaxRowsArgs x{};
-        x.logits = b.logits; x.n_parts = ks_v; x.part_stride = (size_t)M * V; x.M = M; x.vocab = V;
-        if (!rt->sampling) { x.row_tok = d_tok; x.row_pos = d_pos; x.log = rt->b_log; x.step = rt->b_step; x.max_steps = d.max_new_tokens; }
-        CU(rt, launch_argmax_rows(x, st));          // with a sampler set it only adds up the partial planes
-        if (rt->sampling) {
-            SampleArgs sa{};
-            sa.logits = b.logits; sa.row_stride = (size_t)V; sa.M = M; sa.vocab = V; sa.params = rt->d_sample;
-            sa.row_seq = d_seq; sa.row_tok = d_tok; sa.row_pos = d_pos; sa.log = rt->b_log; sa.step = rt->b_step; sa.max_steps = d.max_new_tokens;
-            CU(rt, launch_sample_rows(sa, st));
-            launches++;
-        }
-        CU(rt, launch_step_advance(rt->b_step, st));
-        launches += 2;
+        if (int r2 = batch_sample(rt, M, d_tok, d_pos, d_seq, ks_v, &launches)) return r2;
     }
     rt->n_launches += launches;
+    return 0;
+}
+
+// Logits of row m of the pass of M rows that run_rows has just issued, into place `slot` of want_logits: final norm and vocabulary
+// projection of xr[m] + the partial planes of the last down projection.
+int want_row(lum_rt* rt, int m, int M, size_t slot) {
+    const lum_model_desc& d = rt->d;
+    lum_rt::Rows& b = rt->rows;
+    const int H = d.hidden;
+    const Tensor& hw = d.tied_head ? rt->embed : rt->lm_head;
+    GemvArgs a{};
+    a.status = rt->status; a.use_pdl = 0; a.gain_kind = kind_of(d.embed_dtype); a.eps = rt->eps6; a.wkind = hw.kind;
+    a.nseg = 1; a.seg[0] = {hw.w, hw.s, (int)hw.rows, hw.kc};
+    a.K = H; a.epi = EPI_STORE; a.gain = rt->final_norm.w; a.y = rt->want_logits + slot * rt->vocab_l;
+    a.x = b.xr + (size_t)m * H;
+    a.parts = b.down + (size_t)m * H; a.n_parts = gemm_pick_ksplit(H, M, rt->ffn_l, rt->sm_count); a.part_stride = M * H;
+    CU(rt, launch_gemv(a, rt->sm_count, rt->stream));
+    rt->n_launches++;
     return 0;
 }
 
@@ -977,6 +1232,7 @@ int run_rows(lum_rt* rt, int M, int* d_tok, int* d_pos, const int* d_seq, int se
 int run_prompt_rows(lum_rt* rt, int n, const int32_t* forced, int pos0) {
     if (int r = ensure_rows(rt, 1)) return r;
     lum_rt::Rows& b = rt->rows;
+    size_t want0 = 0;
     for (int c0 = 0; c0 < n; c0 += b.cap) {
         const int M = n - c0 < b.cap ? n - c0 : b.cap;
         const bool last = c0 + M == n;
@@ -991,6 +1247,13 @@ int run_prompt_rows(lum_rt* rt, int n, const int32_t* forced, int pos0) {
             CU(rt, cudaGetLastError());
         }
         if (int r = run_rows(rt, M, b.tok, b.pos, nullptr, rt->cur_seq, last ? 1 : 0)) return r;
+        size_t w1 = want0;
+        while (w1 < rt->want.size() && rt->want[w1] < c0 + M) w1++;
+        if (w1 > want0) {
+            if (rt->d.block_kind == 1) { if (int r = block_want_rows(rt, want0, (int)(w1 - want0), c0)) return r; }
+            else for (size_t i = want0; i < w1; i++) if (int r = want_row(rt, rt->want[i] - c0, M, i)) return r;
+            want0 = w1;
+        }
     }
     rt->n_tokens_run += (uint64_t)n;
     return 0;
@@ -1029,16 +1292,198 @@ int run_tokens(lum_rt* rt, int n, const int32_t* forced, int pos0) {
         rt->n_launches += 1;
         return 0;
     }
+    size_t wi = 0;
     for (int i = 0; i < n; i++) {
         if (forced) {
             set_state_kernel<<<1, 1, 0, rt->stream>>>(rt->state, pos0 + i, forced[i], 0, 1, 0);
             CU(rt, cudaGetLastError());
         }
-        const bool head = !rt->body_only && (!forced || i + 1 == n);
+        const bool wanted = forced && wi < rt->want.size() && rt->want[wi] == i;
+        const bool head = !rt->body_only && (!forced || i + 1 == n || wanted);
         if (int r = run_step(rt, head)) return r;
+        if (wanted) {
+            CU(rt, cudaMemcpyAsync(rt->want_logits + wi * rt->vocab_l, rt->logits, (size_t)rt->vocab_l * 4, cudaMemcpyDeviceToDevice, rt->stream));
+            wi++;
+        }
         rt->n_launches += (uint64_t)(rt->launches_full > 0 ? rt->launches_full - (head ? 0 : 1) : 0);
     }
     rt->n_tokens_run += (uint64_t)n;
+    return 0;
+}
+
+// Checks the paged-cache fields and sets up the host side of the pool; makes `d` the runtime's description.
+int setup_pages(lum_rt* rt, const lum_model_desc& d) {
+    if (d.kv_page_rows < 0 || d.kv_pool_pages < 0 || (d.kv_page_rows == 0 && d.kv_pool_pages != 0)) return fail(rt, LUM_E_INVALID, "kv_page_rows / kv_pool_pages must not be negative; a pool needs a page size");
+    if (d.kv_page_rows > 0) {
+        if (d.kv_page_rows < 64 || (d.kv_page_rows & (d.kv_page_rows - 1)) || d.max_seq % d.kv_page_rows)
+            return fail(rt, LUM_E_INVALID, "kv_page_rows %d must be a power of two >= 64 that divides max_seq %d", d.kv_page_rows, d.max_seq);
+        if (rt->cfg.use_mega) return fail(rt, LUM_E_UNSUPPORTED, "the persistent-kernel executor reads contiguous caches only");
+    }
+    rt->d = d;
+    rt->page_rows = d.kv_page_rows; rt->page_lg = 0; rt->pages_per_seq = 0; rt->pool_pages = 0;
+    if (rt->page_rows) {
+        while ((1 << rt->page_lg) < rt->page_rows) rt->page_lg++;
+        rt->pages_per_seq = d.max_seq / rt->page_rows;
+        rt->pool_pages = d.kv_pool_pages > 0 ? d.kv_pool_pages : d.max_batch * rt->pages_per_seq;
+        rt->h_page_table.assign((size_t)d.max_batch * rt->pages_per_seq, -1);
+        rt->page_ref.assign((size_t)rt->pool_pages, 0);
+        rt->page_free.clear();
+        for (int i = rt->pool_pages - 1; i >= 0; i--) rt->page_free.push_back(i);      // page 0 is handed out first
+    }
+    rt->h_next_pos = 0;
+    return 0;
+}
+
+// What every decoder family needs besides its weights, caches and activations: logits, decode state, sampler, token logs, page table.
+int alloc_decode_state(lum_rt* rt) {
+    const lum_model_desc& d = rt->d;
+#define TRY(x) do { if (int r_ = (x)) return r_; } while (0)
+    TRY(dev_alloc(rt, (void**)&rt->logits, (size_t)rt->vocab_l * 4));
+    TRY(dev_alloc(rt, (void**)&rt->state, sizeof(DecodeState)));
+    TRY(dev_alloc(rt, (void**)&rt->tokens_out, (size_t)d.max_new_tokens * 4));
+    TRY(dev_alloc(rt, (void**)&rt->am_val, kArgmaxSlots * 4));
+    TRY(dev_alloc(rt, (void**)&rt->am_idx, kArgmaxSlots * 4));
+    TRY(dev_alloc(rt, (void**)&rt->am_cnt, 4));
+    if (rt->page_rows) {
+        TRY(dev_alloc(rt, (void**)&rt->d_page_table, rt->h_page_table.size() * 4));
+        cudaMemsetAsync(rt->d_page_table, 0, rt->h_page_table.size() * 4, rt->stream);
+    }
+    TRY(dev_alloc(rt, (void**)&rt->d_sample, sizeof(SampleParams)));
+    cudaMemcpyAsync(rt->d_sample, &rt->samp, sizeof(SampleParams), cudaMemcpyHostToDevice, rt->stream);
+    TRY(dev_alloc(rt, (void**)&rt->status, 4));
+    if (d.max_batch > 1) {
+        TRY(dev_alloc(rt, (void**)&rt->b_step, 4));
+        TRY(dev_alloc(rt, (void**)&rt->b_log, (size_t)d.max_new_tokens * d.max_batch * 4));
+        cudaMemsetAsync(rt->b_step, 0, 4, rt->stream);
+    }
+#undef TRY
+    cudaMemsetAsync(rt->am_cnt, 0, 4, rt->stream);
+    cudaMemsetAsync(rt->status, 0, 4, rt->stream);
+    cudaMemsetAsync(rt->tokens_out, 0, (size_t)d.max_new_tokens * 4, rt->stream);
+    DecodeState s0{};
+    s0.pos = 0; s0.tok = 0; s0.step = 0; s0.max_steps = d.max_new_tokens; s0.vocab = d.vocab; s0.max_seq = d.max_seq; s0.log = 0; s0.last_tok = 0;
+    CU(rt, cudaMemcpyAsync(rt->state, &s0, sizeof s0, cudaMemcpyHostToDevice, rt->stream));
+    CU(rt, cudaStreamSynchronize(rt->stream));
+    rt->dim_s = 1; rt->dim_p = 0;
+    rt->max_batch = d.max_batch; rt->cur_seq = 0; rt->batch_n = 0;
+    rt->prefill_min_rows = rt->cfg.prefill_min_rows > 0 ? rt->cfg.prefill_min_rows : 4;
+    return 0;
+}
+
+// A decoder whose layers are described one by one (block_kind 1): weights in the chunked layout, caches, activations.
+int init_blocks(lum_rt* rt, lum_model_desc d, const lum_layer_desc* layers) {
+    if (d.tp_size <= 0) { d.tp_size = 1; d.tp_rank = 0; }
+    if (d.ep_size <= 0) { d.ep_size = 1; d.ep_rank = 0; }
+    if (d.max_batch <= 0) d.max_batch = 1;
+    if (d.max_new_tokens <= 0) d.max_new_tokens = 4096;
+    if (d.block_kind != 1) return fail(rt, LUM_E_INVALID, "model_init_layers: block_kind %d (1: parallel sublayers)", d.block_kind);
+    if (d.tp_size != 1 || d.ep_size != 1 || rt->tp_size > 1) return fail(rt, LUM_E_UNSUPPORTED, "block_kind 1 runs on one GPU");
+    if (d.max_batch > 1024) return fail(rt, LUM_E_INVALID, "max_batch %d (at most 1024 sequences)", d.max_batch);
+    if (d.n_layers <= 0 || d.hidden <= 0 || d.vocab <= 0 || d.max_seq <= 0) return fail(rt, LUM_E_INVALID, "model dimensions must be positive");
+    if (d.weight_dtype != LUM_F32 && d.weight_dtype != LUM_BF16) return fail(rt, LUM_E_UNSUPPORTED, "block_kind 1: weight dtype must be F32 or BF16");
+    if (d.embed_dtype != LUM_F32 && d.embed_dtype != LUM_BF16) return fail(rt, LUM_E_UNSUPPORTED, "embedding dtype must be F32 or BF16");
+    if (d.kv_dtype != LUM_F32 && d.kv_dtype != LUM_BF16) return fail(rt, LUM_E_UNSUPPORTED, "KV dtype must be F32 or BF16");
+    if (d.norm_kind < 0 || d.norm_kind > 1 || d.pos_kind < 0 || d.pos_kind > 1 || (d.qk_norm != 0 && d.qk_norm != 2) || d.dist_bias < 0 || d.dist_bias > 1 || d.tied_head ||
+        d.n_experts || d.attn_sinks || d.proj_bias || d.rope_style)
+        return fail(rt, LUM_E_UNSUPPORTED, "block_kind 1: norm_kind 0 / 1, pos_kind 0 / 1, qk_norm 0 / 2, dist_bias 0 / 1; no tied head, experts, sinks, biases or rotation");
+    const int kind = kind_of(d.weight_dtype), ek = kind_of(d.embed_dtype), CK = chunk_elems(kind), H = d.hidden;
+    auto up = [](int n, int to) { return (n + to - 1) / to * to; };
+    int first_mix = -1;
+    for (int l = 0; l < d.n_layers; l++) {
+        const lum_layer_desc& g = layers[l];
+        if (g.n_q_heads <= 0 || g.n_kv_heads <= 0 || g.qk_dim <= 0 || g.v_dim <= 0 || g.window < 0 || g.ffn < 0 || g.n_q_heads % g.n_kv_heads)
+            return fail(rt, LUM_E_INVALID, "layer %d: sizes must be positive and the query heads a multiple of the K/V heads", l);
+        if (!band_supported(g.n_q_heads, g.n_kv_heads, head_pad(g.qk_dim), head_pad(g.v_dim))) return fail(rt, LUM_E_UNSUPPORTED, "layer %d: head sizes %d / %d are too large", l, g.qk_dim, g.v_dim);
+        if (g.v_mix) {
+            if (first_mix < 0) first_mix = l;
+            else if (g.n_kv_heads * g.v_dim != layers[first_mix].n_kv_heads * layers[first_mix].v_dim)
+                return fail(rt, LUM_E_INVALID, "layer %d: value mixing needs the %d values of layer %d", l, layers[first_mix].n_kv_heads * layers[first_mix].v_dim, first_mix);
+        }
+    }
+    if (int r = setup_pages(rt, d)) return r;
+#define TRY(x) do { if (int r_ = (x)) { free_model(rt); return r_; } } while (0)
+    rt->nq_l = layers[0].n_q_heads; rt->nkv_l = layers[0].n_kv_heads; rt->ffn_l = layers[0].ffn; rt->vocab_l = d.vocab;
+    rt->ep_size = 1; rt->ep_rank = 0;
+    rt->h_chunks = up(H, CK) / CK; rt->ldx = up(H, 8); rt->head_nt = up(d.vocab, 8);
+    rt->ldq = rt->q_floats = rt->attn_chunks = rt->act_chunks = rt->vf_floats = 0;
+    rt->x2 = rt->part = nullptr; rt->attn_part = nullptr;
+    auto container = [&](void** p, int nt, int chunks) -> int {
+        const size_t bytes = chunked_bytes((size_t)nt, (size_t)chunks);
+        if (int r = dev_alloc(rt, p, bytes)) return r;
+        cudaMemsetAsync(*p, 0, bytes, rt->stream);
+        return 0;
+    };
+    auto part = [&](Tensor& t, void* base, int nt, int row0, int rows, int cols) {
+        t = Tensor();
+        t.w = base; t.kind = kind; t.kc = kLayoutChunked; t.nt = nt; t.crow0 = (size_t)row0;
+        t.rows = t.full_rows = (size_t)rows; t.cols = t.full_cols = t.kdev = (size_t)cols;
+    };
+    auto vec = [&](Tensor& t, int n) { return alloc_tensor(rt, t, WK_F32, 1, n, 1, n, 0, 0); };
+    TRY(alloc_tensor(rt, rt->embed, ek, d.vocab, H, d.vocab, H, 0, 0));
+    TRY(vec(rt->final_norm, H));
+    if (d.norm_kind == 1) TRY(vec(rt->final_norm_b, H));
+    {
+        void* base = nullptr;
+        TRY(container(&base, rt->head_nt, rt->h_chunks));
+        part(rt->lm_head, base, rt->head_nt, 0, d.vocab, H);
+    }
+    rt->L.resize((size_t)d.n_layers);
+    const size_t kv_elem = d.kv_dtype == LUM_BF16 ? 2 : 4;
+    for (int l = 0; l < d.n_layers; l++) {
+        LayerW& w = rt->L[(size_t)l];
+        w.g = layers[l];
+        const int qd = w.g.n_q_heads * w.g.qk_dim, kd = w.g.n_kv_heads * w.g.qk_dim, vd = w.g.n_kv_heads * w.g.v_dim, od = w.g.n_q_heads * w.g.v_dim, F = w.g.ffn;
+        w.dkp = head_pad(w.g.qk_dim); w.dvp = head_pad(w.g.v_dim);
+        w.mix = !w.g.v_mix ? 0 : l == first_mix ? 1 : 2;
+        w.k_off = up(qd, 8); w.v_off = w.k_off + up(kd, 8); w.act_row0 = w.v_off + up(vd, 8);
+        w.nt_in = w.act_row0 + up(F, CK);
+        w.o_chunks = up(od, CK) / CK; w.dn_chunks = up(F, CK) / CK;
+        TRY(container(&w.w_in, w.nt_in, rt->h_chunks));
+        part(w.q, w.w_in, w.nt_in, 0, qd, H); part(w.k, w.w_in, w.nt_in, w.k_off, kd, H); part(w.v, w.w_in, w.nt_in, w.v_off, vd, H);
+        TRY(container(&w.w_o, up(H, 8), w.o_chunks));
+        part(w.o, w.w_o, up(H, 8), 0, H, od);
+        if (F) {
+            part(w.up, w.w_in, w.nt_in, w.act_row0, F, H);
+            TRY(container(&w.w_dn, up(H, 8), w.dn_chunks));
+            part(w.down, w.w_dn, up(H, 8), 0, H, F);
+            TRY(vec(w.act_par, 2));
+        }
+        TRY(vec(w.attn_norm, H));
+        if (d.norm_kind == 1) TRY(vec(w.attn_norm_b, H));
+        if (d.qk_norm) { TRY(vec(w.q_norm, qd)); TRY(vec(w.k_norm, kd)); }
+        if (w.mix) TRY(vec(w.v_mix, 1));
+        if (d.dist_bias) { TRY(vec(w.temp, w.g.n_q_heads)); TRY(vec(w.dist_r1, w.g.n_q_heads)); TRY(vec(w.dist_r2, w.g.n_q_heads)); }
+        w.k_elems = (size_t)w.g.n_kv_heads * w.dkp; w.v_elems = (size_t)w.g.n_kv_heads * w.dvp;
+        TRY(dev_alloc(rt, &w.kc, kv_rows_total(rt) * w.k_elems * kv_elem));
+        TRY(dev_alloc(rt, &w.vc, kv_rows_total(rt) * w.v_elems * kv_elem));
+        cudaMemsetAsync(w.kc, 0, kv_rows_total(rt) * w.k_elems * kv_elem, rt->stream);
+        cudaMemsetAsync(w.vc, 0, kv_rows_total(rt) * w.v_elems * kv_elem, rt->stream);
+        auto most = [](int& a, int b) { if (b > a) a = b; };
+        most(rt->ldq, w.act_row0); most(rt->q_floats, w.g.n_q_heads * w.dkp); most(rt->attn_chunks, w.o_chunks); most(rt->act_chunks, w.dn_chunks);
+        if (w.mix) most(rt->vf_floats, vd);
+    }
+    auto zeroed = [&](float** p, size_t n) -> int {
+        if (int r = dev_alloc(rt, (void**)p, n * 4)) return r;
+        cudaMemsetAsync(*p, 0, n * 4, rt->stream);
+        return 0;
+    };
+    rt->qkv_floats = (size_t)rt->ldq; rt->attn_floats = (size_t)rt->attn_chunks * CK; rt->h_floats = (size_t)rt->act_chunks * CK;
+    TRY(zeroed(&rt->x, (size_t)rt->ldx));
+    TRY(zeroed(&rt->qkv, rt->qkv_floats));
+    TRY(zeroed(&rt->attn, rt->attn_floats));
+    TRY(zeroed(&rt->h, rt->h_floats));
+    if (rt->vf_floats) TRY(zeroed(&rt->v_first, (size_t)rt->vf_floats));
+    if (d.pos_kind == 1) {
+        std::vector<double> f((size_t)(H + 1) / 2);
+        for (size_t i = 0; i < f.size(); i++) f[i] = std::pow(10000.0, -2.0 * (double)i / (double)H);
+        TRY(dev_alloc(rt, (void**)&rt->pos_freq, f.size() * 8));
+        CU(rt, cudaMemcpyAsync(rt->pos_freq, f.data(), f.size() * 8, cudaMemcpyHostToDevice, rt->stream));
+        CU(rt, cudaStreamSynchronize(rt->stream));
+    }
+    TRY(alloc_decode_state(rt));
+#undef TRY
+    rt->use_mega = 0; rt->mega_ok = false;
+    rt->has_model = true;
     return 0;
 }
 
@@ -1046,7 +1491,7 @@ int run_tokens(lum_rt* rt, int n, const int32_t* forced, int pos0) {
 int setup_mega(lum_rt* rt) {
     rt->mega_ok = false;
     const lum_model_desc& d = rt->d;
-    if (d.weight_dtype != LUM_Q8_0 || d.tied_head || d.tp_size > 1 || d.max_batch > 1 || d.kv_page_rows > 0) return 0;
+    if (d.block_kind != 0 || d.weight_dtype != LUM_Q8_0 || d.tied_head || d.tp_size > 1 || d.max_batch > 1 || d.kv_page_rows > 0) return 0;
     if (d.n_experts > 0 || d.proj_bias || d.attn_sinks || d.sliding_window > 0 || d.rope_style == 2) return 0;
     std::vector<MegaLayer> hl((size_t)d.n_layers);
     bool packed = rt->lm_head.kc > 0;
@@ -1106,9 +1551,10 @@ int lum_internal_weight_view(lum_rt* rt, int slot, int layer, lum::WeightView* o
     if (!rt || !rt->has_model) return 1;
     Tensor* t = slot_tensor(rt, slot, layer);
     if (!t || !t->w) return 1;
-    *out = {t->w, t->s, t->kind, t->kc, t->rows, t->cols, t->kdev, t->row0, t->col0, t->full_rows, t->full_cols, rt->cfg.device, rt->stream};
+    *out = {t->w, t->s, t->kind, t->kc, t->rows, t->cols, t->kdev, t->row0, t->col0, t->full_rows, t->full_cols, rt->cfg.device, rt->stream, t->nt, t->crow0};
     return 0;
 }
+int lum_internal_label_style(lum_rt* rt) { return rt->d.block_kind; }
 int lum_internal_fail(lum_rt* rt, int code, const char* msg) { return fail(rt, code, "%s", msg); }
 int lum_internal_parallel(lum_rt* rt, int* tp_size, int* tp_rank, int* ep_size, int* ep_rank) {
     const lum_model_desc& d = rt->d;
@@ -1373,13 +1819,12 @@ int32_t lum_clear_intermediates(lum_rt* rt) {
     if (!rt->has_model) return 0;
     CU(rt, cudaSetDevice(rt->cfg.device));
     const lum_model_desc& d = rt->d;
-    const size_t qd_l = (size_t)rt->nq_l * d.head_dim, kvd_l = (size_t)rt->nkv_l * d.head_dim;
     CU(rt, cudaMemsetAsync(rt->x, 0, (size_t)d.hidden * 4, rt->stream));
-    CU(rt, cudaMemsetAsync(rt->x2, 0, (size_t)d.hidden * 4, rt->stream));
-    CU(rt, cudaMemsetAsync(rt->part, 0, (size_t)2 * d.hidden * 4, rt->stream));
-    CU(rt, cudaMemsetAsync(rt->qkv, 0, (qd_l + 2 * kvd_l) * 4, rt->stream));
-    CU(rt, cudaMemsetAsync(rt->attn, 0, qd_l * 4, rt->stream));
-    CU(rt, cudaMemsetAsync(rt->h, 0, (size_t)rt->ffn_l * 4, rt->stream));
+    if (rt->x2) CU(rt, cudaMemsetAsync(rt->x2, 0, (size_t)d.hidden * 4, rt->stream));
+    if (rt->part) CU(rt, cudaMemsetAsync(rt->part, 0, (size_t)2 * d.hidden * 4, rt->stream));
+    CU(rt, cudaMemsetAsync(rt->qkv, 0, rt->qkv_floats * 4, rt->stream));
+    CU(rt, cudaMemsetAsync(rt->attn, 0, rt->attn_floats * 4, rt->stream));
+    CU(rt, cudaMemsetAsync(rt->h, 0, rt->h_floats * 4, rt->stream));
     CU(rt, cudaMemsetAsync(rt->logits, 0, (size_t)rt->vocab_l * 4, rt->stream));
     if (int r = lum_kv_reset(rt)) return r;
     set_state_kernel<<<1, 1, 0, rt->stream>>>(rt->state, 0, 0, 0, 1, 1);
@@ -1473,7 +1918,7 @@ int32_t lum_profile_llir(lum_rt* rt, const uint8_t* blob, size_t size, uint64_t 
 static int kv_check(lum_rt* rt, int32_t layer, int32_t kind, int32_t rows, size_t bytes, const char* who) {
     if (!rt || !rt->has_model) return fail(rt, LUM_E_INVALID, "%s: no model", who);
     if (layer < 0 || layer >= rt->d.n_layers || rows < 0 || rows > rt->d.max_seq || (kind != 0 && kind != 1)) return fail(rt, LUM_E_INVALID, "%s: bad layer / kind / rows", who);
-    const size_t want = (size_t)rows * kv_row_bytes(rt);
+    const size_t want = (size_t)rows * kv_row_bytes(rt, rt->L[(size_t)layer], kind);
     if (bytes != want) return fail(rt, LUM_E_INVALID, "%s: %d rows are %zu bytes in the cache's own type, got %zu", who, rows, want, bytes);
     return 0;
 }
@@ -1481,7 +1926,7 @@ int32_t lum_kv_save(lum_rt* rt, int32_t layer, int32_t kind, int32_t rows, void*
     if (int r = kv_check(rt, layer, kind, rows, bytes, "kv_save")) return r;
     if (!host_out) return fail(rt, LUM_E_INVALID, "kv_save: null output");
     CU(rt, cudaSetDevice(rt->cfg.device));
-    const size_t rb = kv_row_bytes(rt);
+    const size_t rb = kv_row_bytes(rt, rt->L[(size_t)layer], kind);
     if (int r = kv_for_spans(rt, rt->cur_seq, layer, kind, rows, "kv_save", [&](char* dev, int r0, int n) -> int {
             CU(rt, cudaMemcpyAsync((char*)host_out + (size_t)r0 * rb, dev, (size_t)n * rb, cudaMemcpyDeviceToHost, rt->stream));
             return 0;
@@ -1494,7 +1939,7 @@ int32_t lum_kv_load(lum_rt* rt, int32_t layer, int32_t kind, int32_t rows, const
     if (!host) return fail(rt, LUM_E_INVALID, "kv_load: null input");
     CU(rt, cudaSetDevice(rt->cfg.device));
     if (int r = kv_ensure(rt, rt->cur_seq, 0, rows)) return r;
-    const size_t rb = kv_row_bytes(rt);
+    const size_t rb = kv_row_bytes(rt, rt->L[(size_t)layer], kind);
     if (int r = kv_for_spans(rt, rt->cur_seq, layer, kind, rows, "kv_load", [&](char* dev, int r0, int n) -> int {
             CU(rt, cudaMemcpyAsync(dev, (const char*)host + (size_t)r0 * rb, (size_t)n * rb, cudaMemcpyHostToDevice, rt->stream));
             return 0;
@@ -1525,18 +1970,19 @@ int32_t lum_kv_copy(lum_rt* rt, int32_t src_seq, int32_t dst_seq, int32_t rows) 
         if (rest) {
             if (int r = kv_ensure(rt, dst_seq, full * rt->page_rows, rows)) return r;
             const int se = rt->h_page_table[(size_t)src_seq * rt->pages_per_seq + full], de = rt->h_page_table[(size_t)dst_seq * rt->pages_per_seq + full];
-            const size_t rb = kv_row_bytes(rt), pb = (size_t)rt->page_rows * rb;
             for (const LayerW& w : rt->L) {
-                CU(rt, cudaMemcpyAsync((char*)w.kc + de * pb, (const char*)w.kc + se * pb, rest * rb, cudaMemcpyDeviceToDevice, rt->stream));
-                CU(rt, cudaMemcpyAsync((char*)w.vc + de * pb, (const char*)w.vc + se * pb, rest * rb, cudaMemcpyDeviceToDevice, rt->stream));
+                const size_t kb = kv_row_bytes(rt, w, 0), vb = kv_row_bytes(rt, w, 1), pr = rt->page_rows;
+                CU(rt, cudaMemcpyAsync((char*)w.kc + de * pr * kb, (const char*)w.kc + se * pr * kb, rest * kb, cudaMemcpyDeviceToDevice, rt->stream));
+                CU(rt, cudaMemcpyAsync((char*)w.vc + de * pr * vb, (const char*)w.vc + se * pr * vb, rest * vb, cudaMemcpyDeviceToDevice, rt->stream));
             }
         }
         return 0;
     }
-    const size_t row_bytes = (size_t)rt->nkv_l * rt->d.head_dim * (rt->d.kv_dtype == LUM_BF16 ? 2 : 4), seq_bytes = (size_t)rt->d.max_seq * row_bytes;
+    const size_t ms = (size_t)rt->d.max_seq;
     for (const LayerW& w : rt->L) {
-        CU(rt, cudaMemcpyAsync((char*)w.kc + dst_seq * seq_bytes, (const char*)w.kc + src_seq * seq_bytes, rows * row_bytes, cudaMemcpyDeviceToDevice, rt->stream));
-        CU(rt, cudaMemcpyAsync((char*)w.vc + dst_seq * seq_bytes, (const char*)w.vc + src_seq * seq_bytes, rows * row_bytes, cudaMemcpyDeviceToDevice, rt->stream));
+        const size_t kb = kv_row_bytes(rt, w, 0), vb = kv_row_bytes(rt, w, 1);
+        CU(rt, cudaMemcpyAsync((char*)w.kc + dst_seq * ms * kb, (const char*)w.kc + src_seq * ms * kb, rows * kb, cudaMemcpyDeviceToDevice, rt->stream));
+        CU(rt, cudaMemcpyAsync((char*)w.vc + dst_seq * ms * vb, (const char*)w.vc + src_seq * ms * vb, rows * vb, cudaMemcpyDeviceToDevice, rt->stream));
     }
     return 0;
 }
@@ -1596,7 +2042,7 @@ int32_t lum_get_stats(const lum_rt* rt, lum_stats* out) {
         uint64_t wb = 0;
         lum_model_weight_bytes(rt, &wb);
         out->weight_bytes_per_token = wb;
-        out->kv_bytes_per_position = (uint64_t)rt->d.n_layers * 2 * rt->nkv_l * rt->d.head_dim * (rt->d.kv_dtype == LUM_BF16 ? 2 : 4);
+        for (const LayerW& w : rt->L) out->kv_bytes_per_position += kv_row_bytes(rt, w, 0) + kv_row_bytes(rt, w, 1);
         out->launches_per_step = rt->launches_full;
     }
     return 0;
@@ -1713,6 +2159,7 @@ int32_t lum_batch_get_logits(lum_rt* rt, int32_t seq, float* host_out, size_t n)
 int32_t lum_debug_wait_timeout(lum_rt* rt) {
     if (!rt || !rt->has_model) return fail(rt, LUM_E_INVALID, "debug_wait_timeout: no model");
     CU(rt, cudaSetDevice(rt->cfg.device));
+    if (rt->d.block_kind != 0) return fail(rt, LUM_E_UNSUPPORTED, "debug_wait_timeout: needs a model with streaming projections");
     const int H = rt->d.hidden;
     LayerW& w = rt->L[0];
     void* ll = nullptr;
@@ -1798,11 +2245,13 @@ int32_t lum_tp_peer_import(lum_rt* rt, const uint8_t* handles, int32_t n) {
 
 int32_t lum_model_init(lum_rt* rt, const lum_model_desc* dp) {
     if (!rt || !dp) return LUM_E_INVALID;
+    if (dp->block_kind != 0) return fail(rt, LUM_E_INVALID, "model_init: block_kind %d describes its layers one by one (lum_model_init_layers)", dp->block_kind);
     CU(rt, cudaSetDevice(rt->cfg.device));
     cudaStreamSynchronize(rt->stream);
     free_model(rt);
     if (rt->generic) { lum_generic_free(rt->generic); rt->generic = nullptr; }      // a decoder replaces a loaded graph of primitive ops
     lum_model_desc d = *dp;
+    if (d.qk_norm) d.qk_norm = 1;                                                   // (the projection-wide norm is a block_kind 1 mechanism)
     if (d.tp_size <= 0) { d.tp_size = 1; d.tp_rank = 0; }
     if (d.max_batch <= 0) d.max_batch = 1;
     if (d.max_batch > 1024) return fail(rt, LUM_E_INVALID, "max_batch %d (at most 1024 sequences)", d.max_batch);
@@ -1835,24 +2284,7 @@ int32_t lum_model_init(lum_rt* rt, const lum_model_desc* dp) {
     if (d.rope_style == 2 && (d.yarn_factor <= 0.0f || d.yarn_beta_fast <= 0.0f || d.yarn_beta_slow <= 0.0f || d.yarn_orig_max_pos <= 0.0f))
         return fail(rt, LUM_E_INVALID, "rope_style 2 needs the yarn_* parameters");
     if (d.n_q_heads % tp || (d.n_q_heads / tp) % (d.n_kv_heads / tp)) return fail(rt, LUM_E_INVALID, "query heads must divide by tp_size");
-    if (d.kv_page_rows < 0 || d.kv_pool_pages < 0 || (d.kv_page_rows == 0 && d.kv_pool_pages != 0)) return fail(rt, LUM_E_INVALID, "kv_page_rows / kv_pool_pages must not be negative; a pool needs a page size");
-    if (d.kv_page_rows > 0) {
-        if (d.kv_page_rows < 64 || (d.kv_page_rows & (d.kv_page_rows - 1)) || d.max_seq % d.kv_page_rows)
-            return fail(rt, LUM_E_INVALID, "kv_page_rows %d must be a power of two >= 64 that divides max_seq %d", d.kv_page_rows, d.max_seq);
-        if (rt->cfg.use_mega) return fail(rt, LUM_E_UNSUPPORTED, "the persistent-kernel executor reads contiguous caches only");
-    }
-    rt->d = d;
-    rt->page_rows = d.kv_page_rows; rt->page_lg = 0; rt->pages_per_seq = 0; rt->pool_pages = 0;
-    if (rt->page_rows) {
-        while ((1 << rt->page_lg) < rt->page_rows) rt->page_lg++;
-        rt->pages_per_seq = d.max_seq / rt->page_rows;
-        rt->pool_pages = d.kv_pool_pages > 0 ? d.kv_pool_pages : d.max_batch * rt->pages_per_seq;
-        rt->h_page_table.assign((size_t)d.max_batch * rt->pages_per_seq, -1);
-        rt->page_ref.assign((size_t)rt->pool_pages, 0);
-        rt->page_free.clear();
-        for (int i = rt->pool_pages - 1; i >= 0; i--) rt->page_free.push_back(i);      // page 0 is handed out first
-    }
-    rt->h_next_pos = 0;
+    if (int r2 = setup_pages(rt, d)) return r2;
     rt->nq_l = d.n_q_heads / tp; rt->nkv_l = d.n_kv_heads / tp; rt->ffn_l = d.ffn / tp; rt->vocab_l = d.vocab / tp;
     const int H = d.hidden, hd = d.head_dim, r = d.tp_rank;
     const int wk = kind_of(d.weight_dtype), ek = kind_of(d.embed_dtype);
@@ -1903,7 +2335,8 @@ int32_t lum_model_init(lum_rt* rt, const lum_model_desc* dp) {
             TRY(alloc_tensor(rt, w.q_norm, ek, 1, hd, 1, hd, 0, 0));
             TRY(alloc_tensor(rt, w.k_norm, ek, 1, hd, 1, hd, 0, 0));
         }
-        const size_t cache_bytes = rt->page_rows ? (size_t)rt->pool_pages * rt->page_rows * kvd_l * kv_elem : (size_t)d.max_batch * d.max_seq * kvd_l * kv_elem;
+        w.k_elems = w.v_elems = kvd_l;
+        const size_t cache_bytes = kv_rows_total(rt) * kvd_l * kv_elem;
         TRY(dev_alloc(rt, &w.kc, cache_bytes));
         TRY(dev_alloc(rt, &w.vc, cache_bytes));
         cudaMemsetAsync(w.kc, 0, cache_bytes, rt->stream);
@@ -1970,55 +2403,30 @@ int32_t lum_model_init(lum_rt* rt, const lum_model_desc* dp) {
         cudaMemsetAsync(rt->tp_seq, 0, 4, rt->stream);
         cudaMemsetAsync(rt->peer_ticket, 0, 4, rt->stream);
     }
-    TRY(dev_alloc(rt, (void**)&rt->qkv, (qd_l + 2 * kvd_l) * 4));
+    rt->qkv_floats = qd_l + 2 * kvd_l;
+    TRY(dev_alloc(rt, (void**)&rt->qkv, rt->qkv_floats * 4));
     {
         // inputs of the K-sharded projections: as long as the (possibly zero-padded) K of the device layout, zero beyond the data
         const size_t attn_len = rt->L[0].o.kdev > qd_l ? rt->L[0].o.kdev : qd_l, h_len = rt->L[0].down.kdev > (size_t)rt->ffn_l ? rt->L[0].down.kdev : (size_t)rt->ffn_l;
+        rt->attn_floats = attn_len; rt->h_floats = h_len;
         TRY(dev_alloc(rt, (void**)&rt->attn, attn_len * 4));
         TRY(dev_alloc(rt, (void**)&rt->h, h_len * 4));
         cudaMemsetAsync(rt->attn, 0, attn_len * 4, rt->stream);
         cudaMemsetAsync(rt->h, 0, h_len * 4, rt->stream);
     }
-    TRY(dev_alloc(rt, (void**)&rt->logits, (size_t)rt->vocab_l * 4));
-    TRY(dev_alloc(rt, (void**)&rt->state, sizeof(DecodeState)));
-    TRY(dev_alloc(rt, (void**)&rt->tokens_out, (size_t)d.max_new_tokens * 4));
     TRY(dev_alloc(rt, (void**)&rt->attn_part, (size_t)rt->nkv_l * splits * G * (hd + 2) * 4));
     TRY(dev_alloc(rt, (void**)&rt->attn_cnt, (size_t)rt->nkv_l * 4));
-    TRY(dev_alloc(rt, (void**)&rt->am_val, kArgmaxSlots * 4));
-    TRY(dev_alloc(rt, (void**)&rt->am_idx, kArgmaxSlots * 4));
-    TRY(dev_alloc(rt, (void**)&rt->am_cnt, 4));
-    if (rt->page_rows) {
-        TRY(dev_alloc(rt, (void**)&rt->d_page_table, rt->h_page_table.size() * 4));
-        cudaMemsetAsync(rt->d_page_table, 0, rt->h_page_table.size() * 4, rt->stream);
-    }
-    TRY(dev_alloc(rt, (void**)&rt->d_sample, sizeof(SampleParams)));
-    cudaMemcpyAsync(rt->d_sample, &rt->samp, sizeof(SampleParams), cudaMemcpyHostToDevice, rt->stream);
+    TRY(alloc_decode_state(rt));
     TRY(dev_alloc(rt, (void**)&rt->step_ctr, ((size_t)4 * d.n_layers + 1) * sizeof(unsigned int)));
     cudaMemsetAsync(rt->step_ctr, 0, ((size_t)4 * d.n_layers + 1) * sizeof(unsigned int), rt->stream);
-    TRY(dev_alloc(rt, (void**)&rt->status, 4));
 #undef TRY
     cudaMemsetAsync(rt->attn_cnt, 0, (size_t)rt->nkv_l * 4, rt->stream);
-    cudaMemsetAsync(rt->am_cnt, 0, 4, rt->stream);
-    cudaMemsetAsync(rt->status, 0, 4, rt->stream);
-    cudaMemsetAsync(rt->tokens_out, 0, (size_t)d.max_new_tokens * 4, rt->stream);
-    DecodeState s0{};
-    s0.pos = 0; s0.tok = 0; s0.step = 0; s0.max_steps = d.max_new_tokens; s0.vocab = d.vocab; s0.max_seq = d.max_seq; s0.log = 0; s0.last_tok = 0;
-    CU(rt, cudaMemcpyAsync(rt->state, &s0, sizeof s0, cudaMemcpyHostToDevice, rt->stream));
-    CU(rt, cudaStreamSynchronize(rt->stream));
 
     rt->eps6 = round6(d.rms_eps);
     rt->c_inv_d = round6(1.0 / (double)hd);
     rt->c_ln_theta = round6(std::log((double)d.rope_theta));
     rt->c_log2e = round6(1.0 / std::log(2.0));
     rt->c_half_pi = round6(1.5707963267948966);
-    rt->dim_s = 1; rt->dim_p = 0;
-    rt->max_batch = d.max_batch; rt->cur_seq = 0; rt->batch_n = 0;
-    rt->prefill_min_rows = rt->cfg.prefill_min_rows > 0 ? rt->cfg.prefill_min_rows : 4;
-    if (d.max_batch > 1) {
-        if (int r2 = dev_alloc(rt, (void**)&rt->b_step, 4)) { free_model(rt); return r2; }
-        if (int r2 = dev_alloc(rt, (void**)&rt->b_log, (size_t)d.max_new_tokens * d.max_batch * 4)) { free_model(rt); return r2; }
-        cudaMemsetAsync(rt->b_step, 0, 4, rt->stream);
-    }
     rt->has_model = true;
     rt->use_mega = rt->cfg.use_mega;
     rt->kv_prefetch = true;
@@ -2037,6 +2445,16 @@ int32_t lum_model_init(lum_rt* rt, const lum_model_desc* dp) {
     return 0;
 }
 
+int32_t lum_model_init_layers(lum_rt* rt, const lum_model_desc* dp, const lum_layer_desc* layers) {
+    if (!rt || !dp || !layers) return fail(rt, LUM_E_INVALID, "model_init_layers: null argument");
+    CU(rt, cudaSetDevice(rt->cfg.device));
+    cudaStreamSynchronize(rt->stream);
+    free_model(rt);
+    if (rt->generic) { lum_generic_free(rt->generic); rt->generic = nullptr; }
+    if (rt->llir) { lum_llir_free_plan(rt->llir); rt->llir = nullptr; }             // no graph stands behind this model
+    return init_blocks(rt, *dp, layers);
+}
+
 int32_t lum_model_synth(lum_rt* rt, uint64_t seed) {
     if (!rt || !rt->has_model) return fail(rt, LUM_E_INVALID, "synth: no model");
     CU(rt, cudaSetDevice(rt->cfg.device));
@@ -2046,7 +2464,15 @@ int32_t lum_model_synth(lum_rt* rt, uint64_t seed) {
         if (!t) return 0;
         const uint64_t tid = tensor_id(slot, slot_layer_for_id(rt, slot, layer));
         cudaError_t e;
-        if (t->kind == WK_Q8) e = launch_synth_q8(seed, tid, (int8_t*)t->w, t->s, t->rows, t->kdev, t->row0, t->col0, t->full_cols, t->kc, rt->stream, t->cols);
+        if (t->kc == kLayoutChunked) {          // generated row-major, then laid out
+            void* tmp = nullptr;
+            if (cudaMalloc(&tmp, t->rows * t->cols * (t->kind == WK_BF16 ? 2 : 4) + 64) != cudaSuccess) return fail(rt, LUM_E_NOMEM, "synth: staging buffer");
+            e = launch_synth_normal(seed, tid, tmp, t->kind, t->rows, t->cols, 0, 0, t->cols, ones, rt->stream);
+            if (e == cudaSuccess) e = launch_chunked_pack(tmp, (uint32_t)t->kind, t->rows, t->cols, t->w, t->kind, t->nt, t->crow0, rt->stream);
+            cudaStreamSynchronize(rt->stream);
+            cudaFree(tmp);
+        }
+        else if (t->kind == WK_Q8) e = launch_synth_q8(seed, tid, (int8_t*)t->w, t->s, t->rows, t->kdev, t->row0, t->col0, t->full_cols, t->kc, rt->stream, t->cols);
         else e = launch_synth_normal(seed, tid, t->w, t->kind, t->rows, t->cols, t->row0, t->col0, t->full_cols, ones, rt->stream);
         if (e != cudaSuccess) return fail(rt, LUM_E_CUDA, "synth slot %d layer %d: %s", slot, layer, cudaGetErrorString(e));
         return 0;
@@ -2054,11 +2480,13 @@ int32_t lum_model_synth(lum_rt* rt, uint64_t seed) {
     if (int r = fill(LUM_S_EMBED, 0, 0)) return r;
     if (int r = fill(LUM_S_FINAL_NORM, 0, 1)) return r;
     if (int r = fill(LUM_S_LM_HEAD, 0, 0)) return r;
+    if (int r = fill(LUM_S_FINAL_NORM_BIAS, 0, 0)) return r;
     for (int l = 0; l < d.n_layers; l++) {
         const int lin[] = {LUM_S_Q, LUM_S_K, LUM_S_V, LUM_S_O, LUM_S_GATE, LUM_S_UP, LUM_S_DOWN, LUM_S_ROUTER, LUM_S_ROUTER_BIAS, LUM_S_EXP_GATE_UP,
-                           LUM_S_EXP_GATE_UP_BIAS, LUM_S_EXP_DOWN, LUM_S_EXP_DOWN_BIAS, LUM_S_Q_BIAS, LUM_S_K_BIAS, LUM_S_V_BIAS, LUM_S_O_BIAS, LUM_S_SINKS};
+                           LUM_S_EXP_GATE_UP_BIAS, LUM_S_EXP_DOWN, LUM_S_EXP_DOWN_BIAS, LUM_S_Q_BIAS, LUM_S_K_BIAS, LUM_S_V_BIAS, LUM_S_O_BIAS, LUM_S_SINKS,
+                           LUM_S_ATTN_NORM_BIAS, LUM_S_V_MIX, LUM_S_ACT};
         for (int s : lin) if (int r = fill(s, l, 0)) return r;
-        const int nrm[] = {LUM_S_ATTN_NORM, LUM_S_MLP_NORM, LUM_S_Q_NORM, LUM_S_K_NORM};
+        const int nrm[] = {LUM_S_ATTN_NORM, LUM_S_MLP_NORM, LUM_S_Q_NORM, LUM_S_K_NORM, LUM_S_TEMP, LUM_S_DIST_R1, LUM_S_DIST_R2};
         for (int s : nrm) if (int r = fill(s, l, 1)) return r;
     }
     CU(rt, cudaStreamSynchronize(rt->stream));
@@ -2073,8 +2501,16 @@ int32_t lum_model_get_weight_f32(lum_rt* rt, int32_t slot, int32_t layer, size_t
     if (offset + n > t->rows * t->cols) return fail(rt, LUM_E_INVALID, "get_weight: range outside the tensor");
     if (t->kind == WK_Q8 && (offset % t->cols || n % t->cols)) return fail(rt, LUM_E_INVALID, "get_weight: Q8_0 ranges must cover whole rows");
     float* tmp = nullptr;
-    cudaError_t e = cudaMalloc((void**)&tmp, n * 4 + 16);
+    const bool chunked = t->kc == kLayoutChunked;
+    cudaError_t e = cudaMalloc((void**)&tmp, (chunked ? t->rows * t->cols : n) * 4 + 16);
     if (e != cudaSuccess) return fail(rt, LUM_E_NOMEM, "get_weight: %s", cudaGetErrorString(e));
+    if (chunked) {
+        e = launch_chunked_unpack(t->w, t->kind, t->nt, t->crow0, t->rows, t->cols, tmp, nullptr, rt->stream);
+        if (e == cudaSuccess) e = cudaMemcpyAsync(host_out, tmp + offset, n * 4, cudaMemcpyDeviceToHost, rt->stream);
+        if (e == cudaSuccess) e = cudaStreamSynchronize(rt->stream);
+        cudaFree(tmp);
+        return e == cudaSuccess ? 0 : fail(rt, LUM_E_CUDA, "get_weight: %s", cudaGetErrorString(e));
+    }
     if (t->kind == WK_Q8) e = launch_q8_dequant_rows(t->w, t->s, (int)t->kdev, t->kc, offset / t->cols, n / t->cols, tmp, rt->stream, (int)t->cols);
     else e = launch_to_f32((const uint8_t*)t->w + offset * (t->kind == WK_BF16 ? 2 : 4), t->kind, tmp, n, rt->stream);
     if (e == cudaSuccess) e = cudaMemcpyAsync(host_out, tmp, n * 4, cudaMemcpyDeviceToHost, rt->stream);
@@ -2091,6 +2527,7 @@ int32_t lum_model_weight_bytes(const lum_rt* rt, uint64_t* bytes) {
         b += w.q.bytes() + w.k.bytes() + w.v.bytes() + w.o.bytes() + w.gate.bytes() + w.up.bytes() + w.down.bytes();
         b += w.attn_norm.bytes() + w.mlp_norm.bytes();
         if (rt->d.qk_norm) b += w.q_norm.bytes() + w.k_norm.bytes();
+        b += w.attn_norm_b.bytes() + w.v_mix.bytes() + w.temp.bytes() + w.dist_r1.bytes() + w.dist_r2.bytes() + w.act_par.bytes();
         if (rt->d.n_experts > 0) {
             // a token reads the router and top_k experts (gate_up + down, their biases)
             const uint64_t H = (uint64_t)rt->d.hidden, F = (uint64_t)rt->d.ffn, eb = rt->embed.kind == WK_BF16 ? 2 : 4;
@@ -2108,15 +2545,11 @@ int32_t lum_model_weight_bytes(const lum_rt* rt, uint64_t* bytes) {
 int32_t lum_kv_reset(lum_rt* rt) {
     if (!rt || !rt->has_model) return fail(rt, LUM_E_INVALID, "kv_reset: no model");
     CU(rt, cudaSetDevice(rt->cfg.device));
-    size_t bytes = (size_t)rt->max_batch * rt->d.max_seq * kv_row_bytes(rt);   // every sequence
-    if (rt->page_rows) {
-        bytes = (size_t)rt->pool_pages * rt->page_rows * kv_row_bytes(rt);
-        for (int sq = 0; sq < rt->max_batch; sq++) kv_release_seq(rt, sq);
-    }
+    if (rt->page_rows) for (int sq = 0; sq < rt->max_batch; sq++) kv_release_seq(rt, sq);
     rt->h_next_pos = 0;
-    for (LayerW& w : rt->L) {
-        CU(rt, cudaMemsetAsync(w.kc, 0, bytes, rt->stream));
-        CU(rt, cudaMemsetAsync(w.vc, 0, bytes, rt->stream));
+    for (LayerW& w : rt->L) {       // every sequence
+        CU(rt, cudaMemsetAsync(w.kc, 0, kv_rows_total(rt) * kv_row_bytes(rt, w, 0), rt->stream));
+        CU(rt, cudaMemsetAsync(w.vc, 0, kv_rows_total(rt) * kv_row_bytes(rt, w, 1), rt->stream));
     }
     rt->dim_p = 0;
     return 0;
@@ -2124,14 +2557,13 @@ int32_t lum_kv_reset(lum_rt* rt) {
 
 int32_t lum_kv_read(lum_rt* rt, int32_t layer, int32_t kind, int32_t rows, float* host_out) {
     if (!rt || !rt->has_model || !host_out) return fail(rt, LUM_E_INVALID, "kv_read: no model or null output");
-    if (layer < 0 || layer >= rt->d.n_layers || rows < 0 || rows > rt->d.max_seq) return fail(rt, LUM_E_INVALID, "kv_read: bad layer/rows");
+    if (layer < 0 || layer >= rt->d.n_layers || rows < 0 || rows > rt->d.max_seq || (kind != 0 && kind != 1)) return fail(rt, LUM_E_INVALID, "kv_read: bad layer/kind/rows");
     CU(rt, cudaSetDevice(rt->cfg.device));
-    const size_t n = (size_t)rows * rt->nkv_l * rt->d.head_dim;
+    const size_t row_elems = kv_row_elems(rt->L[(size_t)layer], kind), n = (size_t)rows * row_elems;
     if (!n) return 0;
     float* tmp = nullptr;
     cudaError_t e = cudaMalloc((void**)&tmp, n * 4);
     if (e != cudaSuccess) return fail(rt, LUM_E_NOMEM, "kv_read: %s", cudaGetErrorString(e));
-    const size_t row_elems = (size_t)rt->nkv_l * rt->d.head_dim;
     const int rc = kv_for_spans(rt, rt->cur_seq, layer, kind, rows, "kv_read", [&](char* dev, int r0, int nr) -> int {
         const cudaError_t e2 = launch_to_f32(dev, rt->d.kv_dtype == LUM_BF16 ? WK_BF16 : WK_F32, tmp + (size_t)r0 * row_elems, (size_t)nr * row_elems, rt->stream);
         return e2 == cudaSuccess ? 0 : fail(rt, LUM_E_CUDA, "kv_read: %s", cudaGetErrorString(e2));
@@ -2179,7 +2611,35 @@ int32_t lum_execute(lum_rt* rt) {
         const int tok = rt->tokens_in[(size_t)i];
         if (tok < 0 || tok >= rt->d.vocab) return fail(rt, LUM_E_INVALID, "execute: token id %d outside the vocabulary", tok);
     }
-    return run_tokens(rt, (int)s, rt->tokens_in.data(), (int)p);
+    rt->want_n = 0;
+    if (!rt->want.empty()) {
+        if (rt->want.back() >= (int64_t)s) { rt->want.clear(); return fail(rt, LUM_E_INVALID, "execute: logits of a row beyond 's' = %llu were asked for", (unsigned long long)s); }
+        if (rt->d.tp_size > 1 || (rt->mega_ok && rt->use_mega)) { rt->want.clear(); return fail(rt, LUM_E_UNSUPPORTED, "execute: logits of chosen rows need one GPU and a kernel-per-op executor"); }
+        const size_t n = rt->want.size();
+        if (n * rt->vocab_l > rt->want_cap) { if (int r = dev_alloc(rt, (void**)&rt->want_logits, n * rt->vocab_l * 4)) return r; rt->want_cap = n * rt->vocab_l; }
+        if (n > rt->want_idx_cap) { if (int r = dev_alloc(rt, (void**)&rt->want_idx, n * 4)) return r; rt->want_idx_cap = n; }
+    }
+    const int r = run_tokens(rt, (int)s, rt->tokens_in.data(), (int)p);
+    if (!r) rt->want_n = (int)rt->want.size();
+    rt->want.clear();
+    return r;
+}
+
+int32_t lum_want_logits(lum_rt* rt, const int32_t* rows, int32_t n) {
+    if (!rt || !rt->has_model || n < 0 || (n > 0 && !rows)) return fail(rt, LUM_E_INVALID, "want_logits: no model or null rows");
+    for (int i = 0; i < n; i++)
+        if (rows[i] < 0 || (i > 0 && rows[i] <= rows[i - 1])) return fail(rt, LUM_E_INVALID, "want_logits: rows must be increasing");
+    if (n > 0) rt->want.assign(rows, rows + n); else rt->want.clear();
+    return 0;
+}
+
+int32_t lum_get_wanted(lum_rt* rt, float* host_out, size_t n) {
+    if (!rt || !rt->has_model || !host_out) return fail(rt, LUM_E_INVALID, "get_wanted: no model or null output");
+    if (n != (size_t)rt->want_n * rt->vocab_l) return fail(rt, LUM_E_INVALID, "get_wanted: the last execute kept %d rows of %d logits, asked for %zu values", rt->want_n, rt->vocab_l, n);
+    CU(rt, cudaSetDevice(rt->cfg.device));
+    if (n) CU(rt, cudaMemcpyAsync(host_out, rt->want_logits, n * 4, cudaMemcpyDeviceToHost, rt->stream));
+    CU(rt, cudaStreamSynchronize(rt->stream));
+    return check_status(rt);
 }
 
 int32_t lum_get_logits(lum_rt* rt, float* host_out, size_t n) {

@@ -113,6 +113,25 @@ pub struct lum_model_desc {
     pub ep_rank: i32,
     pub kv_page_rows: i32,
     pub kv_pool_pages: i32,
+    pub block_kind: i32,
+    pub norm_kind: i32,
+    pub pos_kind: i32,
+    pub dist_bias: i32,
+    pub residual_mult: f32,
+    pub logit_scale: f32,
+}
+
+#[repr(C)]
+#[derive(Clone, Copy, Debug, Default)]
+pub struct lum_layer_desc {
+    pub n_q_heads: i32,
+    pub n_kv_heads: i32,
+    pub qk_dim: i32,
+    pub v_dim: i32,
+    pub window: i32,
+    pub v_mix: i32,
+    pub ffn: i32,
+    pub scale: f32,
 }
 
 #[repr(C)]
@@ -145,6 +164,7 @@ unsafe extern "C" {
     pub fn lum_device_info(rt: *const lum_rt, sm_count: *mut i32, mem_bytes: *mut u64, cc: *mut i32) -> i32;
 
     pub fn lum_model_init(rt: *mut lum_rt, desc: *const lum_model_desc) -> i32;
+    pub fn lum_model_init_layers(rt: *mut lum_rt, desc: *const lum_model_desc, layers: *const lum_layer_desc) -> i32;
     pub fn lum_model_set_weight(rt: *mut lum_rt, slot: i32, layer: i32, data: *const c_void, bytes: usize, dtype: u32) -> i32;
     pub fn lum_model_set_weight_shard(rt: *mut lum_rt, slot: i32, layer: i32, data: *const c_void, bytes: usize, dtype: u32) -> i32;
     pub fn lum_load_safetensors(rt: *mut lum_rt, path: *const c_char, n_loaded: *mut i32, n_ignored: *mut i32) -> i32;
@@ -177,6 +197,8 @@ unsafe extern "C" {
     pub fn lum_set_tokens(rt: *mut lum_rt, ids: *const i32, n: usize) -> i32;
     pub fn lum_execute(rt: *mut lum_rt) -> i32;
     pub fn lum_get_logits(rt: *mut lum_rt, host_out: *mut f32, n: usize) -> i32;
+    pub fn lum_want_logits(rt: *mut lum_rt, rows: *const i32, n: i32) -> i32;
+    pub fn lum_get_wanted(rt: *mut lum_rt, host_out: *mut f32, n: usize) -> i32;
     pub fn lum_get_token(rt: *mut lum_rt, token: *mut i32) -> i32;
     pub fn lum_decode_greedy(rt: *mut lum_rt, n_steps: i32) -> i32;
     pub fn lum_get_decoded(rt: *mut lum_rt, host_out: *mut i32, n: usize) -> i32;

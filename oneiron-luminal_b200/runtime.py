@@ -13,7 +13,7 @@ from __future__ import annotations
 
 import ctypes as C
 import os
-from typing import Dict, Iterable, Optional, Sequence
+from typing import Dict, Iterable, List, Optional, Sequence
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 _LIB_NAME = "liblum_b200.so"
@@ -33,6 +33,7 @@ SLOT = {
     "gate": 7, "up": 8, "down": 9, "final_norm": 10, "lm_head": 11, "q_norm": 12, "k_norm": 13,
     "q_bias": 14, "k_bias": 15, "v_bias": 16, "o_bias": 17, "sinks": 18, "router": 19, "router_bias": 20,
     "exp_gate_up": 21, "exp_gate_up_bias": 22, "exp_down": 23, "exp_down_bias": 24,
+    "attn_norm_bias": 25, "final_norm_bias": 26, "v_mix": 27, "temp": 28, "dist_r1": 29, "dist_r2": 30, "act": 31,
 }
 
 
@@ -55,6 +56,8 @@ class ModelDesc(C.Structure):
         ("yarn_factor", C.c_float), ("yarn_beta_fast", C.c_float), ("yarn_beta_slow", C.c_float), ("yarn_orig_max_pos", C.c_float),
         ("n_experts", C.c_int32), ("top_k", C.c_int32), ("swiglu_limit", C.c_float), ("ep_size", C.c_int32), ("ep_rank", C.c_int32),
         ("kv_page_rows", C.c_int32), ("kv_pool_pages", C.c_int32),
+        ("block_kind", C.c_int32), ("norm_kind", C.c_int32), ("pos_kind", C.c_int32), ("dist_bias", C.c_int32),
+        ("residual_mult", C.c_float), ("logit_scale", C.c_float),
     ]
 
     def copy(self, **kw) -> "ModelDesc":
@@ -63,6 +66,13 @@ class ModelDesc(C.Structure):
         for k, v in kw.items():
             setattr(d, k, v)
         return d
+
+
+class LayerDesc(C.Structure):
+    """Mirror of ``lum_layer_desc`` (include/lum_b200.h): one layer of a model whose layers are described one by one."""
+
+    _fields_ = [("n_q_heads", C.c_int32), ("n_kv_heads", C.c_int32), ("qk_dim", C.c_int32), ("v_dim", C.c_int32),
+                ("window", C.c_int32), ("v_mix", C.c_int32), ("ffn", C.c_int32), ("scale", C.c_float)]
 
 
 class Stats(C.Structure):
@@ -188,6 +198,9 @@ def load_library() -> C.CDLL:
         "lum_last_error": (C.c_char_p, [vp]),
         "lum_device_info": (i32, [vp, P(i32), P(u64), P(i32)]),
         "lum_model_init": (i32, [vp, P(ModelDesc)]),
+        "lum_model_init_layers": (i32, [vp, P(ModelDesc), P(LayerDesc)]),
+        "lum_want_logits": (i32, [vp, P(i32), i32]),
+        "lum_get_wanted": (i32, [vp, P(C.c_float), sz]),
         "lum_model_set_weight": (i32, [vp, i32, i32, vp, sz, u32]),
         "lum_model_set_weight_shard": (i32, [vp, i32, i32, vp, sz, u32]),
         "lum_load_safetensors": (i32, [vp, C.c_char_p, P(i32), P(i32)]),
@@ -375,6 +388,8 @@ class B200Runtime:
         self._h = C.c_void_p(handle)
         self._lib = lib
         self.desc: Optional[ModelDesc] = None
+        self.layers: Optional[List[LayerDesc]] = None      # models whose layers are described one by one
+        self._n_want = 0
 
     # ---- lifecycle -------------------------------------------------------------------------------
     @classmethod
@@ -456,9 +471,28 @@ class B200Runtime:
         return {"sm_count": sm.value, "mem_bytes": mem.value, "cc": cc.value}
 
     # ---- model -----------------------------------------------------------------------------------
-    def load_model(self, desc: ModelDesc) -> None:
-        self._ck(self._lib.lum_model_init(self._h, C.byref(desc)))
+    def load_model(self, desc: ModelDesc, layers: Optional[Sequence[LayerDesc]] = None) -> None:
+        """``layers``: one descriptor per layer for models with ``block_kind`` 1 (see ``models.from_config``)."""
+        if layers is None:
+            self._ck(self._lib.lum_model_init(self._h, C.byref(desc)))
+        else:
+            if len(layers) != desc.n_layers:
+                raise ValueError(f"{len(layers)} layer descriptors for {desc.n_layers} layers")
+            self._ck(self._lib.lum_model_init_layers(self._h, C.byref(desc), (LayerDesc * len(layers))(*layers)))
         self.desc = desc.copy()
+        self.layers = None if layers is None else list(layers)
+
+    def load_pretrained(self, folder: str, **kw):
+        """A folder with config.json and model.safetensors: the model class is chosen by the configuration (``models.REGISTRY``);
+        keywords as ``models.from_config``.  Returns the ``ModelSpec``."""
+        from . import models
+        spec = models.from_config(os.path.join(folder, "config.json"), **kw)
+        self.load_model(spec.desc, spec.layers)
+        loaded, _ = self.load_safetensors(os.path.join(folder, "model.safetensors"))
+        want = len(spec.tensor_names())
+        if loaded != want:
+            raise LumError(-1, f"{folder}: model.safetensors has {loaded} of the {want} tensors this model needs")
+        return spec
 
     def load_llir(self, blob: bytes, max_seq: int = 4096, kv_dtype: str = "bf16", max_new_tokens: int = 4096) -> None:
         """``Runtime::load_llir`` (src/op.rs:16): recognise the decoder a serialised graph describes and set it up."""
@@ -471,6 +505,7 @@ class B200Runtime:
             self.desc = None
             return
         self._ck(self._lib.lum_load_llir(self._h, buf, len(blob), max_seq, DTYPE[kv_dtype], max_new_tokens))
+        self.layers = None
         self.desc = d.copy(max_seq=max_seq, kv_dtype=DTYPE[kv_dtype], max_new_tokens=max_new_tokens)
         self.token_input, self.pos_input, self.logits_output = tok, pos, out
 
@@ -500,12 +535,19 @@ class B200Runtime:
         self._ck(self._lib.lum_profile_llir(self._h, buf, len(blob), int(dm.get("s", 1)), int(dm.get("p", 0)), trials, C.byref(us), text, 160))
         return us.value, text.value.decode()
 
+    def _kv_row_elems(self, layer: int, kind: str) -> int:
+        d = self.desc
+        if self.layers is None:
+            return (d.n_kv_heads // max(1, d.tp_size)) * d.head_dim
+        g = self.layers[layer]
+        return g.n_kv_heads * (-(-(g.qk_dim if kind == "k" else g.v_dim) // 16) * 16)     # heads padded to multiples of 16
+
     def kv_save(self, layer: int, kind: str, rows: int):
         """Rows [0, rows) of one layer's K or V cache as raw bytes in the cache's own element type."""
         import numpy as np
         d = self.desc
         esz = 2 if d.kv_dtype == DTYPE["bf16"] else 4
-        out = np.empty(rows * (d.n_kv_heads // max(1, d.tp_size)) * d.head_dim * esz, dtype=np.uint8)
+        out = np.empty(rows * self._kv_row_elems(layer, kind) * esz, dtype=np.uint8)
         self._ck(self._lib.lum_kv_save(self._h, layer, 0 if kind == "k" else 1, rows, out.ctypes.data_as(C.c_void_p), out.nbytes))
         return out
 
@@ -581,8 +623,7 @@ class B200Runtime:
 
     def kv_read(self, layer: int, kind: str, rows: int):
         import numpy as np
-        d = self.desc
-        out = np.empty((rows, (d.n_kv_heads // max(1, d.tp_size)) * d.head_dim), dtype=np.float32)
+        out = np.empty((rows, self._kv_row_elems(layer, kind)), dtype=np.float32)
         self._ck(self._lib.lum_kv_read(self._h, layer, 0 if kind == "k" else 1, rows, out.ctypes.data_as(C.POINTER(C.c_float))))
         return out
 
@@ -605,6 +646,19 @@ class B200Runtime:
         n = self.desc.vocab // max(1, self.desc.tp_size)
         out = np.empty(n, dtype=np.float32)
         self._ck(self._lib.lum_get_logits(self._h, out.ctypes.data_as(C.POINTER(C.c_float)), n))
+        return out
+
+    def want_logits(self, rows: Sequence[int]) -> None:
+        """The next ``execute`` keeps the logits of these rows of its tokens (increasing); read them with ``get_wanted``."""
+        rows = [int(r) for r in rows]
+        self._ck(self._lib.lum_want_logits(self._h, (C.c_int32 * max(1, len(rows)))(*rows), len(rows)))
+        self._n_want = len(rows)
+
+    def get_wanted(self):
+        """Logits ``[rows, vocab]`` the last ``execute`` kept."""
+        import numpy as np
+        out = np.empty((self._n_want, self.desc.vocab), dtype=np.float32)
+        self._ck(self._lib.lum_get_wanted(self._h, out.ctypes.data_as(C.POINTER(C.c_float)), out.size))
         return out
 
     def get_token(self) -> int:
