@@ -645,6 +645,96 @@ def run_tensor_core_regime(args, pkg, which: str):
     print(json.dumps(line))
 
 
+# Layers of real models' sizes for the Madipel design: hidden size, query and K/V heads, head size, inner width, window.
+# The closest existing model — the Llama family, Q8_0 — has three feed-forward matrices where this design has two: at 2/3 of the inner
+# width it holds as many weights.
+MADIPEL_SIZES = {
+    "4096x32": dict(width=4096, heads=32, kv=8, dim=128, ff=21504, window=4096),
+    "4096x32w1024": dict(width=4096, heads=32, kv=8, dim=128, ff=21504, window=1024),
+    "2560x32w1024": dict(width=2560, heads=32, kv=8, dim=128, ff=14592, window=1024),
+    "2048x16w512": dict(width=2048, heads=16, kv=4, dim=128, ff=12288, window=512),
+}
+
+
+def madipel_spec(pkg, size: dict, n_layers: int, vocab: int, max_seq: int):
+    mixer = {"heads": size["heads"], "kv_heads": size["kv"], "dim": size["dim"], "vdim": size["dim"], "scale": size["dim"] ** -0.5, "v_mix": True,
+             "mask": {"size": size["window"]}}
+    cfg = {"architecture": "Madipel", "layers": [{"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": size["ff"]}}] * n_layers,
+           "width": size["width"], "vocab": vocab, "residual_mult": 0.5, "logit_scale": 1.0, "norm": {"eps": 1e-5}}
+    return pkg.models.from_config(cfg, dtype="bfloat16", max_seq=max_seq)
+
+
+def run_madipel(args, pkg):
+    """Prompt and decode throughput of the Madipel design (bf16) beside the Llama family (Q8_0) at equal sizes: a cut of `--layers` layers
+    with a vocabulary of 32768, one prompt of `--prompt-len` tokens as rows, then `--steps` x `--tokens-per-step` decoded tokens.  Timed
+    with CUDA events on the runtime's stream; weights are larger than L2."""
+    import torch
+    torch.cuda.set_device(0)
+    peaks, peak_kind = measured_peaks()
+    tf_peak = peaks.get("bf16_tflops_sustained", 1383.9)
+    n, vocab, L, sizes = PROMPT_LEN, 32768, args.layers, []
+    new = args.steps * TOKENS_PER_STEP
+    total_launches = 0
+    sampler = ClockSampler(physical_gpu_index(0))
+    sampler.start()
+    for name in (args.size.split(",") if args.size else MADIPEL_SIZES):
+        z, row = MADIPEL_SIZES[name], {"size": name, **MADIPEL_SIZES[name]}
+        max_seq = (n + (args.warmup + args.steps + 1) * TOKENS_PER_STEP + 63) // 64 * 64
+        for arm in args.arms.split(","):
+            rt = pkg.B200Runtime.initialize(device=0)
+            if arm == "madipel":
+                spec = madipel_spec(pkg, z, L, vocab, max_seq)
+                rt.load_model(spec.desc, spec.layers)
+                w_layers, ff_mats, wb, window = spec.weight_elems_per_token() - vocab * z["width"], 2, 2.0, z["window"]
+            else:
+                desc = pkg.CONFIGS["llama3_8b_q8"].copy(n_layers=L, hidden=z["width"], n_q_heads=z["heads"], n_kv_heads=z["kv"], head_dim=z["dim"],
+                                                        ffn=z["ff"] * 2 // 3, vocab=vocab, max_seq=max_seq)
+                rt.load_model(desc)
+                w_layers = L * z["width"] * (2 * z["heads"] * z["dim"] + 2 * z["kv"] * z["dim"] + 3 * (z["ff"] * 2 // 3))
+                wb, window = 34.0 / 32.0, max_seq
+            rt.synth(SEED)
+            ids = _prompt_tokens(vocab, n)
+            ext = torch.cuda.ExternalStream(rt.stream())
+
+            def timed(fn, reps, warm):
+                for _ in range(warm):
+                    fn()
+                e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                rt.synchronize(); e0.record(ext)
+                for _ in range(reps):
+                    fn()
+                e1.record(ext); rt.synchronize()
+                return e0.elapsed_time(e1) / reps
+
+            def prompt():
+                rt.set_data(ids); rt.execute({"s": n, "p": 0})
+
+            def decode():
+                rt.decode_greedy(TOKENS_PER_STEP)
+
+            ms_p = timed(prompt, args.steps, args.warmup)
+            prompt()
+            ms_d = timed(decode, args.steps, args.warmup) / TOKENS_PER_STEP
+            pairs = sum(min(i + 1, window) for i in range(n))
+            flops = 2.0 * w_layers * n + 2.0 * vocab * z["width"] + L * 4.0 * z["heads"] * z["dim"] * pairs
+            ctx = min(n + (args.warmup + args.steps / 2.0) * TOKENS_PER_STEP, window)
+            bytes_tok = (w_layers + vocab * z["width"]) * wb + L * 2 * 2.0 * z["kv"] * z["dim"] * ctx
+            row[arm] = {"prompt_tokens_per_s": n / ms_p * 1e3, "prompt_ms": ms_p, "prompt_tflops": flops / ms_p / 1e9, "prompt_frac": flops / ms_p / 1e9 / tf_peak,
+                        "decode_tokens_per_s": 1e3 / ms_d, "decode_us": ms_d * 1e3, "decode_gbs": bytes_tok / ms_d / 1e6,
+                        "decode_frac": bytes_tok / ms_d / 1e6 / peaks["hbm_gbs"], "launches_per_step": rt.launches_per_step()}
+            total_launches += int(rt.stats().kernel_launches)
+            rt.close()
+        sizes.append(row)
+    clocks = sampler.stop()
+    first = sizes[0].get("madipel") or sizes[0].get("llama_q8")
+    print(json.dumps({"metric": "madipel_bf16_decode_tokens_per_s", "value": first["decode_tokens_per_s"], "unit": UNIT, "n_gpus": 1, "steps": args.steps,
+                      "warmup": args.warmup, "ms_per_step": first["decode_us"] * TOKENS_PER_STEP / 1e3, "higher_is_better": True, "scaling": "strong",
+                      "vs_baseline": None, "dtype": "bf16 x bf16 -> f32 (madipel), Q8_0 (llama_q8)", "data": "synthetic",
+                      "config": {"workload": "madipel", "layers": L, "vocab": vocab, "prompt_len": n, "tokens_per_step": TOKENS_PER_STEP, "seed": SEED,
+                                 "peak": f"of {peak_kind}: {peaks['hbm_gbs']:.1f} GB/s copy, {tf_peak:.1f} TFLOP/s sustained bf16", "l2": "weights >> 126 MB L2"},
+                      "sizes": sizes, "gpu_launches": total_launches, "clocks": clocks}))
+
+
 def _prefill_parity(pkg, base, ids, rows_token, rows_logits):
     """Against the oracle's committed fixture for this very prompt (tests/golden/llama3_8b_q8_prefill4096_full.npz: whole model, 4096
     rows, the logits after the last prompt token and the greedy sample) when it is there; otherwise the prompt once more, one
@@ -845,9 +935,13 @@ def main():
     ap.add_argument("--report", default=None, help="also write the byte / flop counts of the timed step as a metrics JSON in the reference bench crate's format")
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN, help="prompt tokens before the timed decode (profiling runs use a short one)")
     ap.add_argument("--tokens-per-step", type=int, default=TOKENS_PER_STEP)
-    ap.add_argument("--workload", default=WORKLOAD, choices=["llama3_8b_q8", "qwen3_4b_q8", "llama3_8b_q8_bs32", "llama3_8b_q8_prefill4096", "gpt_oss_20b_q8"],
+    ap.add_argument("--workload", default=WORKLOAD, choices=["llama3_8b_q8", "qwen3_4b_q8", "llama3_8b_q8_bs32", "llama3_8b_q8_prefill4096", "gpt_oss_20b_q8", "madipel"],
                     help="llama3_8b_q8: the configuration the metric is quoted on (default); qwen3_4b_q8: the Qwen3-4B shape; "
-                         "llama3_8b_q8_bs32 / llama3_8b_q8_prefill4096: the same model in the tensor-core regime (batched decode / one long prompt)")
+                         "llama3_8b_q8_bs32 / llama3_8b_q8_prefill4096: the same model in the tensor-core regime (batched decode / one long prompt); "
+                         "madipel: prompt and decode throughput of the Madipel design beside the Llama family at equal sizes")
+    ap.add_argument("--size", default=None, help="madipel: comma-separated sizes (default: all)")
+    ap.add_argument("--layers", type=int, default=8, help="madipel: layers of the cut")
+    ap.add_argument("--arms", default="madipel,llama_q8", help="madipel: which models to time")
     ap.add_argument("--only", default="all", choices=["all", "kernel", "sweep", "floor", "gemm", "gemm512", "gemm32", "prompt2", "sampler"],
                     help="kernel: time only the dominant kernel alone (small, for ncu captures); sweep: the kernel alone over a range of row counts; "
                          "floor: the decode step with all projections shrunk away; gemm: the tensor-core GEMM alone on the layer's shapes "
@@ -862,6 +956,14 @@ def main():
             print(json.dumps({"impl": "reference", "unavailable": "the CPU arm is timed on the batch-1 dense decode workloads only"}))
             return
         run_moe(args, pkg)
+        return
+    if args.workload == "madipel":
+        if args.impl == "reference":
+            print(json.dumps({"impl": "reference", "unavailable": "the reference has no such model"}))
+            return
+        if args.prompt_len == 512:
+            PROMPT_LEN = 4096
+        run_madipel(args, pkg)
         return
     if args.workload in ("llama3_8b_q8_bs32", "llama3_8b_q8_prefill4096"):
         if args.impl == "reference":

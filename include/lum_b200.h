@@ -130,7 +130,7 @@ typedef struct lum_model_desc {
     /* Decoders whose layers are described one by one (lum_model_init_layers); all zero for the families above.
      * block_kind 1: parallel sublayers — h = norm(x), x += residual_mult * (mixer(h) + ff(h)), one norm per layer.  The other fields
      * choose the mechanisms: norm_kind 0 RMS norm, 1 layer norm with bias (rms_eps is its eps, used as given); pos_kind 0 none, 1 a
-     * sinusoidal vector added to the embedding (entry 2i: sin(p * 10000^(-2i / hidden)), 2i + 1: cos); qk_norm 2: RMS norm of q and k
+     * sinusoidal vector added to the embedding (sine / cosine pairs, pair i at frequency 10000^(-2i / hidden)); qk_norm 2: RMS norm of q and k
      * over the whole projection (0: none); dist_bias 1: the score is multiplied by TEMP[h] and DIST_R1[h] * ln(1 + DIST_R2[h] * distance)
      * is taken off; logits are multiplied by logit_scale.  weight_dtype is LUM_BF16 or LUM_F32 (dense, no quantisation), linear layers
      * have no biases, one GPU.  With LUM_F32 everything is computed in 32 bits; with LUM_BF16 matrix operands are bf16 (accumulated

@@ -16,7 +16,7 @@ def layer_norm(x, gain, bias, eps):
 
 
 def sinusoid(positions, width, dtype=np.float64):
-    """Entry 2i is sin(p * 10000^(-2i / width)), entry 2i + 1 the cosine of the same angle."""
+    """Pairs of (sine, cosine) of position * frequency, the frequencies falling geometrically from 1 towards 1 / 10000."""
     e = np.arange(width)
     ang = np.asarray(positions, dtype)[:, None] * np.power(10000.0, -(2.0 * (e // 2)) / width).astype(dtype)
     return np.where(e % 2 == 0, np.sin(ang), np.cos(ang))
