@@ -144,12 +144,7 @@ __global__ void __launch_bounds__(256) embed_row(const EmbedArgs a) {
         if (threadIdx.x == 0 && blockIdx.x == 0) atomicOr(a.status, LUM_ST_BAD_TOKEN);
         return;
     }
-    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < a.H; i += gridDim.x * blockDim.x) {
-        const size_t o = (size_t)tok * a.H + i;
-        float v = a.kind == WK_BF16 ? bf16_bits_to_f32(((const uint16_t*)a.table)[o]) : ((const float*)a.table)[o];
-        if (a.pos_freq) v += sinusoid_at(a.pos_freq, a.state->pos, i);
-        a.x[i] = v;
-    }
+    embed_row_into(a.table, a.kind, a.H, tok, a.pos_freq, a.state->pos, a.x, blockIdx.x * blockDim.x + threadIdx.x, gridDim.x * blockDim.x);
 }
 
 cudaError_t launch_embed(const EmbedArgs& a_in, cudaStream_t st) {

@@ -285,13 +285,30 @@ cudaError_t launch_attn_prompt_tc(const AttnRowsArgs& a, cudaStream_t st) {
 }
 
 // ---------------------------------------------------------------------------------------------------- band attention
-// The same tile scheme for layers with their own head sizes, a window, and a distance bias: key size dkp (a multiple of 16) and value
-// size dvp are run-time numbers, the query heads of a K/V head may be any number R <= 128 (128 / R query rows per tile), tiles of keys
-// start at the first key any row of the tile still sees.  Queries arrive scaled (score factor and temperature).  The output goes
+// The same tiles for layers with their own head sizes, a window, and a distance bias: key size dkp (a multiple of 16) and value
+// size dvp are run-time numbers, the query heads of a K/V head may be any number R <= 128 (QT = 128 / R query rows per CTA), tiles of keys
+// start at the first key any row of the CTA still sees.  Queries arrive scaled (score factor and temperature).  The output goes
 // straight to the operand of the next product.
+//
+// The tensor core works one tile ahead of the softmax: while tile t's scores are exponentiated, S(t + 1) is computed into the other
+// score buffer, and O_t of tile t - 1 — issued at the end of the previous turn — is added up only when the new weights are ready to
+// be stored.  The bias depends on the distance alone: r1 ln(1 + r2 d) is evaluated once per (head, distance) of a tile,
+// R (QT + 63) values instead of 128 x 64, into shared memory (up to 16 heads per K/V head).  Rows are consecutive positions of one
+// sequence.  Scores are kept in units of ln 2 (queries and bias carry the factor 1 / ln 2), so that a weight is one power of two.
 //
 // DVH: value dimensions a thread accumulates (half of the value size, rounded up to 16).
 namespace {
+constexpr float kLog2e = 1.4426950408889634f;
+__device__ __forceinline__ float ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+// x = hi + lo in bf16 with the high term cut off instead of rounded (no conversion instruction for it; |x - hi - lo| <= 2^-17 |x| all the same)
+__device__ __forceinline__ void split2_cut(float x0, float x1, uint32_t* hi, uint32_t* lo) {
+    const uint32_t b0 = __float_as_uint(x0), b1 = __float_as_uint(x1);
+    *hi = __byte_perm(b0, b1, 0x7632);
+    const __nv_bfloat162 l = __floats2bfloat162_rn(x0 - __uint_as_float(b0 & 0xffff0000u), x1 - __uint_as_float(b1 & 0xffff0000u));
+    *lo = *(const uint32_t*)&l;
+}
+constexpr int kBtTabMaxR = 16;                      // R (128 / R + 63) <= 1136 floats up to there
+constexpr int kBtMiscBytes = 2048 + 4608;           // barriers, row exchange, flags; the bias table
 struct BandSmem { int qlo, k, v, phi, plo, misc, total; };      // byte offsets; the high Q term is at 0
 __host__ __device__ inline BandSmem band_smem(int dkp, int dvp) {
     BandSmem s;
@@ -301,7 +318,7 @@ __host__ __device__ inline BandSmem band_smem(int dkp, int dvp) {
     s.phi = s.v + 2 * kAtKT * dvp * 2;
     s.plo = s.phi + kAtPBytes;
     s.misc = s.plo + kAtPBytes;
-    s.total = s.misc + kAtMiscBytes;
+    s.total = s.misc + kBtMiscBytes;
     return s;
 }
 }  // namespace
@@ -319,7 +336,9 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_band_tc(const BandArgs a) 
     const uint32_t bar_s = s_base + L.misc, bar_o = bar_s + 8, tmem_slot = bar_s + 16;
     float* x_max = (float*)(smem + L.misc + 64);
     int* s_flag = (int*)(smem + L.misc + 64 + 1024);          // [0] largest, [2] smallest position of the CTA's rows, [1] a wait ran out
-    constexpr uint32_t kCols = DVH > 96 ? 512u : DVH > 32 ? 256u : 128u;      // S in columns 0..63, O_t from 64 on (2 DVH columns)
+    float* tab = (float*)(smem + L.misc + 2048);
+    constexpr uint32_t kCols = DVH > 64 ? 512u : 256u;        // S: columns 0..63 and 64..127 in turn, O_t from 128 on (2 DVH columns)
+    constexpr uint32_t kOCol = 128;
 
     if (tid == 0) { mbar_init(bar_s, 1); mbar_init(bar_o, 1); mbar_fence_init(); s_flag[0] = -1; s_flag[1] = 0; s_flag[2] = 0x7fffffff; }
     if (warp == 0) tmem_alloc(tmem_slot, kCols);
@@ -329,7 +348,7 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_band_tc(const BandArgs a) 
     const uint32_t tmem = *(volatile uint32_t*)(smem + L.misc + 16);
 
     const int row = (warp & 3) * 32 + lane, half = warp >> 2;
-    const int g_row = row / QT, m_row = q0 + (row - g_row * QT);
+    const int g_row = row / QT, qi_row = row - g_row * QT, m_row = q0 + qi_row;
     const bool row_ok = g_row < R && m_row < a.M;
     int pos_row = row_ok ? a.row_pos[m_row] : -1;
     if (pos_row >= a.max_seq) pos_row = -1;                    // flagged by the kernel that appended the row
@@ -339,9 +358,6 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_band_tc(const BandArgs a) 
         for (int o = 16; o > 0; o >>= 1) { pm = max(pm, __shfl_xor_sync(0xffffffffu, pm, o)); pn = min(pn, __shfl_xor_sync(0xffffffffu, pn, o)); }
         if (lane == 0 && pm >= 0) { atomicMax(&s_flag[0], pm); atomicMin(&s_flag[2], pn); }
     }
-    const int head = kvh * R + (row_ok ? g_row : 0);
-    const float r1 = a.r1 ? a.r1[head] : 0.0f, r2 = a.r1 ? a.r2[head] : 0.0f;
-    const bool biased = a.r1 != nullptr;
 
     // ---- Q tile -> two bf16 operands in shared memory
     for (int ch = tid; ch < 128 * kgr; ch += kAtThreads) {
@@ -350,8 +366,8 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_band_tc(const BandArgs a) 
         if (g < R && m < a.M) {
             const float4* src = (const float4*)(a.q + ((size_t)m * p.n_q + (size_t)kvh * R + g) * dkp + c * 8);
             const float4 v0 = src[0], v1 = src[1];
-            split2(v0.x, v0.y, &hi.x, &lo.x); split2(v0.z, v0.w, &hi.y, &lo.y);
-            split2(v1.x, v1.y, &hi.z, &lo.z); split2(v1.z, v1.w, &hi.w, &lo.w);
+            split2_cut(v0.x * kLog2e, v0.y * kLog2e, &hi.x, &lo.x); split2_cut(v0.z * kLog2e, v0.w * kLog2e, &hi.y, &lo.y);
+            split2_cut(v1.x * kLog2e, v1.y * kLog2e, &hi.z, &lo.z); split2_cut(v1.z * kLog2e, v1.w * kLog2e, &hi.w, &lo.w);
         }
         *(uint4*)(smem + c * 2048 + r * 16) = hi;
         *(uint4*)(smem + L.qlo + c * 2048 + r * 16) = lo;
@@ -359,137 +375,169 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_band_tc(const BandArgs a) 
     __syncthreads();
     const int pos_max = s_flag[0], pos_min = s_flag[2];
     const int first = pos_max < 0 ? 0 : (a.window > 0 && pos_min + 1 > a.window) ? pos_min + 1 - a.window : 0;     // no row sees an earlier key
-    const int t_lo = first / kAtKT, t_hi = pos_max >= 0 ? pos_max / kAtKT + 1 : t_lo;
+    const int t_lo = first / kAtKT, n_t = pos_max >= 0 ? pos_max / kAtKT + 1 - t_lo : 0;
     const int reach = a.window > 0 ? a.window : 0x7fffffff;    // this row sees distances 0 .. reach - 1
+    const bool biased = a.r1 != nullptr, use_tab = biased && R <= kBtTabMaxR;
+    const int TW = QT + kAtKT - 1, head = kvh * R + (row_ok ? g_row : 0);
+    const float* my_tab = tab + (g_row < R ? g_row : 0) * TW + qi_row + kAtKT - 1 - half * 32;      // [-i]: key i of this thread's half tile
 
     const size_t k_row = (size_t)p.n_kv * dkp, v_row = (size_t)p.n_kv * dvp;
     const __nv_bfloat16* kc = (const __nv_bfloat16*)a.k_cache + (size_t)kvh * dkp;
     const __nv_bfloat16* vc = (const __nv_bfloat16*)a.v_cache + (size_t)kvh * dvp;
-    // one operand tile: 64 positions x `gr` 16-byte groups; a warp takes 8 positions x 4 groups at a time
-    auto load_part = [&](int t, size_t tile_row, uint32_t dst, const __nv_bfloat16* src, size_t row_elems, int gr) {
-        const int gq = (gr + 3) / 4;
-        for (int w = warp; w < 8 * gq; w += kAtThreads / 32) {
-            const int kb = w / gq, key = kb * 8 + (lane >> 2), c = (w - kb * gq) * 4 + (lane & 3), j = t * kAtKT + key;
-            const bool in = j <= pos_max;                      // rows never written read as zeros
-            if (c < gr) cp_async16(dst + c * 1024 + key * 16, src + (tile_row + (size_t)(in ? key : 0)) * row_elems + c * 8, in ? 16u : 0u);
+    // one operand tile (i-th of this CTA): 64 positions x `gr` 16-byte groups; a warp takes 8 positions x 4 groups at a time.  One copy
+    // group per call, empty beyond the last tile.
+    auto load_tile = [&](int i, uint32_t dst, const __nv_bfloat16* src, size_t row_elems, int gr) {
+        if (i < n_t) {
+            const int t = t_lo + i, gq = (gr + 3) / 4;
+            // the tile's 64 positions start on a multiple of 64: one sequence slot or one page (of at least 64 rows) holds them all
+            const size_t tile_row = kv_phys_row(a.pg, a.seq0, a.max_seq, t * kAtKT);
+            for (int w = warp; w < 8 * gq; w += kAtThreads / 32) {
+                const int kb = w / gq, key = kb * 8 + (lane >> 2), c = (w - kb * gq) * 4 + (lane & 3), j = t * kAtKT + key;
+                const bool in = j <= pos_max;                  // rows never written read as zeros
+                if (c < gr) cp_async16(dst + c * 1024 + key * 16, src + (tile_row + (size_t)(in ? key : 0)) * row_elems + c * 8, in ? 16u : 0u);
+            }
         }
-    };
-    auto load_tile = [&](int t, int buf) {
-        // the tile's 64 positions start on a multiple of 64: one sequence slot or one page (of at least 64 rows) holds them all
-        const size_t tile_row = kv_phys_row(a.pg, a.seq0, a.max_seq, t * kAtKT);
-        load_part(t, tile_row, s_base + L.k + buf * kAtKT * dkp * 2, kc, k_row, kgr);
-        load_part(t, tile_row, s_base + L.v + buf * kAtKT * dvp * 2, vc, v_row, vgr);
         cp_async_commit();
+    };
+    auto load_k = [&](int i) { load_tile(i, s_base + L.k + (i & 1) * kAtKT * dkp * 2, kc, k_row, kgr); };
+    auto load_v = [&](int i) { load_tile(i, s_base + L.v + (i & 1) * kAtKT * dvp * 2, vc, v_row, vgr); };
+    const uint32_t idesc_s = idesc_bf16(128, kAtKT, false), idesc_o = idesc_bf16(128, dvp, true);
+    auto issue_s = [&](int i) {                                // thread 0: scores of tile i
+        const uint32_t kb = s_base + L.k + (i & 1) * kAtKT * dkp * 2, d = tmem + (i & 1) * kAtKT;
+        for (int term = 0; term < 2; term++) {
+            const uint32_t qb = s_base + (term ? L.qlo : 0);
+            for (int ks = 0; ks < dkp / 16; ks++)
+                umma_bf16(d, umma_smem_desc(qb + ks * 2 * 2048, 2048, 128), umma_smem_desc(kb + ks * 2 * 1024, 1024, 128), idesc_s, (term | ks) ? 1u : 0u);
+        }
+        umma_commit(bar_s);
     };
 
     float o_acc[DVH];
 #pragma unroll
     for (int i = 0; i < DVH; i++) o_acc[i] = 0.0f;
-    float m_run = -INFINITY, l_run = 0.0f;
-    const uint32_t idesc_s = idesc_bf16(128, kAtKT, false), idesc_o = idesc_bf16(128, dvp, true);
+    float m_run = -INFINITY, l_run = 0.0f, alpha_prev = 1.0f;
     const uint32_t lane_base = tmem + ((uint32_t)((warp & 3) * 32) << 16);
-
-    if (t_lo < t_hi) load_tile(t_lo, 0);
-    uint32_t phase = 0;
-    bool failed = false;
-#pragma unroll 1
-    for (int t = t_lo; t < t_hi; t++) {
-        const int buf = (t - t_lo) & 1;
-        if (t + 1 < t_hi) { load_tile(t + 1, buf ^ 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
-        fence_proxy_async_smem();
-        __syncthreads();
-        if (tid == 0) {
-            tc_fence_after_sync();
-            const uint32_t kb = s_base + L.k + buf * kAtKT * dkp * 2;
-            for (int term = 0; term < 2; term++) {
-                const uint32_t qb = s_base + (term ? L.qlo : 0);
-                for (int ks = 0; ks < dkp / 16; ks++)
-                    umma_bf16(tmem, umma_smem_desc(qb + ks * 2 * 2048, 2048, 128), umma_smem_desc(kb + ks * 2 * 1024, 1024, 128), idesc_s,
-                              (term | ks) ? 1u : 0u);
-            }
-            umma_commit(bar_s);
-        }
-        // distance corrections of this thread's 32 keys, while the tensor core computes the scores
-        const int j0 = t * kAtKT + half * 32;
-        float s[32];
-        if (biased) {
+    auto add_o = [&]() {                                       // o_acc = alpha o_acc + O_t, of the tile whose alpha is alpha_prev
 #pragma unroll
-            for (int i = 0; i < 32; i++) s[i] = r1 * logf(fmaf(r2, (float)max(pos_row - (j0 + i), 0), 1.0f));      // (masked keys: any finite value)
-        } else {
-#pragma unroll
-            for (int i = 0; i < 32; i++) s[i] = 0.0f;
-        }
-        if (!mbar_wait(bar_s, phase)) failed = true;
-        tc_fence_after_sync();
-
-        // ---- softmax of this thread's row over its 32 keys of the tile
-        {
-            uint32_t v0[16], v1[16];
-            tmem_ld16(lane_base + half * 32, v0);
-            tmem_ld16(lane_base + half * 32 + 16, v1);
+        for (int c = 0; c < DVH / 16; c++) {
+            uint32_t v[16];
+            tmem_ld16(lane_base + kOCol + half * DVH + c * 16, v);      // (columns beyond dvp: never written, never stored)
             tmem_ld_wait();
 #pragma unroll
-            for (int i = 0; i < 16; i++) { s[i] = __uint_as_float(v0[i]) - s[i]; s[16 + i] = __uint_as_float(v1[i]) - s[16 + i]; }
+            for (int i = 0; i < 16; i++) o_acc[c * 16 + i] = fmaf(o_acc[c * 16 + i], alpha_prev, __uint_as_float(v[i]));
+        }
+    };
+
+    bool failed = false;
+    int done = 0;                                              // tiles whose O_t was issued
+    if (n_t > 0) {
+        load_k(0); load_k(1); load_v(0);
+        cp_async_wait<2>();
+        fence_proxy_async_smem();
+        __syncthreads();
+        if (tid == 0) { tc_fence_after_sync(); issue_s(0); }
+    }
+#pragma unroll 1
+    for (int i = 0; i < n_t; i++) {
+        const uint32_t par = (uint32_t)(i & 1);
+        const int j0 = (t_lo + i) * kAtKT;
+        if (use_tab) {
+            const int d0 = pos_min - j0 - (kAtKT - 1);         // smallest distance in the tile: row 0, last key
+            for (int x = tid; x < R * TW; x += kAtThreads) {
+                const int g = x / TW;
+                tab[x] = a.r1[kvh * R + g] * kLog2e * logf(fmaf(a.r2[kvh * R + g], (float)max(d0 + x - g * TW, 0), 1.0f));
+            }
+        }
+        if (!mbar_wait(bar_s, par)) failed = true;             // S(i) is there, and K(i)'s buffer is free
+        load_k(i + 2);
+        cp_async_wait<2>();                                    // K(i + 1) has landed
+        fence_proxy_async_smem();
+        tc_fence_before_sync();
+        if (__syncthreads_or(failed ? 1 : 0)) { failed = true; break; }      // the tensor core never answered: give up, together
+        tc_fence_after_sync();
+        if (tid == 0 && i + 1 < n_t) issue_s(i + 1);
+
+        // ---- softmax of this thread's row over its 32 keys of the tile
+        float s[32];
+        {
+            uint32_t v0[16], v1[16];
+            tmem_ld16(lane_base + par * kAtKT + half * 32, v0);
+            tmem_ld16(lane_base + par * kAtKT + half * 32 + 16, v1);
+            tmem_ld_wait();
+#pragma unroll
+            for (int k = 0; k < 16; k++) { s[k] = __uint_as_float(v0[k]); s[16 + k] = __uint_as_float(v1[k]); }
+        }
+        const int dist0 = pos_row - (j0 + half * 32);          // distance of this thread's first key
+        if (use_tab) {
+#pragma unroll
+            for (int k = 0; k < 32; k++) s[k] -= my_tab[-k];
+        } else if (biased) {
+            const float r1 = a.r1[head] * kLog2e, r2 = a.r2[head];
+#pragma unroll
+            for (int k = 0; k < 32; k++) s[k] -= r1 * logf(fmaf(r2, (float)max(dist0 - k, 0), 1.0f));
         }
         float mx = -INFINITY;
+        if (__any_sync(0xffffffffu, dist0 < 31 || dist0 >= reach)) {       // some key of some row of the warp is out of sight
 #pragma unroll
-        for (int i = 0; i < 32; i++) {
-            const int d = pos_row - (j0 + i);
-            s[i] = (d >= 0 && d < reach) ? s[i] : -INFINITY;
-            mx = fmaxf(mx, s[i]);
+            for (int k = 0; k < 32; k++) s[k] = (dist0 - k >= 0 && dist0 - k < reach) ? s[k] : -INFINITY;
         }
+#pragma unroll
+        for (int k = 0; k < 32; k++) mx = fmaxf(mx, s[k]);
         x_max[half * 128 + row] = mx;
         named_sync(1, kAtThreads);
         const float m_new = fmaxf(m_run, fmaxf(mx, x_max[(half ^ 1) * 128 + row]));
-        const float alpha = (m_new == -INFINITY) ? 1.0f : expf(m_run - m_new);
+        const float alpha = (m_new == -INFINITY) ? 1.0f : ex2(m_run - m_new);
+        const float m_sub = (m_new == -INFINITY) ? 0.0f : m_new;           // nothing seen yet: 2^-inf = 0 below
         float psum = 0.0f;
         uint32_t ph[16], pl[16];
 #pragma unroll
-        for (int i = 0; i < 32; i += 2) {
-            const float p0 = (s[i] == -INFINITY) ? 0.0f : expf(s[i] - m_new);
-            const float p1 = (s[i + 1] == -INFINITY) ? 0.0f : expf(s[i + 1] - m_new);
+        for (int k = 0; k < 32; k += 2) {
+            const float p0 = ex2(s[k] - m_sub), p1 = ex2(s[k + 1] - m_sub);
             psum += p0 + p1;
-            split2(p0, p1, &ph[i >> 1], &pl[i >> 1]);
+            split2_cut(p0, p1, &ph[k >> 1], &pl[k >> 1]);
         }
         l_run = l_run * alpha + psum;
         m_run = m_new;
+
+        if (i > 0) {                                           // O_t of the tile before; P and V(i - 1) are free after that
+            if (!mbar_wait(bar_o, par ^ 1u)) failed = true;
+            tc_fence_after_sync();
+            add_o();
+        }
+        alpha_prev = alpha;
+        load_v(i + 1);
 #pragma unroll
         for (int c = 0; c < 4; c++) {
             const int off = (half * 4 + c) * 2048 + row * 16;
             *(uint4*)(smem + L.phi + off) = make_uint4(ph[c * 4], ph[c * 4 + 1], ph[c * 4 + 2], ph[c * 4 + 3]);
             *(uint4*)(smem + L.plo + off) = make_uint4(pl[c * 4], pl[c * 4 + 1], pl[c * 4 + 2], pl[c * 4 + 3]);
         }
+        cp_async_wait<2>();                                    // V(i) has landed
         fence_proxy_async_smem();
         tc_fence_before_sync();
         __syncthreads();
         if (tid == 0) {
             tc_fence_after_sync();
-            const uint32_t vb = s_base + L.v + buf * kAtKT * dvp * 2;
+            const uint32_t vb = s_base + L.v + (i & 1) * kAtKT * dvp * 2;
 #pragma unroll
             for (int term = 0; term < 2; term++) {
                 const uint32_t pb = s_base + (term ? L.plo : L.phi);
 #pragma unroll
                 for (int ks = 0; ks < kAtKT / 16; ks++)
-                    umma_bf16(tmem + 64, umma_smem_desc(pb + ks * 2 * 2048, 2048, 128), umma_smem_desc(vb + ks * 256, 128, 1024), idesc_o,
+                    umma_bf16(tmem + kOCol, umma_smem_desc(pb + ks * 2 * 2048, 2048, 128), umma_smem_desc(vb + ks * 256, 128, 1024), idesc_o,
                               (term | ks) ? 1u : 0u);
             }
             umma_commit(bar_o);
         }
-        if (!mbar_wait(bar_o, phase)) failed = true;
+        done = i + 1;
+    }
+    if (done > 0 && !failed) {
+        if (!mbar_wait(bar_o, (uint32_t)((done - 1) & 1))) failed = true;
         tc_fence_after_sync();
-#pragma unroll
-        for (int c = 0; c < DVH / 16; c++) {
-            uint32_t v[16];
-            tmem_ld16(lane_base + 64 + half * DVH + c * 16, v);      // (columns beyond dvp: never written, never stored)
-            tmem_ld_wait();
-#pragma unroll
-            for (int i = 0; i < 16; i++) o_acc[c * 16 + i] = fmaf(o_acc[c * 16 + i], alpha, __uint_as_float(v[i]));
-        }
-        tc_fence_before_sync();
-        phase ^= 1u;
-        if (__syncthreads_or(failed ? 1 : 0)) { if (tid == 0) s_flag[1] = 1; break; }
+        add_o();
     }
     cp_async_wait<0>();
+    if (failed) s_flag[1] = 1;
     __syncthreads();
     if (s_flag[1] && tid == 0 && a.status) atomicOr(a.status, LUM_ST_WAIT_TMEM);
 

@@ -8,6 +8,7 @@
 //                 cache.  FUSED: one row, with all of qkv_rows in the prologue (a decode step's attention is one kernel).
 // Everything here is computed in f32.  The tensor-core form for prompts is in lum_attn_tc.cu.
 #include <cuda_bf16.h>
+#include <cstdlib>
 
 #include "lum_gemv_dev.cuh"
 #include "lum_dense.cuh"
@@ -21,11 +22,25 @@ __global__ void __launch_bounds__(256) norm_rows(const NormRowsArgs a) {
     const int m = blockIdx.x, tid = threadIdx.x, W = a.norm.width;
     const float* x = a.x + (size_t)(a.row_index ? a.row_index[m] : m) * a.ldx;
     float s = 0.0f;
-    for (int i = tid; i < W; i += 256) { const float v = x[i]; nr_row[i] = v; s += v; }
+    const bool vec = (W & 3) == 0 && (a.ldx & 3) == 0;
+    if (vec) {
+#pragma unroll 4
+        for (int i = tid; i < W / 4; i += 256) { const float4 v = ((const float4*)x)[i]; ((float4*)nr_row)[i] = v; s += (v.x + v.y) + (v.z + v.w); }
+    } else {
+        for (int i = tid; i < W; i += 256) { const float v = x[i]; nr_row[i] = v; s += v; }
+    }
     float mean = 0.0f;
     if (a.norm.mode == NORM_LAYER) mean = block_sum(s, red, tid, 256, 1) / (float)W;
     s = 0.0f;
-    for (int i = tid; i < W; i += 256) { const float d = nr_row[i] - mean; s = fmaf(d, d, s); }
+    if (vec) {
+        for (int i = tid; i < W / 4; i += 256) {
+            const float4 v = ((const float4*)nr_row)[i];
+            const float d0 = v.x - mean, d1 = v.y - mean, d2 = v.z - mean, d3 = v.w - mean;
+            s = fmaf(d0, d0, s); s = fmaf(d1, d1, s); s = fmaf(d2, d2, s); s = fmaf(d3, d3, s);
+        }
+    } else {
+        for (int i = tid; i < W; i += 256) { const float d = nr_row[i] - mean; s = fmaf(d, d, s); }
+    }
     const float inv = 1.0f / sqrtf(block_sum(s, red, tid, 256, 1) / (float)W + a.norm.eps);
     auto value = [&](int k) -> float {
         if (k >= W) return 0.0f;
@@ -34,10 +49,23 @@ __global__ void __launch_bounds__(256) norm_rows(const NormRowsArgs a) {
     };
     if (a.kind == WK_BF16) {
         for (int g = tid; g < a.out.chunks * 8; g += 256) {
+            float f[8];
+            if (vec && g * 8 + 8 <= W) {
+#pragma unroll
+                for (int h = 0; h < 2; h++) {
+                    const float4 v = ((const float4*)nr_row)[g * 2 + h], gn = ((const float4*)a.norm.gain)[g * 2 + h];
+                    const float4 b = a.norm.bias ? ((const float4*)a.norm.bias)[g * 2 + h] : make_float4(0.f, 0.f, 0.f, 0.f);
+                    f[4 * h] = (v.x - mean) * inv * gn.x + b.x; f[4 * h + 1] = (v.y - mean) * inv * gn.y + b.y;
+                    f[4 * h + 2] = (v.z - mean) * inv * gn.z + b.z; f[4 * h + 3] = (v.w - mean) * inv * gn.w + b.w;
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < 8; i++) f[i] = value(g * 8 + i);
+            }
             uint32_t w[4];
 #pragma unroll
             for (int i = 0; i < 4; i++) {
-                const __nv_bfloat162 b = __floats2bfloat162_rn(value(g * 8 + 2 * i), value(g * 8 + 2 * i + 1));
+                const __nv_bfloat162 b = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
                 w[i] = *(const uint32_t*)&b;
             }
             *(uint4*)((unsigned char*)a.out.p + row_operand_off(WK_BF16, a.out.chunks, m, g * 8)) = make_uint4(w[0], w[1], w[2], w[3]);
@@ -64,6 +92,7 @@ cudaError_t launch_norm_rows(const NormRowsArgs& a, cudaStream_t st) {
 __device__ __forceinline__ float proj_inv_rms(const float* v, int n, const float* gain, float eps, float* red, int tid) {
     if (!gain) return 1.0f;
     float s = 0.0f;
+#pragma unroll 16
     for (int i = tid; i < n; i += 256) { const float t = v[i]; s = fmaf(t, t, s); }
     return 1.0f / sqrtf(block_sum(s, red, tid, 256, 1) / (float)n + eps);
 }
@@ -102,7 +131,22 @@ __global__ void __launch_bounds__(256) qkv_rows(const BandArgs a) {
     const float* row = p.qkv + (size_t)m * p.ld;
     const float *q = row + p.q_off, *k = row + p.k_off, *v = row + p.v_off;
     const float iq = proj_inv_rms(q, p.n_q * p.dk, p.q_gain, p.eps, red, tid), ik = proj_inv_rms(k, p.n_kv * p.dk, p.k_gain, p.eps, red, tid);
-    for (int i = tid; i < p.n_q * p.dkp; i += 256) a.q_out[(size_t)m * p.n_q * p.dkp + i] = prep_query(p, q, iq, i / p.dkp, i % p.dkp);
+    if (p.q_gain && (p.dk & 3) == 0 && ((p.ld | p.q_off) & 3) == 0) {      // four at a time (dkp is a multiple of 16)
+        const int n4 = p.dkp / 4;
+#pragma unroll 4
+        for (int i = tid; i < p.n_q * n4; i += 256) {
+            const int h = i / n4, e = (i - h * n4) * 4, src = (h * p.dk + e) / 4;
+            float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (e < p.dk) {
+                const float4 v = ((const float4*)q)[src], g = ((const float4*)p.q_gain)[src];
+                const float f = p.temp ? p.scale * p.temp[h] : p.scale;
+                o = make_float4(v.x * iq * g.x * f, v.y * iq * g.y * f, v.z * iq * g.z * f, v.w * iq * g.w * f);
+            }
+            ((float4*)(a.q_out + (size_t)m * p.n_q * p.dkp))[i] = o;
+        }
+    } else {
+        for (int i = tid; i < p.n_q * p.dkp; i += 256) a.q_out[(size_t)m * p.n_q * p.dkp + i] = prep_query(p, q, iq, i / p.dkp, i % p.dkp);
+    }
     const size_t prow = kv_phys_row(a.pg, seq, a.max_seq, pos);
     const size_t ko = prow * p.n_kv * p.dkp, vo = prow * p.n_kv * p.dvp;
     for (int i = tid; i < p.n_kv * p.dkp; i += 256) cache_store(a.k_cache, a.kv_bf16, ko + i, prep_key(p, k, ik, i / p.dkp, i % p.dkp));
@@ -121,9 +165,12 @@ cudaError_t launch_qkv_rows(const BandArgs& a, cudaStream_t st) {
 //   scores   4 lanes per key, each a share of the head dimension for all 8 queries; two shuffles; distance bias; shared memory
 //   softmax  one warp per query head: running maximum and sum
 //   values   thread = two value dimensions and a share of the keys
+// A tile's key and value loads are all issued before anything of the previous tile is waited for again: the next tile's keys are in
+// flight during this tile's softmax, its values during its scores.
 // The splits of a row are the CTAs of a thread-block cluster and fold their (maximum, sum, vector) through its shared memory.
 namespace {
 constexpr int kBdTK = 64, kBdR = 8, kBdMaxSplits = 16;
+constexpr int kBdKv = 4, kBdVv = 16;     // 16-byte key groups / value pairs of a tile a thread keeps in registers (longer heads: the rest is loaded where used)
 struct BdSmem {      // offsets in floats
     int q, sc, red, o, ml, wgt, knew, vnew, part, total;
 };
@@ -144,8 +191,14 @@ __host__ __device__ inline BdSmem bd_layout(int dkp, int dvp) {
 }
 }  // namespace
 
-template <bool BF16, bool FUSED>
-__global__ void __launch_bounds__(256) attn_band(const BandArgs a, int S, int HB) {
+template <bool BF16> struct BandPair { using type = uint32_t; };      // two values as they lie in the cache
+template <> struct BandPair<false> { using type = float2; };
+__device__ __forceinline__ float2 band_pair(uint32_t w) { return make_float2(__uint_as_float(w << 16), __uint_as_float(w & 0xffff0000u)); }
+__device__ __forceinline__ float2 band_pair(float2 v) { return v; }
+
+// RB: query heads the registers are laid out for (4 or 8)
+template <bool BF16, bool FUSED, int RB>
+__global__ void __launch_bounds__(256, 2) attn_band(const BandArgs a, int S, int HB) {
     extern __shared__ __align__(16) float bd[];
     const QkvArgs& p = a.p;
     const BdSmem L = bd_layout(p.dkp, p.dvp);
@@ -194,55 +247,82 @@ __global__ void __launch_bounds__(256) attn_band(const BandArgs a, int S, int HB
     const int lo = (a.window > 0 && pos + 1 > a.window) ? pos + 1 - a.window : 0;
     const int per = (pos + 1 - lo + S - 1) / S, k0 = lo + sp * per, k1 = min(pos + 1, k0 + per);
     const int npair = p.dvp / 2, nsub = npair >= 256 ? 1 : 256 / npair, sub = tid / npair, dv2 = tid - sub * npair;
-    float acc[kBdR][2];
+    float acc[RB][2];
 #pragma unroll
-    for (int r = 0; r < kBdR; r++) acc[r][0] = acc[r][1] = 0.0f;
+    for (int r = 0; r < RB; r++) acc[r][0] = acc[r][1] = 0.0f;
+
+    const int key = tid >> 2, part = tid & 3, kgr = p.dkp / (BF16 ? 8 : 4);
+    const size_t esz = BF16 ? 2 : 4;
+    // row `j` of this K/V head (the row of this very step: from shared memory, its store to the cache may still be on the way)
+    auto key_row = [&](int j) -> const char* {
+        if (FUSED && j == pos) return (const char*)(bd + L.knew);
+        return (const char*)a.k_cache + (kv_phys_row(a.pg, seq, FUSED ? 0 : a.max_seq, j) * k_row + (size_t)kvh * p.dkp) * esz;
+    };
+    using VRaw = typename BandPair<BF16>::type;
+    auto value_pair = [&](int j) -> VRaw {
+        const char* vr = (const char*)(bd + L.vnew);
+        if (!(FUSED && j == pos)) vr = (const char*)a.v_cache + (kv_phys_row(a.pg, seq, FUSED ? 0 : a.max_seq, j) * v_row + (size_t)kvh * p.dvp) * esz;
+        return *((const VRaw*)vr + dv2);
+    };
+    float d[RB];
+    auto dot_group = [&](const uint4& raw, int c) {
+        if (BF16) {
+            const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
+            float kf[8];
+#pragma unroll
+            for (int t = 0; t < 4; t++) { kf[2 * t] = __uint_as_float(w[t] << 16); kf[2 * t + 1] = __uint_as_float(w[t] & 0xffff0000u); }
+#pragma unroll
+            for (int r = 0; r < RB; r++) {
+                const float4 q0 = *(const float4*)(q_s + r * p.dkp + c * 8), q1 = *(const float4*)(q_s + r * p.dkp + c * 8 + 4);
+                d[r] = fmaf(q0.x, kf[0], d[r]); d[r] = fmaf(q0.y, kf[1], d[r]); d[r] = fmaf(q0.z, kf[2], d[r]); d[r] = fmaf(q0.w, kf[3], d[r]);
+                d[r] = fmaf(q1.x, kf[4], d[r]); d[r] = fmaf(q1.y, kf[5], d[r]); d[r] = fmaf(q1.z, kf[6], d[r]); d[r] = fmaf(q1.w, kf[7], d[r]);
+            }
+        } else {
+            const float kf[4] = {__uint_as_float(raw.x), __uint_as_float(raw.y), __uint_as_float(raw.z), __uint_as_float(raw.w)};
+#pragma unroll
+            for (int r = 0; r < RB; r++) {
+                const float4 q0 = *(const float4*)(q_s + r * p.dkp + c * 4);
+                d[r] = fmaf(q0.x, kf[0], d[r]); d[r] = fmaf(q0.y, kf[1], d[r]); d[r] = fmaf(q0.z, kf[2], d[r]); d[r] = fmaf(q0.w, kf[3], d[r]);
+            }
+        }
+    };
+    uint4 kreg[kBdKv];
+    auto load_keys = [&](int j0, int nk) {
+        if (key < nk) {
+            const uint4* kr = (const uint4*)key_row(j0 + key);
+#pragma unroll
+            for (int i = 0; i < kBdKv; i++) if (part + 4 * i < kgr) kreg[i] = kr[part + 4 * i];
+        }
+    };
     __syncthreads();
+    if (k0 < k1) load_keys(k0, min(kBdTK, k1 - k0));
 
     for (int j0 = k0; j0 < k1; j0 += kBdTK) {
         const int nk = min(kBdTK, k1 - j0);
+        VRaw vreg[kBdVv];
+        if (sub < nsub) {
+#pragma unroll
+            for (int i = 0; i < kBdVv; i++) if (sub + i * nsub < nk) vreg[i] = value_pair(j0 + sub + i * nsub);
+        }
         {   // scores
-            const int key = tid >> 2, part = tid & 3, j = j0 + key;
-            float d[kBdR];
+            const int j = j0 + key;
 #pragma unroll
-            for (int r = 0; r < kBdR; r++) d[r] = 0.0f;
+            for (int r = 0; r < RB; r++) d[r] = 0.0f;
             if (key < nk) {
-                const size_t ro = (kv_phys_row(a.pg, seq, FUSED ? 0 : a.max_seq, j) * k_row + (size_t)kvh * p.dkp);
-                const char* kr = (FUSED && j == pos) ? (const char*)(bd + L.knew) : (const char*)a.k_cache + ro * (BF16 ? 2 : 4);
-                if (BF16) {
-#pragma unroll 4
-                    for (int c = part; c < p.dkp / 8; c += 4) {
-                        const uint4 raw = *((const uint4*)kr + c);
-                        const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
-                        float kf[8];
 #pragma unroll
-                        for (int t = 0; t < 4; t++) { kf[2 * t] = __uint_as_float(w[t] << 16); kf[2 * t + 1] = __uint_as_float(w[t] & 0xffff0000u); }
-#pragma unroll
-                        for (int r = 0; r < kBdR; r++) {
-                            const float4 q0 = *(const float4*)(q_s + r * p.dkp + c * 8), q1 = *(const float4*)(q_s + r * p.dkp + c * 8 + 4);
-                            d[r] = fmaf(q0.x, kf[0], d[r]); d[r] = fmaf(q0.y, kf[1], d[r]); d[r] = fmaf(q0.z, kf[2], d[r]); d[r] = fmaf(q0.w, kf[3], d[r]);
-                            d[r] = fmaf(q1.x, kf[4], d[r]); d[r] = fmaf(q1.y, kf[5], d[r]); d[r] = fmaf(q1.z, kf[6], d[r]); d[r] = fmaf(q1.w, kf[7], d[r]);
-                        }
-                    }
-                } else {
-#pragma unroll 4
-                    for (int c = part; c < p.dkp / 4; c += 4) {
-                        const float4 kf = *((const float4*)kr + c);
-#pragma unroll
-                        for (int r = 0; r < kBdR; r++) {
-                            const float4 q0 = *(const float4*)(q_s + r * p.dkp + c * 4);
-                            d[r] = fmaf(q0.x, kf.x, d[r]); d[r] = fmaf(q0.y, kf.y, d[r]); d[r] = fmaf(q0.z, kf.z, d[r]); d[r] = fmaf(q0.w, kf.w, d[r]);
-                        }
-                    }
+                for (int i = 0; i < kBdKv; i++) if (part + 4 * i < kgr) dot_group(kreg[i], part + 4 * i);
+                if (kgr > 4 * kBdKv) {
+                    const uint4* kr = (const uint4*)key_row(j);
+                    for (int c = part + 4 * kBdKv; c < kgr; c += 4) dot_group(kr[c], c);
                 }
             }
 #pragma unroll
-            for (int r = 0; r < kBdR; r++) {
+            for (int r = 0; r < RB; r++) {
                 d[r] += __shfl_xor_sync(0xffffffffu, d[r], 1);
                 d[r] += __shfl_xor_sync(0xffffffffu, d[r], 2);
             }
 #pragma unroll
-            for (int r = 0; r < kBdR; r++) {
+            for (int r = 0; r < RB; r++) {
                 if ((r & 3) == part && r < nr) {
                     float s = d[r];
                     if (a.r1) s -= distance_bias(a.r1[head0 + r], a.r2[head0 + r], (float)(pos - j));
@@ -250,6 +330,7 @@ __global__ void __launch_bounds__(256) attn_band(const BandArgs a, int S, int HB
                 }
             }
         }
+        if (j0 + kBdTK < k1) load_keys(j0 + kBdTK, min(kBdTK, k1 - j0 - kBdTK));
         __syncthreads();
         if (warp < nr) {   // softmax bookkeeping of query head `warp`
             float* s = sc + warp * (kBdTK + 4);
@@ -267,26 +348,23 @@ __global__ void __launch_bounds__(256) attn_band(const BandArgs a, int S, int HB
         __syncthreads();
         if (sub < nsub) {
 #pragma unroll
-            for (int r = 0; r < kBdR; r++) if (r < nr) { const float c = c_s[r]; acc[r][0] *= c; acc[r][1] *= c; }
-            for (int t = sub; t < nk; t += nsub) {
-                const int j = j0 + t;
-                const size_t ro = kv_phys_row(a.pg, seq, FUSED ? 0 : a.max_seq, j) * v_row + (size_t)kvh * p.dvp;
-                const char* vr = (FUSED && j == pos) ? (const char*)(bd + L.vnew) : (const char*)a.v_cache + ro * (BF16 ? 2 : 4);
-                float v0, v1;
-                if (BF16) { const uint32_t w = *((const uint32_t*)vr + dv2); v0 = __uint_as_float(w << 16); v1 = __uint_as_float(w & 0xffff0000u); }
-                else { const float2 w = *((const float2*)vr + dv2); v0 = w.x; v1 = w.y; }
+            for (int r = 0; r < RB; r++) if (r < nr) { const float c = c_s[r]; acc[r][0] *= c; acc[r][1] *= c; }
+            auto take = [&](const VRaw& raw, int t) {
+                const float2 v = band_pair(raw);
 #pragma unroll
-                for (int r = 0; r < kBdR; r++) {
-                    if (r < nr) { const float w = sc[r * (kBdTK + 4) + t]; acc[r][0] = fmaf(w, v0, acc[r][0]); acc[r][1] = fmaf(w, v1, acc[r][1]); }
-                }
-            }
+                for (int r = 0; r < RB; r++)
+                    if (r < nr) { const float w = sc[r * (kBdTK + 4) + t]; acc[r][0] = fmaf(w, v.x, acc[r][0]); acc[r][1] = fmaf(w, v.y, acc[r][1]); }
+            };
+#pragma unroll
+            for (int i = 0; i < kBdVv; i++) if (sub + i * nsub < nk) take(vreg[i], sub + i * nsub);
+            for (int t = sub + kBdVv * nsub; t < nk; t += nsub) take(value_pair(j0 + t), t);
         }
         __syncthreads();
     }
     // ---- fold the key shares, then the splits
     if (sub < nsub)
 #pragma unroll
-        for (int r = 0; r < kBdR; r++)
+        for (int r = 0; r < RB; r++)
             if (r < nr) *(float2*)(bd + L.part + (sub * kBdR + r) * p.dvp + 2 * dv2) = make_float2(acc[r][0], acc[r][1]);
     __syncthreads();
     for (int i = tid; i < nr * p.dvp; i += 256) {
@@ -343,16 +421,23 @@ static cudaError_t launch_band(const BandArgs& a_in, int rows, bool fused, int s
     const int R = p.n_q / p.n_kv;
     int HB = (R + kBdR - 1) / kBdR;
     const size_t smem = (size_t)bd_layout(p.dkp, p.dvp).total * 4;
-    const void* fn = a.kv_bf16 ? (fused ? (const void*)attn_band<true, true> : (const void*)attn_band<true, false>)
-                               : (fused ? (const void*)attn_band<false, true> : (const void*)attn_band<false, false>);
+    static const void* const fns[2][2][2] = {
+        {{(const void*)attn_band<false, false, 4>, (const void*)attn_band<false, false, 8>}, {(const void*)attn_band<false, true, 4>, (const void*)attn_band<false, true, 8>}},
+        {{(const void*)attn_band<true, false, 4>, (const void*)attn_band<true, false, 8>}, {(const void*)attn_band<true, true, 4>, (const void*)attn_band<true, true, 8>}}};
+    const void* fn = fns[a.kv_bf16 ? 1 : 0][fused ? 1 : 0][R > 4 ? 1 : 0];
     if (smem > 48 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         if (e != cudaSuccess) return e;
     }
-    // splits: enough CTAs for the SMs, none shorter than a tile of keys at full window, within the portable cluster size
+    // splits: enough CTAs for the SMs, none shorter than half a tile of keys at full reach
     const int reach = a.window > 0 && a.window < a.max_seq ? a.window : a.max_seq;
+    static const int env_s = [] { const char* e = getenv("LUM_BAND_SPLITS"); return e ? atoi(e) : kBdMaxSplits; }();
     int S = 1;
-    while (S < 8 && (long long)p.n_kv * HB * rows * S * 2 <= sm_count && reach >= S * 2 * kBdTK / 2) S *= 2;
+    while (S < env_s && S < kBdMaxSplits && (long long)p.n_kv * HB * rows * S * 2 <= sm_count && reach >= S * 2 * kBdTK / 2) S *= 2;
+    if (S > 8) {      // beyond the portable cluster size
+        const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        if (e != cudaSuccess) return e;
+    }
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(S, p.n_kv * HB, rows); cfg.blockDim = dim3(256); cfg.dynamicSmemBytes = smem; cfg.stream = st;
     cudaLaunchAttribute at[2];

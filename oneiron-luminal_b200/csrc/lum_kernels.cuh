@@ -159,11 +159,20 @@ struct EmbedArgs {
     int use_pdl;
     const double* pos_freq;// optional [ceil(H / 2)]: sin (entry 2i) and cos (2i + 1) of position * pos_freq[i] are added
 };
-// the sinusoidal position vector's entry i (angles in f64: exact to f32 rounding at any position)
-__device__ __forceinline__ float sinusoid_at(const double* freq, int pos, int i) {
+// entries 2 i and 2 i + 1 of the sinusoidal position vector (angles in f64: exact to f32 rounding at any position)
+__device__ __forceinline__ float2 sinusoid_pair(const double* freq, int pos, int i) {
     double s, c;
-    sincos((double)pos * freq[i >> 1], &s, &c);
-    return (float)((i & 1) ? c : s);
+    sincos((double)pos * freq[i], &s, &c);
+    return make_float2((float)s, (float)c);
+}
+// one row of the embedding table as f32, plus the position vector when pos_freq is given; thread `t` of `n`
+__device__ __forceinline__ void embed_row_into(const void* table, int kind, int H, int tok, const double* pos_freq, int pos, float* x, int t, int n) {
+    for (int i = t; i < (H + 1) / 2; i += n) {
+        const size_t o = (size_t)tok * H + 2 * i;
+        const float2 add = pos_freq ? sinusoid_pair(pos_freq, pos, i) : make_float2(0.0f, 0.0f);
+        x[2 * i] = (kind == WK_BF16 ? bf16_bits_to_f32(((const uint16_t*)table)[o]) : ((const float*)table)[o]) + add.x;
+        if (2 * i + 1 < H) x[2 * i + 1] = (kind == WK_BF16 ? bf16_bits_to_f32(((const uint16_t*)table)[o + 1]) : ((const float*)table)[o + 1]) + add.y;
+    }
 }
 
 // message of the last failed stand-alone operator on this thread (read back through lum_last_error(NULL))

@@ -31,12 +31,7 @@ __global__ void __launch_bounds__(256) embed_rows(const void* table, int kind, i
         if (threadIdx.x == 0) atomicOr(status, LUM_ST_BAD_TOKEN);
         return;
     }
-    for (int i = threadIdx.x; i < H; i += 256) {
-        const size_t o = (size_t)tok * H + i;
-        float v = kind == WK_BF16 ? bf16_bits_to_f32(((const uint16_t*)table)[o]) : ((const float*)table)[o];
-        if (pos_freq) v += sinusoid_at(pos_freq, row_pos[m], i);
-        x[(size_t)m * ldx + i] = v;
-    }
+    embed_row_into(table, kind, H, tok, pos_freq, pos_freq ? row_pos[m] : 0, x + (size_t)m * ldx, threadIdx.x, 256);
 }
 
 // ---------------------------------------------------------------------------------------------------- RoPE + cache append
