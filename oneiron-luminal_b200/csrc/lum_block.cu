@@ -178,7 +178,7 @@ __host__ __device__ inline BdSmem bd_layout(int dkp, int dvp) {
     BdSmem s;
     s.q = 0;
     s.sc = s.q + kBdR * dkp;
-    s.red = s.sc + kBdR * (kBdTK + 4);
+    s.red = s.sc + kBdR * kBdTK;                         // scores / weights [key][8]
     s.ml = s.red + 32;                                   // maximum [8], sum [8], correction [8]
     s.wgt = s.ml + 32;                                   // [splits][8]
     s.o = s.wgt + kBdMaxSplits * kBdR;
@@ -326,15 +326,15 @@ __global__ void __launch_bounds__(256, 2) attn_band(const BandArgs a, int S, int
                 if ((r & 3) == part && r < nr) {
                     float s = d[r];
                     if (a.r1) s -= distance_bias(a.r1[head0 + r], a.r2[head0 + r], (float)(pos - j));
-                    sc[r * (kBdTK + 4) + key] = key < nk ? s : -INFINITY;
+                    sc[key * kBdR + r] = key < nk ? s : -INFINITY;
                 }
             }
         }
         if (j0 + kBdTK < k1) load_keys(j0 + kBdTK, min(kBdTK, k1 - j0 - kBdTK));
         __syncthreads();
         if (warp < nr) {   // softmax bookkeeping of query head `warp`
-            float* s = sc + warp * (kBdTK + 4);
-            const float s0 = s[lane], s1 = s[lane + 32];
+            float* s = sc + warp;
+            const float s0 = s[lane * kBdR], s1 = s[(lane + 32) * kBdR];
             float mx = fmaxf(s0, s1);
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -342,7 +342,7 @@ __global__ void __launch_bounds__(256, 2) attn_band(const BandArgs a, int S, int
             const float p0 = expf(s0 - mn), p1 = expf(s1 - mn);      // exp(-inf) = 0 beyond the last key
             const float ps = warp_sum(p0 + p1);
             __syncwarp();
-            s[lane] = p0; s[lane + 32] = p1;
+            s[lane * kBdR] = p0; s[(lane + 32) * kBdR] = p1;
             if (lane == 0) { const float c = mo == -INFINITY ? 0.0f : expf(mo - mn); m_s[warp] = mn; l_s[warp] = l_s[warp] * c + ps; c_s[warp] = c; }
         }
         __syncthreads();
@@ -351,9 +351,11 @@ __global__ void __launch_bounds__(256, 2) attn_band(const BandArgs a, int S, int
             for (int r = 0; r < RB; r++) if (r < nr) { const float c = c_s[r]; acc[r][0] *= c; acc[r][1] *= c; }
             auto take = [&](const VRaw& raw, int t) {
                 const float2 v = band_pair(raw);
+                float w[RB];                                       // (heads beyond nr: whatever is there, never read back)
 #pragma unroll
-                for (int r = 0; r < RB; r++)
-                    if (r < nr) { const float w = sc[r * (kBdTK + 4) + t]; acc[r][0] = fmaf(w, v.x, acc[r][0]); acc[r][1] = fmaf(w, v.y, acc[r][1]); }
+                for (int r = 0; r < RB; r += 4) *(float4*)&w[r] = *(const float4*)(sc + t * kBdR + r);
+#pragma unroll
+                for (int r = 0; r < RB; r++) { acc[r][0] = fmaf(w[r], v.x, acc[r][0]); acc[r][1] = fmaf(w[r], v.y, acc[r][1]); }
             };
 #pragma unroll
             for (int i = 0; i < kBdVv; i++) if (sub + i * nsub < nk) take(vreg[i], sub + i * nsub);

@@ -2728,7 +2728,8 @@ int32_t lum_profile(lum_rt* rt, int32_t trials, double* usec, char* display, siz
     const double us = (double)ms * 1000.0 / trials;
     rt->last_profile_usec = us;
     if (usec) *usec = us;
-    if (display && display_len)
+    if (display && display_len && rt->d.block_kind == 1) snprintf(display, display_len, "%.3f ms/token", us / 1000.0);
+    else if (display && display_len)
         snprintf(display, display_len, "%.3f ms/token; attention: %d splits per KV head, %s merge", us / 1000.0, rt->n_splits,
                  rt->n_splits < 2 ? "no" : rt->attn_cluster ? "cluster" : "ticket");
     return 0;

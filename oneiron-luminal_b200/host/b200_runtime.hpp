@@ -51,6 +51,15 @@ public:
     ~B200Runtime() { if (h_) lum_destroy(h_); }
 
     void load_model(const lum_model_desc& d) { ck(lum_model_init(h_, &d)); desc_ = d; }
+    // a decoder whose layers are described one by one (block_kind 1)
+    void load_model(const lum_model_desc& d, const std::vector<lum_layer_desc>& layers) {
+        if ((int)layers.size() != d.n_layers) throw Error(LUM_E_INVALID, "load_model: one descriptor per layer");
+        ck(lum_model_init_layers(h_, &d, layers.data()));
+        desc_ = d;
+    }
+    // logits of chosen rows of the next execute, then [rows][vocab]
+    void want_logits(const std::vector<int32_t>& rows) { ck(lum_want_logits(h_, rows.data(), (int32_t)rows.size())); n_want_ = rows.size(); }
+    std::vector<float> get_wanted() { std::vector<float> v(n_want_ * (size_t)desc_.vocab); ck(lum_get_wanted(h_, v.data(), v.size())); return v; }
     // `Runtime::load_llir` (src/op.rs:16) for a graph serialised as include/lum_llir.h describes
     void load_llir(const std::vector<uint8_t>& blob, int max_seq, lum_dtype kv, int max_new_tokens = 4096) {
         ck(lum_load_llir(h_, blob.data(), blob.size(), max_seq, kv, max_new_tokens));
@@ -151,7 +160,7 @@ private:
     void ck(int rc) { if (rc) throw Error(rc, lum_last_error(h_)); }
     lum_rt* h_ = nullptr;
     lum_model_desc desc_{};
-    size_t batch_n_ = 0;
+    size_t batch_n_ = 0, n_want_ = 0;
 };
 
 }  // namespace lum
