@@ -303,7 +303,7 @@ __device__ __forceinline__ void rows_epilogue8(const DenseArgs& a, int m, int n,
 
 namespace {
 constexpr int kDmThreads = 192;               // producer warp, tensor-core warp, four epilogue warps
-constexpr int kDmMaxStages = 8;
+constexpr int kDmMaxStages = 16;
 constexpr int kDmABytes = 128 * 128;          // 128 rows x one chunk
 
 __host__ __device__ constexpr uint32_t dm_idesc(int N) {      // kind::f16, bf16 x bf16 -> f32, both operands K-major, M = 128
@@ -324,13 +324,13 @@ __global__ void __launch_bounds__(kDmThreads, 1) dense_gemm_tc(const DenseArgs a
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int stage_bytes = kDmABytes + TN * 128;
     const uint32_t s_base = smem_u32(dm_smem);
-    const uint32_t bars = s_base + stages * stage_bytes;      // full[8], empty[8], acc_full[2], acc_empty[2], drained, then the slot
+    const uint32_t bars = s_base + stages * stage_bytes;      // full[16], empty[16], acc_full[2], acc_empty[2], drained, the slot, the abort word
     auto full = [&](int s) { return bars + s * 8; };
-    auto empty = [&](int s) { return bars + 64 + s * 8; };
-    auto acc_full = [&](int b) { return bars + 128 + b * 8; };
-    auto acc_empty = [&](int b) { return bars + 144 + b * 8; };
-    const uint32_t drained = bars + 160, slot = bars + 168;
-    volatile int* abort = (volatile int*)(dm_smem + stages * stage_bytes + 176);
+    auto empty = [&](int s) { return bars + 128 + s * 8; };
+    auto acc_full = [&](int b) { return bars + 256 + b * 8; };
+    auto acc_empty = [&](int b) { return bars + 272 + b * 8; };
+    const uint32_t drained = bars + 288, slot = bars + 296;
+    volatile int* abort = (volatile int*)(dm_smem + stages * stage_bytes + 304);
     if (tid == 0) {
         for (int s = 0; s < stages; s++) { mbar_init(full(s), 1); mbar_init(empty(s), 1); }
         for (int b = 0; b < 2; b++) { mbar_init(acc_full(b), 1); mbar_init(acc_empty(b), 128); }
@@ -343,7 +343,7 @@ __global__ void __launch_bounds__(kDmThreads, 1) dense_gemm_tc(const DenseArgs a
     tc_fence_before_sync();
     __syncthreads();
     tc_fence_after_sync();
-    const uint32_t tmem = *(volatile uint32_t*)(dm_smem + stages * stage_bytes + 168);
+    const uint32_t tmem = *(volatile uint32_t*)(dm_smem + stages * stage_bytes + 296);
 
     const int mt = (a.M + 127) / 128, ntile = (a.nt + TN - 1) / TN, n_tiles = mt * ntile;
     const int KC0 = a.seg[0].chunks, KC = KC0 + (a.nk > 1 ? a.seg[1].chunks : 0);
@@ -513,7 +513,9 @@ cudaError_t launch_dense_gemm(const DenseArgs& a_in, int sm_count, cudaStream_t 
         dense_gemm_f32<<<dim3((a.nt + 63) / 64, (a.M + 63) / 64), 256, 0, st>>>(a);
         return cudaGetLastError();
     }
-    // tile width: the fewest (rounds over the SMs) x (time of a tile); a narrow tile does not fill the tensor pipe
+    // tile width: the fewest (rounds over the SMs) x (time of a tile); a narrow tile does not fill the tensor pipe.  (With few rows a chunk
+    // of K takes about 0.4 us whatever the tile's width, so that narrower tiles on more SMs gain nothing: 64 rows x 27648 x K 4096 took
+    // 61 us with tiles of 256 and 84 us with tiles of 64.)
     const int mt = (a.M + 127) / 128;
     int TN = 256;
     double best = 1e30;
@@ -525,7 +527,7 @@ cudaError_t launch_dense_gemm(const DenseArgs& a_in, int sm_count, cudaStream_t 
     const int stage_bytes = kDmABytes + TN * 128;
     int stages = (220 * 1024) / stage_bytes;
     if (stages > kDmMaxStages) stages = kDmMaxStages;
-    const size_t smem = (size_t)stages * stage_bytes + 256;
+    const size_t smem = (size_t)stages * stage_bytes + 512;
     static bool attr_set = false;
     if (!attr_set) {
         const cudaError_t e = cudaFuncSetAttribute((const void*)dense_gemm_tc, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);

@@ -57,9 +57,10 @@ def test_prompt_portions_and_decoding(pkg, rt, tmp_path, name, dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_other_sizes(pkg, rt, tmp_path, dtype):
-    """One layer, sizes the kernels' tiles do not divide: one head, equal head counts, a width of 34, a single-token window."""
+    """One layer, sizes the kernels' tiles do not divide: one head, equal head counts, widths of 34 and 45, a single-token window."""
     for i, (cfg, n) in enumerate([(mc.config([mc.layer(1, 1, 5, 3, 1, 7)], width=34, vocab=17), 40),
                                   (mc.config([mc.layer(7, 7, 16, 20, 33, 65), mc.layer(7, 7, 8, 20, 2, 1)], width=130, vocab=1001, eps=1e-3), 90),
+                                  (mc.config([mc.layer(5, 5, 31, 9, 21, 27), mc.layer(3, 1, 17, 45, 64, None)], width=45, vocab=30), 140),
                                   (mc.config([mc.layer(24, 1, 96, 64, 40, None, mix=False)], width=64, vocab=64, mult=2.0), 70)]):
         both_ways(pkg, rt, tmp_path / str(i), cfg, mc.weights(cfg, 20 + i), dtype, n)
 
