@@ -88,7 +88,16 @@ typedef enum lum_slot {
     LUM_S_ATTN_NORM_BIAS, LUM_S_FINAL_NORM_BIAS,   /* layer norm: the added vector */
     LUM_S_V_MIX,                                   /* [1]: share of the first mixing layer's values */
     LUM_S_TEMP, LUM_S_DIST_R1, LUM_S_DIST_R2,      /* [heads]: score temperature; distance bias r1 * ln(1 + r2 * distance) */
-    LUM_S_ACT                                      /* [2]: the two learned numbers of xIELU */
+    LUM_S_ACT,                                     /* [2]: the two learned numbers of xIELU */
+    /* sequential sublayers (block_kind 2); file labels as above plus "l<i>.norm2", "l<i>.mlp.gate", "l<i>.mix.{q,k,v}.b", and: */
+    LUM_S_Q_CONV, LUM_S_K_CONV, LUM_S_V_CONV,      /* "mix.{q,k,v}.conv" [channels][taps]: short causal convolution, last tap = current token */
+    LUM_S_LQ1, LUM_S_LK1, LUM_S_LQ2, LUM_S_LK2,    /* "mix.lq1" ... [qk_dim]: weight of the second map of differential attention */
+    LUM_S_HC1_IN, LUM_S_HC1_OUT, LUM_S_HC1_MIX,    /* "hc1.in" [streams], "hc1.out" [streams], "hc1.mix" [from][to]: streams of the residual */
+    LUM_S_HC2_IN, LUM_S_HC2_OUT, LUM_S_HC2_MIX,
+    LUM_S_REC_Y, LUM_S_REC_Y_BIAS, LUM_S_REC_X, LUM_S_REC_X_BIAS,      /* gated linear recurrence: "mix.y[.b]", "mix.x[.b]" */
+    LUM_S_REC_CONV, LUM_S_REC_CONV_BIAS,           /* "mix.conv" [width][taps], "mix.conv.b" */
+    LUM_S_REC_RA, LUM_S_REC_RA_BIAS, LUM_S_REC_RI, LUM_S_REC_RI_BIAS,  /* "mix.ra" [blocks][size][size] (out, in), "mix.ra.b"; "mix.ri", "mix.ri.b" */
+    LUM_S_REC_LAM                                  /* "mix.lam" [width] */
 } lum_slot;
 
 typedef struct lum_model_desc {
@@ -137,6 +146,14 @@ typedef struct lum_model_desc {
      * in f32) and norms, scores, softmax, angles and the residual stream are f32. */
     int32_t block_kind, norm_kind, pos_kind, dist_bias;
     float residual_mult, logit_scale;
+    /* block_kind 2: sequential sublayers — x += mixer(norm1(x)), then x += ff(norm2(x)).  norm_kind 0, or 2: RMS norm whose stored weight is
+     * the gain minus one.  embed_scale multiplies the embedding.  streams 0: one residual vector, as written here; s >= 1 (at most 8): s
+     * copies x_1 .. x_s of it, a sublayer reading u = sum_s IN[s] x_s and leaving x_t = sum_s MIX[s][t] x_s + OUT[t] y (HC1_* for the mixer,
+     * HC2_* for the feed-forward); the model's output is their sum.  loop_times > 1: layers loop_start .. loop_stop - 1 run that many
+     * times in a row with the same weights; every pass has its own cache and state (a "layer run": lum_kv_* count runs, in the
+     * order they happen).  The mechanisms of a layer are chosen in lum_layer_desc. */
+    int32_t streams, loop_start, loop_stop, loop_times;
+    float embed_scale;
 } lum_model_desc;
 
 int32_t lum_model_init(lum_rt* rt, const lum_model_desc* desc);
@@ -150,6 +167,20 @@ typedef struct lum_layer_desc {
     int32_t n_q_heads, n_kv_heads, qk_dim, v_dim;
     int32_t window, v_mix, ffn;
     float scale;
+    /* block_kind 2 */
+    int32_t mixer;      /* 0 attention, 1 gated linear recurrence */
+    int32_t chunk;      /* > 0: position i sees j only if i / chunk == j / chunk */
+    int32_t conv_taps;  /* > 0: causal convolution per channel over that many tokens, on q, k and v or on the recurrence's input */
+    int32_t maps;       /* 2: differential attention — every head has two maps of queries and keys (rows [head][map][qk_dim]) over the same
+                           values; o = a1 - lambda a2, lambda = exp(LQ1 . LK1) - exp(LQ2 . LK2) + diff, RMS norm of o over the head (no gain),
+                           times 1 - diff.  0 / 1: one map */
+    int32_t head_norm;  /* 1: RMS norm of every head (and map) of q and k with one gain [qk_dim] for all of them, before the rotation */
+    int32_t qkv_bias;   /* 1: biases on the q, k, v projections */
+    int32_t rot_dims;   /* > 0 (even, at most qk_dim): dimensions k and k + rot_dims / 2 turn by position * rot_base^(-2 k / rot_dims) */
+    int32_t rec_width, rec_blocks;      /* recurrence: S_t = a S_(t-1) + sqrt(1 - a^2) i u, ln a = -8 r softplus(LAM), r and i from block-
+                                           diagonal products of u; the output is down-projected after multiplying with gelu(Y h) */
+    int32_t ffn_kind;   /* 0 down(xIELU(up h)); 1 clamped gate: g = min(gate h, limit), u = clamp(up h, +-limit), down(g sigmoid(1.702 g) (u + 1)) */
+    float rot_base, diff, ffn_limit;
 } lum_layer_desc;
 int32_t lum_model_init_layers(lum_rt* rt, const lum_model_desc* desc, const lum_layer_desc* layers);
 /* Replaces `set_data(id, data)` for weight tensors (crates/luminal_cuda/src/runtime.rs:160-165).  `data` (host or device memory) holds
@@ -252,6 +283,13 @@ int32_t lum_kv_copy(lum_rt* rt, int32_t src_seq, int32_t dst_seq, int32_t rows);
  * give back: the call succeeds and does nothing.  lum_kv_pool reports the pool: pages in all, pages free, rows per page
  * (all zero for a contiguous cache). */
 int32_t lum_kv_release(lum_rt* rt, int32_t seq);
+/* Layers with a state (recurrences, short convolutions; block_kind 2) keep it per sequence, as it is after the sequence's last token: such
+ * a sequence continues only where it stands (or anew from position 0), lum_kv_copy needs `rows` to be the source's length, and the state is
+ * saved and loaded whole.  lum_state_bytes: its size per sequence (0: the model has none); lum_state_save / lum_state_load: the selected
+ * sequence's, position = tokens it has seen (pair it with lum_kv_save / lum_kv_load of the same rows). */
+int32_t lum_state_bytes(const lum_rt* rt, size_t* bytes);
+int32_t lum_state_save(lum_rt* rt, void* host_out, size_t bytes, int32_t* position);
+int32_t lum_state_load(lum_rt* rt, const void* host, size_t bytes, int32_t position);
 int32_t lum_kv_pool(const lum_rt* rt, int32_t* pages_total, int32_t* pages_free, int32_t* page_rows);
 
 /* ---------------------------------------------------------------------------------------------

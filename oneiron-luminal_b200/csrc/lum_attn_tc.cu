@@ -296,8 +296,15 @@ cudaError_t launch_attn_prompt_tc(const AttnRowsArgs& a, cudaStream_t st) {
 // R (QT + 63) values instead of 128 x 64, into shared memory (up to 16 heads per K/V head).  Rows are consecutive positions of one
 // sequence.  Scores are kept in units of ln 2 (queries and bias carry the factor 1 / ln 2), so that a weight is one power of two.
 //
+// Two maps (differential attention): the CTAs of the two maps of a K/V head and the same rows are a cluster of two.  Each finishes its own
+// softmax; the second hands lambda * its output over through the first one's shared memory, and the first subtracts, norms the head
+// and stores.
+//
 // DVH: value dimensions a thread accumulates (half of the value size, rounded up to 16).
 namespace {
+__device__ __forceinline__ void cluster_st_f32x4(uint32_t addr, float4 v) {
+    asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "f"(v.x), "f"(v.y), "f"(v.z), "f"(v.w) : "memory");
+}
 constexpr float kLog2e = 1.4426950408889634f;
 __device__ __forceinline__ float ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 // x = hi + lo in bf16 with the high term cut off instead of rounded (no conversion instruction for it; |x - hi - lo| <= 2^-17 |x| all the same)
@@ -310,7 +317,8 @@ __device__ __forceinline__ void split2_cut(float x0, float x1, uint32_t* hi, uin
 constexpr int kBtTabMaxR = 16;                      // R (128 / R + 63) <= 1136 floats up to there
 constexpr int kBtMiscBytes = 2048 + 4608;           // barriers, row exchange, flags; the bias table
 struct BandSmem { int qlo, k, v, phi, plo, misc, total; };      // byte offsets; the high Q term is at 0
-__host__ __device__ inline BandSmem band_smem(int dkp, int dvp) {
+__host__ __device__ inline int band_xch_ld(int dvp) { return dvp + 4; }      // floats per row of the hand-over between two maps (from offset 0)
+__host__ __device__ inline BandSmem band_smem(int dkp, int dvp, int maps) {
     BandSmem s;
     s.qlo = 128 * dkp * 2;
     s.k = 2 * s.qlo;
@@ -318,6 +326,7 @@ __host__ __device__ inline BandSmem band_smem(int dkp, int dvp) {
     s.phi = s.v + 2 * kAtKT * dvp * 2;
     s.plo = s.phi + kAtPBytes;
     s.misc = s.plo + kAtPBytes;
+    if (maps == 2 && s.misc < 128 * band_xch_ld(dvp) * 4) s.misc = 128 * band_xch_ld(dvp) * 4;
     s.total = s.misc + kBtMiscBytes;
     return s;
 }
@@ -328,9 +337,10 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_band_tc(const BandArgs a) 
     extern __shared__ __align__(128) unsigned char smem[];
     const QkvArgs& p = a.p;
     const int dkp = p.dkp, dvp = p.dvp, kgr = dkp / 8, vgr = dvp / 8;
-    const BandSmem L = band_smem(dkp, dvp);
+    const BandSmem L = band_smem(dkp, dvp, p.maps);
+    const int maps = p.maps, kh = blockIdx.x, map = kh % maps;                       // kh: this map's keys; kvh: the values of both
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int R = p.n_q / p.n_kv, kvh = blockIdx.x, QT = 128 / R;
+    const int R = p.n_q / p.n_kv, kvh = kh / maps, QT = 128 / R;
     const int q0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * QT;      // later rows first: without a window they have the most keys
     const uint32_t s_base = smem_u32(smem);
     const uint32_t bar_s = s_base + L.misc, bar_o = bar_s + 8, tmem_slot = bar_s + 16;
@@ -364,7 +374,7 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_band_tc(const BandArgs a) 
         const int r = ch / kgr, c = ch - r * kgr, g = r / QT, m = q0 + (r - g * QT);
         uint4 hi = make_uint4(0u, 0u, 0u, 0u), lo = hi;
         if (g < R && m < a.M) {
-            const float4* src = (const float4*)(a.q + ((size_t)m * p.n_q + (size_t)kvh * R + g) * dkp + c * 8);
+            const float4* src = (const float4*)(a.q + (((size_t)m * p.n_q + (size_t)kvh * R + g) * maps + map) * dkp + c * 8);
             const float4 v0 = src[0], v1 = src[1];
             split2_cut(v0.x * kLog2e, v0.y * kLog2e, &hi.x, &lo.x); split2_cut(v0.z * kLog2e, v0.w * kLog2e, &hi.y, &lo.y);
             split2_cut(v1.x * kLog2e, v1.y * kLog2e, &hi.z, &lo.z); split2_cut(v1.z * kLog2e, v1.w * kLog2e, &hi.w, &lo.w);
@@ -374,15 +384,15 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_band_tc(const BandArgs a) 
     }
     __syncthreads();
     const int pos_max = s_flag[0], pos_min = s_flag[2];
-    const int first = pos_max < 0 ? 0 : (a.window > 0 && pos_min + 1 > a.window) ? pos_min + 1 - a.window : 0;     // no row sees an earlier key
+    const int first = pos_max < 0 ? 0 : a.chunk > 0 ? pos_min / a.chunk * a.chunk : (a.window > 0 && pos_min + 1 > a.window) ? pos_min + 1 - a.window : 0;     // no row sees an earlier key
     const int t_lo = first / kAtKT, n_t = pos_max >= 0 ? pos_max / kAtKT + 1 - t_lo : 0;
-    const int reach = a.window > 0 ? a.window : 0x7fffffff;    // this row sees distances 0 .. reach - 1
+    const int reach = a.chunk > 0 ? max(pos_row, 0) % a.chunk + 1 : a.window > 0 ? a.window : 0x7fffffff;    // this row sees distances 0 .. reach - 1
     const bool biased = a.r1 != nullptr, use_tab = biased && R <= kBtTabMaxR;
     const int TW = QT + kAtKT - 1, head = kvh * R + (row_ok ? g_row : 0);
     const float* my_tab = tab + (g_row < R ? g_row : 0) * TW + qi_row + kAtKT - 1 - half * 32;      // [-i]: key i of this thread's half tile
 
-    const size_t k_row = (size_t)p.n_kv * dkp, v_row = (size_t)p.n_kv * dvp;
-    const __nv_bfloat16* kc = (const __nv_bfloat16*)a.k_cache + (size_t)kvh * dkp;
+    const size_t k_row = (size_t)p.n_kv * maps * dkp, v_row = (size_t)p.n_kv * dvp;
+    const __nv_bfloat16* kc = (const __nv_bfloat16*)a.k_cache + (size_t)kh * dkp;
     const __nv_bfloat16* vc = (const __nv_bfloat16*)a.v_cache + (size_t)kvh * dvp;
     // one operand tile (i-th of this CTA): 64 positions x `gr` 16-byte groups; a warp takes 8 positions x 4 groups at a time.  One copy
     // group per call, empty beyond the last tile.
@@ -545,8 +555,46 @@ __global__ void __launch_bounds__(kAtThreads, 1) attn_band_tc(const BandArgs a) 
     x_max[half * 128 + row] = l_run;
     __syncthreads();
     const float l_tot = l_run + x_max[(half ^ 1) * 128 + row];
-    if (row_ok) {
-        const float inv = l_tot > 0.0f ? 1.0f / l_tot : 0.0f;
+    float inv = l_tot > 0.0f ? 1.0f / l_tot : 0.0f;
+    if (maps == 2) {
+        const int ld = band_xch_ld(dvp), e0 = half * DVH;
+        cluster_arrive_release();
+        cluster_wait_acquire();                                // the first map's CTA is done with its tiles
+        if (map == 1) {
+            float d1 = 0.0f, d2 = 0.0f;
+            for (int e = lane; e < p.dk; e += 32) { d1 = fmaf(a.lq1[e], a.lk1[e], d1); d2 = fmaf(a.lq2[e], a.lk2[e], d2); }
+            d1 = warp_sum(d1); d2 = warp_sum(d2);
+            const float f = inv * (expf(d1) - expf(d2) + a.diff);
+            const uint32_t to = cluster_map(s_base + (uint32_t)(row * ld + e0) * 4, 0u);
+#pragma unroll
+            for (int i = 0; i < DVH; i += 4)
+                if (e0 + i < dvp) cluster_st_f32x4(to + i * 4, make_float4(o_acc[i] * f, o_acc[i + 1] * f, o_acc[i + 2] * f, o_acc[i + 3] * f));
+        }
+        cluster_arrive_release();
+        cluster_wait_acquire();
+        if (map == 0) {
+            const float* other = (const float*)smem + row * ld + e0;
+            float ss = 0.0f;
+#pragma unroll
+            for (int i = 0; i < DVH; i += 4) {
+                if (e0 + i < dvp) {
+                    const float4 v = *(const float4*)(other + i);
+                    const float w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+                    for (int k = 0; k < 4; k++) {
+                        const float t = fmaf(o_acc[i + k], inv, -w[k]);
+                        o_acc[i + k] = t;
+                        if (e0 + i + k < p.dv) ss = fmaf(t, t, ss);
+                    }
+                }
+            }
+            __syncthreads();                                   // every l_run has been read
+            x_max[half * 128 + row] = ss;
+            __syncthreads();
+            inv = (1.0f - a.diff) / sqrtf((ss + x_max[(half ^ 1) * 128 + row]) / (float)p.dv + p.eps);
+        }
+    }
+    if (row_ok && map == 0) {
         const int col0 = head * p.dv, e0 = half * DVH;
         unsigned char* out = (unsigned char*)a.out.p;
         if ((p.dv & 7) == 0) {
@@ -577,7 +625,7 @@ bool band_prompt_tc_supported(const BandArgs& a) {
     const QkvArgs& p = a.p;
     const int R = p.n_kv > 0 ? p.n_q / p.n_kv : 0;
     return a.kv_bf16 && a.out_kind == WK_BF16 && a.row_seq == nullptr && R >= 1 && R <= 128 && p.n_q == R * p.n_kv && p.dkp % 16 == 0 && p.dvp % 16 == 0 &&
-           p.dvp <= 256 && band_smem(p.dkp, p.dvp).total <= 226 * 1024;
+           p.dvp <= 256 && p.maps <= 2 && band_smem(p.dkp, p.dvp, p.maps).total <= 226 * 1024;
 }
 
 cudaError_t launch_band_prompt_tc(const BandArgs& a, cudaStream_t st) {
@@ -585,13 +633,19 @@ cudaError_t launch_band_prompt_tc(const BandArgs& a, cudaStream_t st) {
     const int dvh = (a.p.dvp / 2 + 15) / 16 * 16;
     const void* fn = dvh <= 16 ? (const void*)attn_band_tc<16> : dvh <= 32 ? (const void*)attn_band_tc<32> : dvh <= 64 ? (const void*)attn_band_tc<64>
                      : dvh <= 96 ? (const void*)attn_band_tc<96> : (const void*)attn_band_tc<128>;
-    const int smem = band_smem(a.p.dkp, a.p.dvp).total;
+    BandArgs b = a;
+    if (b.p.maps < 1) b.p.maps = 1;
+    const int smem = band_smem(b.p.dkp, b.p.dvp, b.p.maps).total;
     const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
     if (e != cudaSuccess) return e;
     const int QT = 128 / (a.p.n_q / a.p.n_kv);
-    BandArgs b = a;
     void* params[] = {&b};
-    return cudaLaunchKernel(fn, dim3(a.p.n_kv, (a.M + QT - 1) / QT), dim3(kAtThreads), params, (size_t)smem, st);
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(b.p.n_kv * b.p.maps, (a.M + QT - 1) / QT); cfg.blockDim = dim3(kAtThreads); cfg.dynamicSmemBytes = (size_t)smem; cfg.stream = st;
+    cudaLaunchAttribute at[1];
+    at[0].id = cudaLaunchAttributeClusterDimension; at[0].val.clusterDim.x = 2; at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
+    cfg.attrs = at; cfg.numAttrs = b.p.maps == 2 ? 1 : 0;
+    return cudaLaunchKernelExC(&cfg, fn, params);
 }
 
 }  // namespace lum

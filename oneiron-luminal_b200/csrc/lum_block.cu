@@ -1,11 +1,15 @@
-// Row-wise kernels of decoder layers whose sublayers share one norm, and their attention: norms, query / key preparation with the
-// cache append, and attention over a window with learned per-head temperature and distance bias.
+// Row-wise kernels of decoder layers that are described one by one, and their attention: norms, residual streams, query / key
+// preparation with the cache append, and attention over a window or a chunk with learned per-head temperature and distance bias, or
+// as the difference of two maps.
 //
 //   norm_rows     RMS or layer norm of rows of the residual stream -> operand of the next product
+//   stream_rows   several residual streams: a sublayer's output taken in, the next sublayer's input mixed and normalised
 //   qkv_rows      queries and keys normalised over the whole projection, queries scaled (score factor x temperature), values mixed
 //                 with the first mixing layer's; keys and values rounded to the cache type and appended
+//   qkv_head_rows the same for heads prepared one by one: short convolution, norm per head, rotation
 //   attn_band     attention of single rows over the cache: any head sizes, any number of query heads per K/V head, f32 or bf16
-//                 cache.  FUSED: one row, with all of qkv_rows in the prologue (a decode step's attention is one kernel).
+//                 cache.  PREP 1 / 2: one row, with all of qkv_rows / qkv_head_rows in the prologue (a decode step's attention is one
+//                 kernel).
 // Everything here is computed in f32.  The tensor-core form for prompts is in lum_attn_tc.cu.
 #include <cuda_bf16.h>
 #include <cstdlib>
@@ -44,7 +48,7 @@ __global__ void __launch_bounds__(256) norm_rows(const NormRowsArgs a) {
     const float inv = 1.0f / sqrtf(block_sum(s, red, tid, 256, 1) / (float)W + a.norm.eps);
     auto value = [&](int k) -> float {
         if (k >= W) return 0.0f;
-        float v = (nr_row[k] - mean) * inv * a.norm.gain[k];
+        float v = (nr_row[k] - mean) * inv * (a.norm.gain0 + a.norm.gain[k]);
         return a.norm.bias ? v + a.norm.bias[k] : v;
     };
     if (a.kind == WK_BF16) {
@@ -53,7 +57,10 @@ __global__ void __launch_bounds__(256) norm_rows(const NormRowsArgs a) {
             if (vec && g * 8 + 8 <= W) {
 #pragma unroll
                 for (int h = 0; h < 2; h++) {
-                    const float4 v = ((const float4*)nr_row)[g * 2 + h], gn = ((const float4*)a.norm.gain)[g * 2 + h];
+                    const float4 v = ((const float4*)nr_row)[g * 2 + h];
+                    float4 gn = ((const float4*)a.norm.gain)[g * 2 + h];
+                    const float z = a.norm.gain0;
+                    gn = make_float4(gn.x + z, gn.y + z, gn.z + z, gn.w + z);
                     const float4 b = a.norm.bias ? ((const float4*)a.norm.bias)[g * 2 + h] : make_float4(0.f, 0.f, 0.f, 0.f);
                     f[4 * h] = (v.x - mean) * inv * gn.x + b.x; f[4 * h + 1] = (v.y - mean) * inv * gn.y + b.y;
                     f[4 * h + 2] = (v.z - mean) * inv * gn.z + b.z; f[4 * h + 3] = (v.w - mean) * inv * gn.w + b.w;
@@ -160,6 +167,228 @@ cudaError_t launch_qkv_rows(const BandArgs& a, cudaStream_t st) {
     return cudaGetLastError();
 }
 
+// ------------------------------------------------------------------------------------------------ heads prepared one by one
+// One head (and map) of n dimensions in shared memory, by one warp: RMS norm with a shared gain, then the rotation, in place.
+__device__ __forceinline__ void head_norm_rotate(float* v, int n, const float* gain, float eps, const float2* rot, int rot_dims, int lane) {
+    __syncwarp();
+    if (gain) {
+        float s = 0.0f;
+        for (int e = lane; e < n; e += 32) s = fmaf(v[e], v[e], s);
+        const float inv = 1.0f / sqrtf(warp_sum(s) / (float)n + eps);
+        for (int e = lane; e < n; e += 32) v[e] = v[e] * inv * gain[e];
+        __syncwarp();
+    }
+    const int half = rot_dims / 2;
+    for (int e = lane; e < half; e += 32) {
+        const float2 cs = rot[e];
+        const float x = v[e], y = v[e + half];
+        v[e] = x * cs.x - y * cs.y;
+        v[e + half] = fmaf(y, cs.x, x * cs.y);
+    }
+    __syncwarp();
+}
+// Rows of a pass, RB at a time; the convolved columns of a row lie in shared memory until its heads are done.
+template <int RB>
+__global__ void __launch_bounds__(256) qkv_head_rows(const BandArgs a) {
+    extern __shared__ __align__(16) float qh[];
+    const QkvArgs& p = a.p;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int nq = p.n_q * p.maps, nk = p.n_kv * p.maps, half = p.rot_dims / 2;
+    const int m0 = blockIdx.x * RB, nr = min(RB, a.M - m0);
+    bool bad = false;
+    for (int r = 0; r < nr; r++) {
+        const int pos = a.row_pos[m0 + r], seq = a.row_seq ? a.row_seq[m0 + r] : a.seq0;
+        bad = bad || pos < 0 || pos >= a.max_seq || seq < 0 || seq >= a.max_batch;
+    }
+    if (bad) {
+        if (tid == 0) atomicOr(a.status, LUM_ST_BAD_POS);
+        return;
+    }
+    const size_t ring_seq = (size_t)p.conv.taps * p.conv.ch;
+    if (p.conv.taps == 4 && !a.row_seq && m0 >= 3) {                       // the rows before are in this pass: a sliding window in registers
+        for (int c = tid * 4; c < p.ld; c += 1024) {
+            float4 w[4];                                                   // of one column each
+#pragma unroll
+            for (int i = 0; i < 4; i++) w[i] = *(const float4*)(p.conv.w + (size_t)(c + i) * 4);
+            const float* src = p.qkv + (size_t)(m0 - 3) * p.ld + c;
+            float4 x[RB + 3];
+#pragma unroll
+            for (int r = 0; r < RB + 3; r++) if (r < nr + 3) x[r] = *(const float4*)(src + (size_t)r * p.ld);
+#pragma unroll
+            for (int r = 0; r < RB; r++) {
+                if (r < nr) {
+                    float4 o;
+                    o.x = fmaf(w[0].w, x[r + 3].x, fmaf(w[0].z, x[r + 2].x, fmaf(w[0].y, x[r + 1].x, w[0].x * x[r].x)));
+                    o.y = fmaf(w[1].w, x[r + 3].y, fmaf(w[1].z, x[r + 2].y, fmaf(w[1].y, x[r + 1].y, w[1].x * x[r].y)));
+                    o.z = fmaf(w[2].w, x[r + 3].z, fmaf(w[2].z, x[r + 2].z, fmaf(w[2].y, x[r + 1].z, w[2].x * x[r].z)));
+                    o.w = fmaf(w[3].w, x[r + 3].w, fmaf(w[3].z, x[r + 2].w, fmaf(w[3].y, x[r + 1].w, w[3].x * x[r].w)));
+                    *(float4*)(qh + r * p.ld + c) = o;
+                }
+            }
+        }
+    } else {
+        for (int r = 0; r < nr; r++) {
+            const int m = m0 + r, pos = a.row_pos[m], seq = a.row_seq ? a.row_seq[m] : a.seq0;
+            const float* src = p.qkv + (size_t)m * p.ld;
+            float* ring = p.conv.ring + seq * ring_seq;
+            for (int c = tid; c < p.ld; c += 256) {
+                qh[r * p.ld + c] = conv_at(p.conv, ring, src, p.ld, a.row_seq ? 0 : m, pos, c);
+                // one row of its sequence: its value takes the place in the ring that no row of this pass reads
+                if (p.conv.taps > 0 && (a.row_seq || a.M == 1)) ring[(size_t)(pos % p.conv.taps) * p.conv.ch + c] = src[c];
+            }
+        }
+    }
+    __syncthreads();
+    for (int job = warp; job < nr * (nq + nk); job += 8) {
+        const int r = job / (nq + nk), h = job - r * (nq + nk), m = m0 + r, pos = a.row_pos[m];
+        const bool is_q = h < nq;
+        float* v = qh + r * p.ld + (is_q ? p.q_off + h * p.dk : p.k_off + (h - nq) * p.dk);
+        head_norm_rotate(v, p.dk, is_q ? p.q_gain : p.k_gain, p.eps, p.rot + (size_t)pos * half, p.rot_dims, lane);
+        if (is_q) {
+            float* o = a.q_out + ((size_t)m * nq + h) * p.dkp;
+            for (int e = lane; e < p.dkp; e += 32) o[e] = e < p.dk ? v[e] * p.scale : 0.0f;
+        } else {
+            const size_t ko = kv_phys_row(a.pg, a.row_seq ? a.row_seq[m] : a.seq0, a.max_seq, pos) * nk * p.dkp + (size_t)(h - nq) * p.dkp;
+            for (int e = lane; e < p.dkp; e += 32) cache_store(a.k_cache, a.kv_bf16, ko + e, e < p.dk ? v[e] : 0.0f);
+        }
+    }
+    for (int r = 0; r < nr; r++) {
+        const size_t vo = kv_phys_row(a.pg, a.row_seq ? a.row_seq[m0 + r] : a.seq0, a.max_seq, a.row_pos[m0 + r]) * p.n_kv * p.dvp;
+        const float* v = qh + r * p.ld + p.v_off;
+        for (int i = tid; i < p.n_kv * p.dvp; i += 256) {
+            const int h = i / p.dvp, e = i - h * p.dvp;
+            cache_store(a.v_cache, a.kv_bf16, vo + i, e < p.dv ? v[h * p.dv + e] : 0.0f);
+        }
+    }
+}
+cudaError_t launch_qkv_head_rows(const BandArgs& a, cudaStream_t st) {
+    if (a.M <= 0 || !a.p.per_head || a.p.maps < 1 || a.p.ld % 4) return cudaErrorInvalidValue;
+    const size_t row = (size_t)a.p.ld * 4;
+    const int RB = a.row_seq || a.M < 64 ? 1 : row * 4 <= 100 * 1024 ? 4 : row * 2 <= 200 * 1024 ? 2 : 1;
+    if (row * RB > 200 * 1024) return cudaErrorInvalidValue;
+    const void* fn = RB == 4 ? (const void*)qkv_head_rows<4> : RB == 2 ? (const void*)qkv_head_rows<2> : (const void*)qkv_head_rows<1>;
+    if (row * RB > 48 * 1024) {
+        const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        if (e != cudaSuccess) return e;
+    }
+    BandArgs b = a;
+    void* params[] = {&b};
+    return cudaLaunchKernel(fn, dim3((a.M + RB - 1) / RB), dim3(256), params, row * RB, st);
+}
+
+// ------------------------------------------------------------------------------------------------ residual streams
+// One CTA per row.  SM: streams the registers are laid out for.
+template <int SM>
+__global__ void __launch_bounds__(256) stream_rows(const StreamRowsArgs a) {
+    extern __shared__ __align__(16) float sr_row[];
+    __shared__ float red[32], mix[SM * SM], out[SM], nxt[SM];
+    const StreamArgs& h = a.hc;
+    const int m = blockIdx.x, tid = threadIdx.x, W = a.width, n = h.n;
+    if (tid < n) {
+        out[tid] = h.out ? h.out[tid] : 1.0f;
+        nxt[tid] = h.next ? h.next[tid] : 1.0f;
+    }
+    for (int i = tid; i < n * n; i += 256) mix[i] = h.mix ? h.mix[i] : (i / n == i % n ? 1.0f : 0.0f);
+    if (a.use_pdl) { pdl_launch_dependents(); pdl_grid_wait(); }
+    int tok = 0;
+    if (!a.y) {
+        tok = a.state ? a.state->tok : a.row_tok[m];
+        const int pos = a.state ? a.state->pos : a.row_pos[m];
+        if (tok < 0 || tok >= a.vocab) { if (tid == 0) atomicOr(a.status, LUM_ST_BAD_TOKEN); tok = 0; }
+        if (pos < 0 || pos >= a.max_seq) { if (tid == 0) atomicOr(a.status, LUM_ST_BAD_POS); }
+    }
+    __syncthreads();
+    float* x = h.x + (size_t)m * n * h.ldx;
+    float ss = 0.0f;
+    const bool vec_table = (W & 3) == 0;
+    for (int i = tid; i < h.ldx / 4; i += 256) {
+        float4 y, u = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (a.y) {
+            y = ((const float4*)(a.y + (size_t)m * a.ldy))[i];
+            float4 old[SM];
+#pragma unroll
+            for (int s = 0; s < SM; s++) if (s < n) old[s] = ((const float4*)(x + (size_t)s * h.ldx))[i];
+#pragma unroll
+            for (int t = 0; t < SM; t++) {
+                if (t < n) {
+                    const float o = out[t];
+                    float4 v = make_float4(o * y.x, o * y.y, o * y.z, o * y.w);
+#pragma unroll
+                    for (int s = 0; s < SM; s++)
+                        if (s < n) {
+                            const float w = mix[s * n + t];
+                            v.x = fmaf(w, old[s].x, v.x); v.y = fmaf(w, old[s].y, v.y); v.z = fmaf(w, old[s].z, v.z); v.w = fmaf(w, old[s].w, v.w);
+                        }
+                    ((float4*)(x + (size_t)t * h.ldx))[i] = v;
+                    const float g = nxt[t];
+                    u.x = fmaf(g, v.x, u.x); u.y = fmaf(g, v.y, u.y); u.z = fmaf(g, v.z, u.z); u.w = fmaf(g, v.w, u.w);
+                }
+            }
+        } else {
+            float e[4] = {0.f, 0.f, 0.f, 0.f};
+            const size_t o = (size_t)tok * W + 4 * i;
+            if (vec_table && a.table_kind == WK_BF16) {
+                const uint2 b = *(const uint2*)((const uint16_t*)a.table + o);
+                e[0] = __uint_as_float(b.x << 16); e[1] = __uint_as_float(b.x & 0xffff0000u); e[2] = __uint_as_float(b.y << 16); e[3] = __uint_as_float(b.y & 0xffff0000u);
+                if (4 * i >= W) e[0] = e[1] = e[2] = e[3] = 0.0f;
+            } else {
+#pragma unroll
+                for (int k = 0; k < 4; k++)
+                    if (4 * i + k < W) e[k] = a.table_kind == WK_BF16 ? bf16_bits_to_f32(((const uint16_t*)a.table)[o + k]) : ((const float*)a.table)[o + k];
+            }
+            y = make_float4(e[0] * a.scale, e[1] * a.scale, e[2] * a.scale, e[3] * a.scale);
+            for (int t = 0; t < n; t++) {
+                ((float4*)(x + (size_t)t * h.ldx))[i] = y;
+                const float g = nxt[t];
+                u.x = fmaf(g, y.x, u.x); u.y = fmaf(g, y.y, u.y); u.z = fmaf(g, y.z, u.z); u.w = fmaf(g, y.w, u.w);
+            }
+        }
+        if (h.u) ((float4*)(h.u + (size_t)m * h.ldx))[i] = u;
+        else {
+            ((float4*)sr_row)[i] = u;
+            ss = fmaf(u.x, u.x, ss); ss = fmaf(u.y, u.y, ss); ss = fmaf(u.z, u.z, ss); ss = fmaf(u.w, u.w, ss);      // (columns beyond W are zero)
+        }
+    }
+    if (h.u) return;
+    const float inv = 1.0f / sqrtf(block_sum(ss, red, tid, 256, 1) / (float)W + a.norm.eps);
+    if (a.kind == WK_BF16) {
+        for (int g = tid; g < a.out.chunks * 8; g += 256) {
+            uint32_t w[4];
+            float f[8];
+#pragma unroll
+            for (int i = 0; i < 8; i++) f[i] = g * 8 + i < W ? sr_row[g * 8 + i] * inv * (a.norm.gain0 + a.norm.gain[g * 8 + i]) : 0.0f;
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                const __nv_bfloat162 b = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
+                w[i] = *(const uint32_t*)&b;
+            }
+            *(uint4*)((unsigned char*)a.out.p + row_operand_off(WK_BF16, a.out.chunks, m, g * 8)) = make_uint4(w[0], w[1], w[2], w[3]);
+        }
+    } else {
+        float* o = (float*)a.out.p + (size_t)m * a.out.chunks * 32;
+        for (int k = tid; k < a.out.chunks * 32; k += 256) o[k] = k < W ? sr_row[k] * inv * (a.norm.gain0 + a.norm.gain[k]) : 0.0f;
+    }
+}
+cudaError_t launch_stream_rows(const StreamRowsArgs& a_in, cudaStream_t st) {
+    StreamRowsArgs a = a_in;
+    if (a.M <= 0 || a.hc.n < 1 || a.hc.n > kMaxStreams || a.hc.ldx % 8 || a.hc.ldx < a.width || (!a.hc.u && (a.norm.mode != NORM_RMS || a.width > a.out.chunks * chunk_elems(a.kind))))
+        return cudaErrorInvalidValue;
+    const void* fn = a.hc.n <= 1 ? (const void*)stream_rows<1> : a.hc.n <= 2 ? (const void*)stream_rows<2> : a.hc.n <= 4 ? (const void*)stream_rows<4> : (const void*)stream_rows<8>;
+    const size_t smem = a.hc.u ? 0 : (size_t)a.hc.ldx * 4;
+    if (smem > 48 * 1024) {
+        const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        if (e != cudaSuccess) return e;
+        if (smem > 200 * 1024) return cudaErrorInvalidValue;
+    }
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(a.M); cfg.blockDim = dim3(256); cfg.dynamicSmemBytes = smem; cfg.stream = st;
+    cudaLaunchAttribute at[1];
+    at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization; at[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = at; cfg.numAttrs = a.use_pdl ? 1 : 0;
+    void* params[] = {&a};
+    return cudaLaunchKernelExC(&cfg, fn, params);
+}
+
 // ------------------------------------------------------------------------------------------------ attention, row by row
 // One CTA = (split of the visible keys, K/V head and block of up to 8 of its query heads, row).  64 keys at a time:
 //   scores   4 lanes per key, each a share of the head dimension for all 8 queries; two shuffles; distance bias; shared memory
@@ -168,8 +397,10 @@ cudaError_t launch_qkv_rows(const BandArgs& a, cudaStream_t st) {
 // A tile's key and value loads are all issued before anything of the previous tile is waited for again: the next tile's keys are in
 // flight during this tile's softmax, its values during its scores.
 // The splits of a row are the CTAs of a thread-block cluster and fold their (maximum, sum, vector) through its shared memory.
+// With two maps the cluster holds the splits of both (rank = map * splits + split): keys and queries are the map's, values are shared,
+// and the fold subtracts the maps, head by head.
 namespace {
-constexpr int kBdTK = 64, kBdR = 8, kBdMaxSplits = 16;
+constexpr int kBdTK = 64, kBdR = 8, kBdMaxSplits = 16;    // (splits of both maps together)
 constexpr int kBdKv = 4, kBdVv = 16;     // 16-byte key groups / value pairs of a tile a thread keeps in registers (longer heads: the rest is loaded where used)
 struct BdSmem {      // offsets in floats
     int q, sc, red, o, ml, wgt, knew, vnew, part, total;
@@ -197,25 +428,77 @@ __device__ __forceinline__ float2 band_pair(uint32_t w) { return make_float2(__u
 __device__ __forceinline__ float2 band_pair(float2 v) { return v; }
 
 // RB: query heads the registers are laid out for (4 or 8)
-template <bool BF16, bool FUSED, int RB>
+// PREP: 0 rows prepared before, 1 prologue over the whole projection, 2 prologue head by head
+template <bool BF16, int PREP, int RB>
 __global__ void __launch_bounds__(256, 2) attn_band(const BandArgs a, int S, int HB) {
     extern __shared__ __align__(16) float bd[];
     const QkvArgs& p = a.p;
     const BdSmem L = bd_layout(p.dkp, p.dvp);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int sp = blockIdx.x, kvh = blockIdx.y / HB, hb = blockIdx.y % HB, m = blockIdx.z;
+    constexpr bool FUSED = PREP != 0;
+    const int maps = PREP == 1 ? 1 : p.maps, map = blockIdx.x / S, sp = blockIdx.x - map * S;
+    const int kvh = blockIdx.y / HB, hb = blockIdx.y % HB, m = blockIdx.z;
     const int R = p.n_q / p.n_kv, r0 = hb * kBdR, nr = min(kBdR, R - r0), head0 = kvh * R + r0;
     float *q_s = bd + L.q, *sc = bd + L.sc, *red = bd + L.red, *o_s = bd + L.o, *m_s = bd + L.ml, *l_s = m_s + 8, *c_s = m_s + 16;
-    if (FUSED) { pdl_launch_dependents(); pdl_grid_wait(); }
+    __shared__ float lam_s;
+    if (FUSED) pdl_launch_dependents();
+    if (maps == 2 && warp == 7) {                              // the second map's weight (weights only: nothing to wait for)
+        float d1 = 0.0f, d2 = 0.0f;
+        for (int e = lane; e < p.dk; e += 32) { d1 = fmaf(a.lq1[e], a.lk1[e], d1); d2 = fmaf(a.lq2[e], a.lk2[e], d2); }
+        d1 = warp_sum(d1); d2 = warp_sum(d2);
+        if (lane == 0) lam_s = expf(d1) - expf(d2) + a.diff;
+    }
+    if (FUSED) pdl_grid_wait();
     const int pos = FUSED ? a.state->pos : a.row_pos[m];
-    const int seq = FUSED ? 0 : (a.row_seq ? a.row_seq[m] : a.seq0);
+    const int seq = FUSED ? (PREP == 2 ? a.seq0 : 0) : (a.row_seq ? a.row_seq[m] : a.seq0);
     if (pos < 0 || pos >= a.max_seq || seq < 0 || seq >= a.max_batch) {          // (the same for every CTA of the cluster)
         if (FUSED && tid == 0 && sp == 0) atomicOr(a.status, LUM_ST_BAD_POS);
         return;
     }
-    const size_t k_row = (size_t)p.n_kv * p.dkp, v_row = (size_t)p.n_kv * p.dvp;
+    const size_t k_row = (size_t)p.n_kv * maps * p.dkp, v_row = (size_t)p.n_kv * p.dvp;
+    const int kh = kvh * maps + map;                           // this map's keys
 
-    if (FUSED) {
+    if (PREP == 2) {
+        const size_t prow = kv_phys_row(a.pg, 0, 0, pos);
+        float* ring = p.conv.ring ? p.conv.ring + (size_t)seq * p.conv.taps * p.conv.ch : nullptr;
+        float* ring_now = ring + (size_t)(p.conv.taps ? pos % p.conv.taps : 0) * p.conv.ch;
+        const float2* rot = p.rot + (size_t)pos * (p.rot_dims / 2);
+        // a warp per head: this CTA's queries, its key, its value; the step's own values enter the ring once per head (the CTA of the
+        // first split; the row of the ring they replace is read by nobody)
+        for (int job = warp; job < kBdR + 2; job += 8) {
+            const bool is_q = job < kBdR, is_k = job == kBdR;
+            float* v = is_q ? q_s + job * p.dkp : bd + L.part + (is_k ? p.dvp : 0);      // (f32 forms of key and value: the shares' area is free yet)
+            const int n = job == kBdR + 1 ? p.dv : p.dk, np = job == kBdR + 1 ? p.dvp : p.dkp;
+            const int c0 = is_q ? p.q_off + ((head0 + job) * maps + map) * p.dk : is_k ? p.k_off + kh * p.dk : p.v_off + kvh * p.dv;
+            const bool real = !is_q || job < nr, keep = sp == 0 && (is_q || (hb == 0 && (is_k || map == 0)));
+            for (int e = lane; e < np; e += 32) {
+                float t = 0.0f;
+                if (real && e < n) {
+                    t = conv_at(p.conv, ring, p.qkv, 0, 0, pos, c0 + e);
+                    if (keep && p.conv.taps > 0) ring_now[c0 + e] = p.qkv[c0 + e];
+                }
+                v[e] = t;
+            }
+            if (is_q) {
+                if (real) {
+                    head_norm_rotate(v, p.dk, p.q_gain, p.eps, rot, p.rot_dims, lane);
+                    for (int e = lane; e < p.dk; e += 32) v[e] *= p.scale;
+                }
+            } else if (is_k) {
+                head_norm_rotate(v, p.dk, p.k_gain, p.eps, rot, p.rot_dims, lane);
+                for (int e = lane; e < p.dkp; e += 32) {
+                    cache_store(bd + L.knew, BF16, e, v[e]);
+                    if (keep) cache_store(a.k_cache, BF16, prow * k_row + (size_t)kh * p.dkp + e, v[e]);
+                }
+            } else {
+                for (int e = lane; e < p.dvp; e += 32) {
+                    const float t = v[e];
+                    cache_store(bd + L.vnew, BF16, e, t);
+                    if (keep) cache_store(a.v_cache, BF16, prow * v_row + (size_t)kvh * p.dvp + e, t);
+                }
+            }
+        }
+    } else if (PREP == 1) {
         const float *q = p.qkv + p.q_off, *k = p.qkv + p.k_off, *v = p.qkv + p.v_off;
         const float iq = proj_inv_rms(q, p.n_q * p.dk, p.q_gain, p.eps, red, tid), ik = proj_inv_rms(k, p.n_kv * p.dk, p.k_gain, p.eps, red, tid);
         for (int i = tid; i < kBdR * p.dkp; i += 256) {
@@ -240,11 +523,11 @@ __global__ void __launch_bounds__(256, 2) attn_band(const BandArgs a, int S, int
     } else {
         for (int i = tid; i < kBdR * p.dkp; i += 256) {
             const int r = i / p.dkp;
-            q_s[i] = r < nr ? a.q[((size_t)m * p.n_q + head0 + r) * p.dkp + (i - r * p.dkp)] : 0.0f;
+            q_s[i] = r < nr ? a.q[(((size_t)m * p.n_q + head0 + r) * maps + map) * p.dkp + (i - r * p.dkp)] : 0.0f;
         }
     }
     if (tid < 8) { m_s[tid] = -INFINITY; l_s[tid] = 0.0f; }
-    const int lo = (a.window > 0 && pos + 1 > a.window) ? pos + 1 - a.window : 0;
+    const int lo = a.chunk > 0 ? pos / a.chunk * a.chunk : (a.window > 0 && pos + 1 > a.window) ? pos + 1 - a.window : 0;
     const int per = (pos + 1 - lo + S - 1) / S, k0 = lo + sp * per, k1 = min(pos + 1, k0 + per);
     const int npair = p.dvp / 2, nsub = npair >= 256 ? 1 : 256 / npair, sub = tid / npair, dv2 = tid - sub * npair;
     float acc[RB][2];
@@ -256,12 +539,12 @@ __global__ void __launch_bounds__(256, 2) attn_band(const BandArgs a, int S, int
     // row `j` of this K/V head (the row of this very step: from shared memory, its store to the cache may still be on the way)
     auto key_row = [&](int j) -> const char* {
         if (FUSED && j == pos) return (const char*)(bd + L.knew);
-        return (const char*)a.k_cache + (kv_phys_row(a.pg, seq, FUSED ? 0 : a.max_seq, j) * k_row + (size_t)kvh * p.dkp) * esz;
+        return (const char*)a.k_cache + (kv_phys_row(a.pg, FUSED ? 0 : seq, FUSED ? 0 : a.max_seq, j) * k_row + (size_t)kh * p.dkp) * esz;
     };
     using VRaw = typename BandPair<BF16>::type;
     auto value_pair = [&](int j) -> VRaw {
         const char* vr = (const char*)(bd + L.vnew);
-        if (!(FUSED && j == pos)) vr = (const char*)a.v_cache + (kv_phys_row(a.pg, seq, FUSED ? 0 : a.max_seq, j) * v_row + (size_t)kvh * p.dvp) * esz;
+        if (!(FUSED && j == pos)) vr = (const char*)a.v_cache + (kv_phys_row(a.pg, FUSED ? 0 : seq, FUSED ? 0 : a.max_seq, j) * v_row + (size_t)kvh * p.dvp) * esz;
         return *((const VRaw*)vr + dv2);
     };
     float d[RB];
@@ -376,6 +659,50 @@ __global__ void __launch_bounds__(256, 2) attn_band(const BandArgs a, int S, int
     }
     __syncthreads();
     float* wgt = bd + L.wgt;
+    if (maps == 2) {
+        const int C = 2 * S, rank = blockIdx.x;
+        cluster_arrive_release();
+        cluster_wait_acquire();
+        const uint32_t ml = smem_u32(m_s), ob = smem_u32(o_s);
+        if (tid < 2 * nr) {                                    // weights of the splits of (map, head)
+            const int mp = tid / nr, r = tid - mp * nr;
+            float M = -INFINITY, Ls = 0.0f;
+            for (int s = 0; s < S; s++) M = fmaxf(M, cluster_ld_f32(cluster_map(ml + r * 4, (uint32_t)(mp * S + s))));
+            for (int s = 0; s < S; s++) {
+                const uint32_t from = (uint32_t)(mp * S + s);
+                const float ms = cluster_ld_f32(cluster_map(ml + r * 4, from)), c = ms == -INFINITY ? 0.0f : expf(ms - M);
+                Ls = fmaf(cluster_ld_f32(cluster_map(ml + 32 + r * 4, from)), c, Ls);
+                wgt[from * kBdR + r] = c;
+            }
+            const float f = (mp ? -lam_s : 1.0f) / Ls;
+            for (int s = 0; s < S; s++) wgt[(mp * S + s) * kBdR + r] *= f;
+        }
+        __syncthreads();
+        float* dif = bd + L.part;
+        for (int r = rank; r < nr; r += C) {                   // whole heads, dealt to the CTAs of the cluster
+            float ss = 0.0f;
+            for (int e = tid; e < p.dv; e += 256) {
+                float v = 0.0f;
+                for (int s = 0; s < C; s++) v = fmaf(cluster_ld_f32(cluster_map(ob + (r * p.dvp + e) * 4, (uint32_t)s)), wgt[s * kBdR + r], v);
+                dif[e] = v;
+                ss = fmaf(v, v, ss);
+            }
+            const float f = (1.0f - a.diff) / sqrtf(block_sum(ss, red, tid, 256, 1) / (float)p.dv + p.eps);
+            for (int e = tid; e < p.dv; e += 256) {
+                const float v = dif[e] * f;
+                const int col = (head0 + r) * p.dv + e;
+                if (FUSED) a.out_x[col] = v;
+                else {
+                    unsigned char* o = (unsigned char*)a.out.p + row_operand_off(a.out_kind, a.out.chunks, m, col);
+                    if (a.out_kind == WK_BF16) *(__nv_bfloat16*)o = __float2bfloat16_rn(v);
+                    else *(float*)o = v;
+                }
+            }
+        }
+        cluster_arrive_release();
+        cluster_wait_acquire();
+        return;
+    }
     if (S > 1) {
         cluster_arrive_release();
         cluster_wait_acquire();
@@ -418,34 +745,38 @@ bool band_supported(int n_q, int n_kv, int dkp, int dvp) {
 
 static cudaError_t launch_band(const BandArgs& a_in, int rows, bool fused, int sm_count, cudaStream_t st) {
     BandArgs a = a_in;
+    if (a.p.maps < 1) a.p.maps = 1;
     const QkvArgs& p = a.p;
+    if (p.maps > 2 || (p.maps == 2 && fused && !p.per_head)) return cudaErrorInvalidValue;
     if (!band_supported(p.n_q, p.n_kv, p.dkp, p.dvp) || rows <= 0) return cudaErrorInvalidValue;
     const int R = p.n_q / p.n_kv;
     int HB = (R + kBdR - 1) / kBdR;
     const size_t smem = (size_t)bd_layout(p.dkp, p.dvp).total * 4;
-    static const void* const fns[2][2][2] = {
-        {{(const void*)attn_band<false, false, 4>, (const void*)attn_band<false, false, 8>}, {(const void*)attn_band<false, true, 4>, (const void*)attn_band<false, true, 8>}},
-        {{(const void*)attn_band<true, false, 4>, (const void*)attn_band<true, false, 8>}, {(const void*)attn_band<true, true, 4>, (const void*)attn_band<true, true, 8>}}};
-    const void* fn = fns[a.kv_bf16 ? 1 : 0][fused ? 1 : 0][R > 4 ? 1 : 0];
+#define LUM_BAND_FNS(BF) {{(const void*)attn_band<BF, 0, 4>, (const void*)attn_band<BF, 0, 8>}, {(const void*)attn_band<BF, 1, 4>, (const void*)attn_band<BF, 1, 8>}, \
+                          {(const void*)attn_band<BF, 2, 4>, (const void*)attn_band<BF, 2, 8>}}
+    static const void* const fns[2][3][2] = {LUM_BAND_FNS(false), LUM_BAND_FNS(true)};
+#undef LUM_BAND_FNS
+    const void* fn = fns[a.kv_bf16 ? 1 : 0][fused ? (p.per_head ? 2 : 1) : 0][R > 4 ? 1 : 0];
     if (smem > 48 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         if (e != cudaSuccess) return e;
     }
     // splits: enough CTAs for the SMs, none shorter than half a tile of keys at full reach
-    const int reach = a.window > 0 && a.window < a.max_seq ? a.window : a.max_seq;
+    const int mask = a.chunk > 0 ? a.chunk : a.window, reach = mask > 0 && mask < a.max_seq ? mask : a.max_seq;
     static const int env_s = [] { const char* e = getenv("LUM_BAND_SPLITS"); return e ? atoi(e) : kBdMaxSplits; }();
     int S = 1;
-    while (S < env_s && S < kBdMaxSplits && (long long)p.n_kv * HB * rows * S * 2 <= sm_count && reach >= S * 2 * kBdTK / 2) S *= 2;
-    if (S > 8) {      // beyond the portable cluster size
+    while (S < env_s && S * p.maps < kBdMaxSplits && (long long)p.n_kv * p.maps * HB * rows * S * 2 <= sm_count && reach >= S * 2 * kBdTK / 2) S *= 2;
+    const int C = S * p.maps;
+    if (C > 8) {      // beyond the portable cluster size
         const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
         if (e != cudaSuccess) return e;
     }
     cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(S, p.n_kv * HB, rows); cfg.blockDim = dim3(256); cfg.dynamicSmemBytes = smem; cfg.stream = st;
+    cfg.gridDim = dim3(C, p.n_kv * HB, rows); cfg.blockDim = dim3(256); cfg.dynamicSmemBytes = smem; cfg.stream = st;
     cudaLaunchAttribute at[2];
     int na = 0;
     if (a.use_pdl && fused) { at[na].id = cudaLaunchAttributeProgrammaticStreamSerialization; at[na].val.programmaticStreamSerializationAllowed = 1; na++; }
-    if (S > 1) { at[na].id = cudaLaunchAttributeClusterDimension; at[na].val.clusterDim.x = S; at[na].val.clusterDim.y = 1; at[na].val.clusterDim.z = 1; na++; }
+    if (C > 1) { at[na].id = cudaLaunchAttributeClusterDimension; at[na].val.clusterDim.x = C; at[na].val.clusterDim.y = 1; at[na].val.clusterDim.z = 1; na++; }
     cfg.attrs = at; cfg.numAttrs = na;
     void* params[] = {&a, &S, &HB};
     return cudaLaunchKernelExC(&cfg, fn, params);

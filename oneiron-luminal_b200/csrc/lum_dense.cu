@@ -20,30 +20,30 @@ __device__ __forceinline__ float any_load(const void* p, uint32_t dtype, size_t 
     if (dtype == 1u) return __half2float(((const __half*)p)[i]);
     return ((const float*)p)[i];
 }
-__global__ void __launch_bounds__(256) chunked_pack(const void* src, uint32_t src_dtype, size_t rows, size_t cols, unsigned char* dst, int kind, int nt, size_t row0) {
+__global__ void __launch_bounds__(256) chunked_pack(const void* src, uint32_t src_dtype, size_t rows, size_t cols, unsigned char* dst, int kind, int nt, RowMap rm) {
     for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < rows * cols; i += (size_t)gridDim.x * 256) {
         const size_t n = i / cols, k = i - n * cols;
-        unsigned char* o = dst + chunked_off(kind, nt, row0 + n, k);
+        unsigned char* o = dst + chunked_off(kind, nt, row_map(rm, n), k);
         if (kind == WK_BF16 && src_dtype == WK_BF16) *(uint16_t*)o = ((const uint16_t*)src)[i];
         else if (kind == WK_BF16) *(__nv_bfloat16*)o = __float2bfloat16_rn(any_load(src, src_dtype, i));
         else *(float*)o = any_load(src, src_dtype, i);
     }
 }
-__global__ void __launch_bounds__(256) chunked_unpack(const unsigned char* src, int kind, int nt, size_t row0, size_t rows, size_t cols, float* f32, void* same) {
+__global__ void __launch_bounds__(256) chunked_unpack(const unsigned char* src, int kind, int nt, RowMap rm, size_t rows, size_t cols, float* f32, void* same) {
     for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < rows * cols; i += (size_t)gridDim.x * 256) {
         const size_t n = i / cols, k = i - n * cols;
-        const unsigned char* o = src + chunked_off(kind, nt, row0 + n, k);
+        const unsigned char* o = src + chunked_off(kind, nt, row_map(rm, n), k);
         if (same) { if (kind == WK_BF16) ((uint16_t*)same)[i] = *(const uint16_t*)o; else ((float*)same)[i] = *(const float*)o; }
         else f32[i] = kind == WK_BF16 ? bf16_bits_to_f32(*(const uint16_t*)o) : *(const float*)o;
     }
 }
 static unsigned blocks_for(size_t n) { const size_t b = (n + 255) / 256; return (unsigned)(b < 1 ? 1 : b > 16384 ? 16384 : b); }
-cudaError_t launch_chunked_pack(const void* src, uint32_t src_dtype, size_t rows, size_t cols, void* dst, int kind, int nt, size_t row0, cudaStream_t st) {
-    chunked_pack<<<blocks_for(rows * cols), 256, 0, st>>>(src, src_dtype, rows, cols, (unsigned char*)dst, kind, nt, row0);
+cudaError_t launch_chunked_pack(const void* src, uint32_t src_dtype, size_t rows, size_t cols, void* dst, int kind, int nt, RowMap rm, cudaStream_t st) {
+    chunked_pack<<<blocks_for(rows * cols), 256, 0, st>>>(src, src_dtype, rows, cols, (unsigned char*)dst, kind, nt, rm);
     return cudaGetLastError();
 }
-cudaError_t launch_chunked_unpack(const void* src, int kind, int nt, size_t row0, size_t rows, size_t cols, float* dst_f32, void* dst_same, cudaStream_t st) {
-    chunked_unpack<<<blocks_for(rows * cols), 256, 0, st>>>((const unsigned char*)src, kind, nt, row0, rows, cols, dst_f32, dst_same);
+cudaError_t launch_chunked_unpack(const void* src, int kind, int nt, RowMap rm, size_t rows, size_t cols, float* dst_f32, void* dst_same, cudaStream_t st) {
+    chunked_unpack<<<blocks_for(rows * cols), 256, 0, st>>>((const unsigned char*)src, kind, nt, rm, rows, cols, dst_f32, dst_same);
     return cudaGetLastError();
 }
 
@@ -77,6 +77,26 @@ __device__ __forceinline__ uint4 ld_stream(const uint4* p) {      // weights are
 }
 }  // namespace
 
+// the residual streams of column n take in a sublayer's output
+__device__ __forceinline__ void streams_take(const StreamArgs& h, int n, float y) {
+    float old[kMaxStreams];
+#pragma unroll
+    for (int s = 0; s < kMaxStreams; s++) old[s] = s < h.n ? h.x[(size_t)s * h.ldx + n] : 0.0f;
+    float u = 0.0f;
+    for (int t = 0; t < h.n; t++) {
+        float v = (h.out ? h.out[t] : 1.0f) * y;
+        if (h.mix) {
+#pragma unroll
+            for (int s = 0; s < kMaxStreams; s++) if (s < h.n) v = fmaf(h.mix[s * h.n + t], old[s], v);
+        } else {
+            v += h.x[(size_t)t * h.ldx + n];
+        }
+        h.x[(size_t)t * h.ldx + n] = v;
+        u = fmaf(h.next ? h.next[t] : 1.0f, v, u);
+    }
+    h.u[n] = u;
+}
+
 // grid = (row ranges) x (C CTAs of a cluster, each with a share of the chunks).  rl_max: row groups of the largest range.
 template <int KIND, bool CL>
 __global__ void __launch_bounds__(kDvThreads, 2) dense_gemv(const DenseArgs a, int C, int rl_max) {
@@ -84,7 +104,8 @@ __global__ void __launch_bounds__(kDvThreads, 2) dense_gemv(const DenseArgs a, i
     extern __shared__ __align__(16) float dv_smem[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int cr = CL ? (int)(blockIdx.x % C) : 0, cq = CL ? (int)(blockIdx.x / C) : (int)blockIdx.x, Q = CL ? (int)(gridDim.x / C) : (int)gridDim.x;
-    const int RG = a.nt / 8, rg0 = (int)((long long)cq * RG / Q), rg1 = (int)((long long)(cq + 1) * RG / Q);
+    const int RG = a.nt / 8, gs = a.pair ? 2 : 1;             // pairs of row groups stay together
+    const int rg0 = (int)((long long)cq * (RG / gs) / Q) * gs, rg1 = (int)((long long)(cq + 1) * (RG / gs) / Q) * gs;
     const int KC0 = a.seg[0].chunks, KC = KC0 + (a.nk > 1 ? a.seg[1].chunks : 0);
     const int c0 = (int)((long long)cr * KC / C), c1 = (int)((long long)(cr + 1) * KC / C);
     float* part = dv_smem;                                    // [8 warps][rl_max * 8]
@@ -127,7 +148,7 @@ __global__ void __launch_bounds__(kDvThreads, 2) dense_gemv(const DenseArgs a, i
         for (int i = tid; i < W; i += kDvThreads) { const float d = xs[i] - mean; s = fmaf(d, d, s); }
         const float inv = 1.0f / sqrtf(block_sum(s, red, tid, kDvThreads, 1) / (float)W + a.norm.eps);
         for (int i = tid; i < W; i += kDvThreads) {
-            float v = (xs[i] - mean) * inv * a.norm.gain[i];
+            float v = (xs[i] - mean) * inv * (a.norm.gain0 + a.norm.gain[i]);
             if (a.norm.bias) v += a.norm.bias[i];
             xs[i] = v;
         }
@@ -190,6 +211,16 @@ __global__ void __launch_bounds__(kDvThreads, 2) dense_gemv(const DenseArgs a, i
         cluster_arrive_release();
         cluster_wait_acquire();
     }
+    if (a.pair) {                                              // (no cluster) gate rows i, up rows i + 8
+        for (int j = tid; j < n_rows / 2; j += kDvThreads) {
+            const int i = (j >> 3) * 16 + (j & 7);
+            float g = 0.0f, u = 0.0f;
+#pragma unroll
+            for (int w = 0; w < kDvWarps; w++) { g += part[(size_t)w * rl_max * 8 + i]; u += part[(size_t)w * rl_max * 8 + i + 8]; }
+            a.act_x[rg0 * 4 + j] = clamped_gate(g, u, a.limit);
+        }
+        return;
+    }
     float sp = 0.0f, sq = 0.0f;
     if (a.act_row0 < a.nt) { sp = softplus(a.act_par[0]); sq = softplus(a.act_par[1]); }
     ArgBest best{-INFINITY, -1};
@@ -203,11 +234,14 @@ __global__ void __launch_bounds__(kDvThreads, 2) dense_gemv(const DenseArgs a, i
             for (int w = 0; w < kDvWarps; w++) v += part[(size_t)w * rl_max * 8 + i];
         }
         const int n = rg0 * 8 + i;
+        if (a.bias) v += a.bias[n];
         if (n >= a.act_row0) a.act_x[n - a.act_row0] = xielu(v, sp, sq);
         else if (n < a.n_real) {
-            if (a.epi == DENSE_RESID) a.y[n] = a.y[n] + a.mult * v;
+            if (a.epi == DENSE_STREAMS) streams_take(a.hc, n, v);
+            else if (a.epi == DENSE_RESID) a.y[n] = a.y[n] + a.mult * v;
             else {
                 v *= a.mult;
+                if (n < a.gelu_rows) v = gelu_tanh(v);
                 a.y[n] = v;
                 if (a.epi == DENSE_ARGMAX) argbest_take(best, v, n);
             }
@@ -231,21 +265,24 @@ __global__ void __launch_bounds__(kDvThreads, 2) dense_gemv(const DenseArgs a, i
 
 cudaError_t launch_dense_gemv(const DenseArgs& a_in, int sm_count, cudaStream_t st) {
     DenseArgs a = a_in;
-    if (a.nk < 1 || a.nk > 2 || a.nt <= 0 || a.nt % 8 || (a.kind != WK_BF16 && a.kind != WK_F32)) return cudaErrorInvalidValue;
+    if (a.nk < 1 || a.nk > 2 || a.nt <= 0 || a.nt % 8 || a.grp_rows || (a.kind != WK_BF16 && a.kind != WK_F32)) return cudaErrorInvalidValue;
+    if (a.epi == DENSE_STREAMS && (a.hc.n < 1 || a.hc.n > kMaxStreams)) return cudaErrorInvalidValue;
     if (a.norm.mode != NORM_NONE && (a.nk != 1 || a.norm.width > a.seg[0].chunks * chunk_elems(a.kind))) return cudaErrorInvalidValue;
     const int RG = a.nt / 8, KC = a.seg[0].chunks + (a.nk > 1 ? a.seg[1].chunks : 0);
     // A long K: split over a cluster of two, so that a CTA has whole shares of both K and the rows and loads half of the vector
     // (measured on 4096 rows x K 25600: 39 us; a cluster of 8: 64 us; a whole decode step with 1 / 2 / 4 / 8: 1118 / 935 / 1124 / 1149 us)
     int C = 1;
-    if (a.norm.mode == NORM_NONE && a.epi != DENSE_ARGMAX && KC >= 32) C = 2;
+    if (a.norm.mode == NORM_NONE && a.epi != DENSE_ARGMAX && !a.pair && KC >= 32) C = 2;
     static const int env_c = [] { const char* e = getenv("LUM_DENSE_CLUSTER"); return e ? atoi(e) : 0; }();
-    if ((env_c == 1 || env_c == 2 || env_c == 4 || env_c == 8) && a.norm.mode == NORM_NONE && a.epi != DENSE_ARGMAX) C = env_c;
+    if ((env_c == 1 || env_c == 2 || env_c == 4 || env_c == 8) && a.norm.mode == NORM_NONE && a.epi != DENSE_ARGMAX && !a.pair) C = env_c;
     int Q = 2 * sm_count / C;
     if (a.epi == DENSE_ARGMAX && Q > kArgmaxSlots) Q = kArgmaxSlots;
     // few rows: no more ranges than blocks of row groups a warp carries anyway would leave half of a warp's loads empty
-    if (Q > RG) Q = RG;
+    const int gs = a.pair ? 2 : 1;
+    if (RG % gs || (a.pair && (a.epi != DENSE_STORE || C != 1))) return cudaErrorInvalidValue;
+    if (Q > RG / gs) Q = RG / gs;
     if (Q < 1) Q = 1;
-    const int rl = (RG + Q - 1) / Q, cl = (KC + C - 1) / C;
+    const int rl = (RG / gs + Q - 1) / Q * gs, cl = (KC + C - 1) / C;
     const size_t smem = ((size_t)kDvWarps * rl * 8 + 32 + (size_t)cl * chunk_elems(a.kind)) * 4;
     if (smem > 220 * 1024) return cudaErrorInvalidValue;
     const void* fn = a.kind == WK_BF16 ? (C > 1 ? (const void*)dense_gemv<WK_BF16, true> : (const void*)dense_gemv<WK_BF16, false>)
@@ -267,8 +304,35 @@ cudaError_t launch_dense_gemv(const DenseArgs& a_in, int sm_count, cudaStream_t 
 }
 
 // ------------------------------------------------------------------------------------------------ many rows
+// 16 finished sums of row m: 8 gate rows and their 8 up rows, container rows n .. n + 15.
+__device__ __forceinline__ void rows_epilogue_pair(const DenseArgs& a, int m, int n, const float (&g)[8], const float (&u)[8]) {
+    float t[8];
+#pragma unroll
+    for (int i = 0; i < 8; i++) t[i] = clamped_gate(g[i], u[i], a.limit);
+    unsigned char* o = (unsigned char*)a.act.p + row_operand_off(a.kind, a.act.chunks, m, n >> 1);
+    if (a.kind == WK_BF16) {
+        uint32_t w[4];
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const __nv_bfloat162 b = __floats2bfloat162_rn(t[2 * i], t[2 * i + 1]);
+            w[i] = *(const uint32_t*)&b;
+        }
+        *(uint4*)o = make_uint4(w[0], w[1], w[2], w[3]);
+    } else {
+        ((float4*)o)[0] = make_float4(t[0], t[1], t[2], t[3]);
+        ((float4*)o)[1] = make_float4(t[4], t[5], t[6], t[7]);
+    }
+}
 // Eight finished sums of row m, container rows n .. n + 7.
-__device__ __forceinline__ void rows_epilogue8(const DenseArgs& a, int m, int n, const float (&v)[8], float sp, float sq) {
+__device__ __forceinline__ void rows_epilogue8(const DenseArgs& a, int m, int n, float (&v)[8], float sp, float sq) {
+    if (a.bias) {
+#pragma unroll
+        for (int i = 0; i < 8; i++) v[i] += a.bias[n + i];
+    }
+    if (n < a.gelu_rows) {                                    // (a multiple of 8; stored with factor 1)
+#pragma unroll
+        for (int i = 0; i < 8; i++) v[i] = gelu_tanh(v[i]);
+    }
     if (n >= a.act_row0) {
         float t[8];
 #pragma unroll
@@ -345,7 +409,9 @@ __global__ void __launch_bounds__(kDmThreads, 1) dense_gemm_tc(const DenseArgs a
     tc_fence_after_sync();
     const uint32_t tmem = *(volatile uint32_t*)(dm_smem + stages * stage_bytes + 296);
 
-    const int mt = (a.M + 127) / 128, ntile = (a.nt + TN - 1) / TN, n_tiles = mt * ntile;
+    // column tiles: a tile's rows of the container belong to one group
+    const int grp = a.grp_rows ? a.grp_rows : a.nt, tpg = (grp + TN - 1) / TN;
+    const int mt = (a.M + 127) / 128, ntile = tpg * (a.nt / grp), n_tiles = mt * ntile;
     const int KC0 = a.seg[0].chunks, KC = KC0 + (a.nk > 1 ? a.seg[1].chunks : 0);
 
     if (warp == 0) {
@@ -353,8 +419,8 @@ __global__ void __launch_bounds__(kDmThreads, 1) dense_gemm_tc(const DenseArgs a
             uint32_t it = 0;
             bool ok = true;
             for (int t = blockIdx.x; t < n_tiles && ok; t += gridDim.x) {
-                const int tm = t % mt, n0 = (t / mt) * TN;
-                const int rows = min(128, ((a.M - tm * 128) + 7) & ~7), wrows = min(TN, a.nt - n0);
+                const int tm = t % mt, gi = (t / mt) / tpg, ng = (t / mt - gi * tpg) * TN, n0 = gi * grp + ng, ca = gi * a.grp_chunks;
+                const int rows = min(128, ((a.M - tm * 128) + 7) & ~7), wrows = min(TN, grp - ng);
                 const uint32_t ab = (uint32_t)rows * 128, bb = (uint32_t)wrows * 128;
                 for (int c = 0; c < KC; c++, it++) {
                     const int s = it % stages;
@@ -363,7 +429,7 @@ __global__ void __launch_bounds__(kDmThreads, 1) dense_gemm_tc(const DenseArgs a
                     const bool second = c >= KC0;
                     const int cc = second ? c - KC0 : c;
                     const DenseK& g = second ? a.seg[1] : a.seg[0];
-                    bulk_g2s(s_base + s * stage_bytes, (const unsigned char*)g.a + ((size_t)tm * g.chunks + cc) * kDmABytes, ab, full(s));
+                    bulk_g2s(s_base + s * stage_bytes, (const unsigned char*)g.a + ((size_t)tm * (g.a_chunks ? g.a_chunks : g.chunks) + ca + cc) * kDmABytes, ab, full(s));
                     bulk_g2s(s_base + s * stage_bytes + kDmABytes, (const unsigned char*)g.w + (size_t)cc * a.nt * 128 + (size_t)n0 * 128, bb, full(s));
                 }
             }
@@ -409,7 +475,7 @@ __global__ void __launch_bounds__(kDmThreads, 1) dense_gemm_tc(const DenseArgs a
         if (a.act_row0 < a.nt) { sp = softplus(a.act_par[0]); sq = softplus(a.act_par[1]); }
         int ti = 0;
         for (int t = blockIdx.x; t < n_tiles; t += gridDim.x, ti++) {
-            const int b = ti & 1, tm = t % mt, n0 = (t / mt) * TN;
+            const int b = ti & 1, tm = t % mt, gi = (t / mt) / tpg, n0 = gi * grp + (t / mt - gi * tpg) * TN, n1 = (gi + 1) * grp;
             int ok = mbar_wait_abortable(acc_full(b), (ti >> 1) & 1, abort) ? 1 : 0;
             if (!__all_sync(0xffffffffu, ok)) { *abort = 1; if (lane == 0) atomicOr(a.status, LUM_ST_WAIT_TMEM); break; }
             tc_fence_after_sync();
@@ -423,10 +489,22 @@ __global__ void __launch_bounds__(kDmThreads, 1) dense_gemm_tc(const DenseArgs a
                 tmem_ld_wait();
                 if (cb + 32 >= TN) { tc_fence_before_sync(); mbar_arrive(acc_empty(b)); }     // the last columns are in registers
                 if (m < a.M) {
+                    if (a.pair) {
+#pragma unroll
+                        for (int h = 0; h < 2; h++) {
+                            const int n = n0 + cb + h * 16;
+                            if (n < n1) {
+                                float g[8], u[8];
+#pragma unroll
+                                for (int i = 0; i < 8; i++) { g[i] = __uint_as_float(h ? v1[i] : v0[i]); u[i] = __uint_as_float(h ? v1[8 + i] : v0[8 + i]); }
+                                rows_epilogue_pair(a, m, n, g, u);
+                            }
+                        }
+                    } else
 #pragma unroll
                     for (int h = 0; h < 4; h++) {
                         const int n = n0 + cb + h * 8;
-                        if (n < a.nt) {
+                        if (n < n1) {
                             float f[8];
 #pragma unroll
                             for (int i = 0; i < 8; i++) f[i] = __uint_as_float(h < 2 ? v0[(h & 1) * 8 + i] : v1[(h & 1) * 8 + i]);
@@ -446,7 +524,8 @@ __global__ void __launch_bounds__(kDmThreads, 1) dense_gemm_tc(const DenseArgs a
 __global__ void __launch_bounds__(256) dense_gemm_f32(const DenseArgs a) {
     __shared__ float As[32][68], Bs[32][68];
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
-    const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+    const int grp = a.grp_rows ? a.grp_rows : a.nt, tpg = (grp + 63) / 64, gi = blockIdx.x / tpg;
+    const int m0 = blockIdx.y * 64, n0 = gi * grp + (blockIdx.x - gi * tpg) * 64, n1 = (gi + 1) * grp, ka = gi * a.grp_chunks * 32;
     float acc[4][4];
 #pragma unroll
     for (int i = 0; i < 4; i++)
@@ -454,7 +533,7 @@ __global__ void __launch_bounds__(256) dense_gemm_f32(const DenseArgs a) {
         for (int j = 0; j < 4; j++) acc[i][j] = 0.0f;
     for (int s = 0; s < a.nk; s++) {
         const DenseK& g = a.seg[s];
-        const int lda = g.chunks * 32;
+        const int lda = (g.a_chunks ? g.a_chunks : g.chunks) * 32;
         for (int c = 0; c < g.chunks; c++) {
 #pragma unroll
             for (int i = 0; i < 2; i++) {
@@ -462,13 +541,13 @@ __global__ void __launch_bounds__(256) dense_gemm_f32(const DenseArgs a) {
                 {
                     const int r = idx >> 3, k4 = idx & 7, m = m0 + r;
                     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-                    if (m < a.M) v = *(const float4*)((const float*)g.a + (size_t)m * lda + c * 32 + k4 * 4);
+                    if (m < a.M) v = *(const float4*)((const float*)g.a + (size_t)m * lda + ka + c * 32 + k4 * 4);
                     As[k4 * 4][r] = v.x; As[k4 * 4 + 1][r] = v.y; As[k4 * 4 + 2][r] = v.z; As[k4 * 4 + 3][r] = v.w;
                 }
                 {
                     const int rg = idx >> 6, k4 = (idx >> 3) & 7, r = rg * 8 + (idx & 7), n = n0 + r;
                     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-                    if (n < a.nt) v = *(const float4*)((const unsigned char*)g.w + chunked_off(WK_F32, a.nt, n, (size_t)c * 32 + k4 * 4));
+                    if (n < n1) v = *(const float4*)((const unsigned char*)g.w + chunked_off(WK_F32, a.nt, n, (size_t)c * 32 + k4 * 4));
                     Bs[k4 * 4][r] = v.x; Bs[k4 * 4 + 1][r] = v.y; Bs[k4 * 4 + 2][r] = v.z; Bs[k4 * 4 + 3][r] = v.w;
                 }
             }
@@ -496,7 +575,14 @@ __global__ void __launch_bounds__(256) dense_gemm_f32(const DenseArgs a) {
                 for (int j = 0; j < 4; j++) As[(ty & 7) * 4 + i][tx * 4 + j] = acc[i][j];
         __syncthreads();
         const int r = tid >> 3, n = n0 + (tid & 7) * 8, m = m0 + half * 32 + r;
-        if (m < a.M && n < a.nt) {
+        if (a.pair) {
+            if (m < a.M && n < n1 && (tid & 1) == 0) {
+                float g[8], u[8];
+#pragma unroll
+                for (int i = 0; i < 8; i++) { g[i] = As[r][(tid & 7) * 8 + i]; u[i] = As[r][(tid & 7) * 8 + 8 + i]; }
+                rows_epilogue_pair(a, m, n, g, u);
+            }
+        } else if (m < a.M && n < n1) {
             float f[8];
 #pragma unroll
             for (int i = 0; i < 8; i++) f[i] = As[r][(tid & 7) * 8 + i];
@@ -508,9 +594,11 @@ __global__ void __launch_bounds__(256) dense_gemm_f32(const DenseArgs a) {
 
 cudaError_t launch_dense_gemm(const DenseArgs& a_in, int sm_count, cudaStream_t st) {
     DenseArgs a = a_in;
-    if (a.nk < 1 || a.nk > 2 || a.nt <= 0 || a.nt % 8 || a.M <= 0 || a.epi == DENSE_ARGMAX || (a.kind != WK_BF16 && a.kind != WK_F32)) return cudaErrorInvalidValue;
+    if (a.nk < 1 || a.nk > 2 || a.nt <= 0 || a.nt % 8 || a.M <= 0 || a.epi == DENSE_ARGMAX || a.epi == DENSE_STREAMS || (a.kind != WK_BF16 && a.kind != WK_F32)) return cudaErrorInvalidValue;
+    if ((a.pair && a.nt % 16) || (a.grp_rows && (a.grp_rows % 8 || a.nt % a.grp_rows))) return cudaErrorInvalidValue;
+    const int grp = a.grp_rows ? a.grp_rows : a.nt, groups = a.nt / grp;
     if (a.kind == WK_F32) {
-        dense_gemm_f32<<<dim3((a.nt + 63) / 64, (a.M + 63) / 64), 256, 0, st>>>(a);
+        dense_gemm_f32<<<dim3((grp + 63) / 64 * groups, (a.M + 63) / 64), 256, 0, st>>>(a);
         return cudaGetLastError();
     }
     // tile width: the fewest (rounds over the SMs) x (time of a tile); a narrow tile does not fill the tensor pipe.  (With few rows a chunk
@@ -520,7 +608,7 @@ cudaError_t launch_dense_gemm(const DenseArgs& a_in, int sm_count, cudaStream_t 
     int TN = 256;
     double best = 1e30;
     for (int tn = 256; tn >= 64; tn >>= 1) {
-        const long long tiles = (long long)mt * ((a.nt + tn - 1) / tn);
+        const long long tiles = (long long)mt * ((grp + tn - 1) / tn) * groups;
         const double cost = (double)((tiles + sm_count - 1) / sm_count) * (tn + (tn < 128 ? 64 : 48));
         if (cost < best) { best = cost; TN = tn; }
     }
@@ -534,7 +622,7 @@ cudaError_t launch_dense_gemm(const DenseArgs& a_in, int sm_count, cudaStream_t 
         if (e != cudaSuccess) return e;
         attr_set = true;
     }
-    const int n_tiles = mt * ((a.nt + TN - 1) / TN);
+    const int n_tiles = mt * ((grp + TN - 1) / TN) * groups;
     dense_gemm_tc<<<n_tiles < sm_count ? n_tiles : sm_count, kDmThreads, smem, st>>>(a, TN, stages);
     return cudaGetLastError();
 }

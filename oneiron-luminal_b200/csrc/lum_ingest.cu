@@ -393,13 +393,19 @@ static const SlotName kBlockLayerNames[] = {
     {LUM_S_ATTN_NORM, "norm1"}, {LUM_S_ATTN_NORM_BIAS, "norm1.b"}, {LUM_S_Q, "mix.q"}, {LUM_S_K, "mix.k"}, {LUM_S_V, "mix.v"}, {LUM_S_O, "mix.o"},
     {LUM_S_Q_NORM, "mix.q.norm"}, {LUM_S_K_NORM, "mix.k.norm"}, {LUM_S_V_MIX, "mix.vmix"}, {LUM_S_TEMP, "mix.temp"}, {LUM_S_DIST_R1, "mix.r1"},
     {LUM_S_DIST_R2, "mix.r2"}, {LUM_S_UP, "mlp.up"}, {LUM_S_DOWN, "mlp.down"}, {LUM_S_ACT, "mlp.act"},
+    {LUM_S_MLP_NORM, "norm2"}, {LUM_S_GATE, "mlp.gate"}, {LUM_S_Q_BIAS, "mix.q.b"}, {LUM_S_K_BIAS, "mix.k.b"}, {LUM_S_V_BIAS, "mix.v.b"},
+    {LUM_S_Q_CONV, "mix.q.conv"}, {LUM_S_K_CONV, "mix.k.conv"}, {LUM_S_V_CONV, "mix.v.conv"}, {LUM_S_LQ1, "mix.lq1"}, {LUM_S_LK1, "mix.lk1"},
+    {LUM_S_LQ2, "mix.lq2"}, {LUM_S_LK2, "mix.lk2"}, {LUM_S_HC1_IN, "hc1.in"}, {LUM_S_HC1_OUT, "hc1.out"}, {LUM_S_HC1_MIX, "hc1.mix"},
+    {LUM_S_HC2_IN, "hc2.in"}, {LUM_S_HC2_OUT, "hc2.out"}, {LUM_S_HC2_MIX, "hc2.mix"}, {LUM_S_REC_Y, "mix.y"}, {LUM_S_REC_Y_BIAS, "mix.y.b"},
+    {LUM_S_REC_X, "mix.x"}, {LUM_S_REC_X_BIAS, "mix.x.b"}, {LUM_S_REC_CONV, "mix.conv"}, {LUM_S_REC_CONV_BIAS, "mix.conv.b"},
+    {LUM_S_REC_RA, "mix.ra"}, {LUM_S_REC_RA_BIAS, "mix.ra.b"}, {LUM_S_REC_RI, "mix.ri"}, {LUM_S_REC_RI_BIAS, "mix.ri.b"}, {LUM_S_REC_LAM, "mix.lam"},
 };
 static const SlotName kBlockTopNames[] = {
     {LUM_S_EMBED, "embed"}, {LUM_S_FINAL_NORM, "final.norm"}, {LUM_S_FINAL_NORM_BIAS, "final.norm.b"}, {LUM_S_LM_HEAD, "head"},
 };
 struct LabelStyle { const SlotName *top, *layer; size_t n_top, n_layer; const char* prefix; };
 static LabelStyle label_style(int style) {
-    if (style == 1) return {kBlockTopNames, kBlockLayerNames, sizeof kBlockTopNames / sizeof *kBlockTopNames, sizeof kBlockLayerNames / sizeof *kBlockLayerNames, "l"};
+    if (style != 0) return {kBlockTopNames, kBlockLayerNames, sizeof kBlockTopNames / sizeof *kBlockTopNames, sizeof kBlockLayerNames / sizeof *kBlockLayerNames, "l"};
     return {kTopNames, kLayerNames, sizeof kTopNames / sizeof *kTopNames, sizeof kLayerNames / sizeof *kLayerNames, "model.layers."};
 }
 
@@ -457,7 +463,7 @@ static int store_weight(lum_rt* rt, int slot, int layer, const void* src, size_t
         if (e != cudaSuccess) return lum_internal_fail(rt, LUM_E_NOMEM, "set_weight: staging buffer");
         e = cudaMemcpy2DAsync(stage, row_bytes, from, src_pitch, row_bytes, t.rows, cudaMemcpyDefault, t.stream);
         if (t.kc == kLayoutChunked) {
-            if (e == cudaSuccess) e = launch_chunked_pack(stage, dtype, t.rows, t.cols, t.w, t.kind, t.nt, t.crow0, t.stream);
+            if (e == cudaSuccess) e = launch_chunked_pack(stage, dtype, t.rows, t.cols, t.w, t.kind, t.nt, t.rm, t.stream);
         } else if (t.kind == WK_Q8) {
             int8_t* pq = (int8_t*)t.w;
             __half* ps = t.s;
@@ -507,7 +513,7 @@ static int fetch_weight(lum_rt* rt, const WeightView& t, std::vector<uint8_t>* o
         out->resize(n * (t.kind == WK_BF16 ? 2 : 4));
         void* rows = nullptr;
         if (e == cudaSuccess) e = cudaMalloc(&rows, out->size() + 64);
-        if (e == cudaSuccess) e = launch_chunked_unpack(t.w, t.kind, t.nt, t.crow0, t.rows, t.cols, nullptr, rows, t.stream);
+        if (e == cudaSuccess) e = launch_chunked_unpack(t.w, t.kind, t.nt, t.rm, t.rows, t.cols, nullptr, rows, t.stream);
         if (e == cudaSuccess) e = cudaMemcpyAsync(out->data(), rows, out->size(), cudaMemcpyDeviceToHost, t.stream);
         const cudaError_t es = cudaStreamSynchronize(t.stream);
         if (e == cudaSuccess) e = es;

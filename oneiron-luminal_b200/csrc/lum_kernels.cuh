@@ -207,6 +207,14 @@ cudaError_t launch_q8_pack_units(const int8_t* q, const __half* s, int rows, int
 cudaError_t launch_q8_unpack_wire(const uint8_t* blocks, int8_t* q, __half* s, size_t n_blocks, cudaStream_t st);
 cudaError_t launch_q8_quantize(const void* src, uint32_t dtype, size_t n_blocks, int8_t* q, __half* s, cudaStream_t st);   // f32 / f16 / bf16 -> planes
 
+// Rows of a weight tensor in a container it shares with others (chunked layout, lum_dense.cuh): row n of the tensor is row
+// row0 + (n / grp) * stride + (n % grp) / 8 * 8 * step + n % grp % 8 — step 2 leaves room for another tensor's groups of 8 rows in between,
+// grp / stride place blocks of rows apart (grp 0: one block).
+struct RowMap { size_t row0; size_t grp = 0, stride = 0; int step = 1; };
+__host__ __device__ inline size_t row_map(const RowMap& m, size_t n) {
+    const size_t b = m.grp ? n / m.grp : 0, r = m.grp ? n - b * m.grp : n;
+    return m.row0 + b * m.stride + (r / 8) * 8 * m.step + r % 8;
+}
 // What the weight-ingest code needs to know about one tensor slot of a loaded model (this rank's shard).
 struct WeightView {
     void* w; __half* s;                  // device storage: quants / values, Q8_0 plane scales (null when packed)
@@ -214,7 +222,7 @@ struct WeightView {
     size_t rows, cols, kdev;             // the shard; kdev = columns of the device layout (>= cols, zero columns beyond)
     size_t row0, col0, full_rows, full_cols;
     int device; cudaStream_t stream;
-    int nt; size_t crow0;                // chunked layout (kc == kLayoutChunked, lum_dense.cuh): padded rows of the container, first row in it
+    int nt; RowMap rm;                   // chunked layout (kc == kLayoutChunked, lum_dense.cuh): padded rows of the container, the tensor's rows in it
 };
 cudaError_t launch_q8_dequant(const int8_t* q, const __half* s, float* out, size_t n_elems, cudaStream_t st);
 cudaError_t launch_q8_dequant_rows(const void* w, const __half* s, int K, int kc, size_t row0, size_t n_rows, float* out, cudaStream_t st, int valid_cols = 0);

@@ -1,0 +1,339 @@
+// Gated linear recurrences behind a short convolution, and the convolution's memory.
+//
+//   conv_tail     after a pass of many rows of one sequence: the last projected values of every channel go to the sequence's ring
+//   recur_step    rows of different sequences (a decode step: one): convolution, the gates' block-diagonal products, the recurrence and
+//                 the multiplication with the other branch in one kernel
+//   recur_conv    many rows of one sequence: the convolved values, also as the operand of the gates' product (dense_gemm, one group
+//                 per block; two bf16 terms, so that the gates are as exact as their weights)
+//   recur_scan    ... and the recurrence over those rows: the time axis is cut into pieces whose (decay, sum) pairs are combined by a
+//                 scan, tile by tile
+// Everything is computed in f32; the state is f32.  It starts at zero at position 0, whatever the slot held before.
+#include <cuda_bf16.h>
+
+#include "lum_gemv_dev.cuh"
+#include "lum_dense.cuh"
+
+namespace lum {
+
+namespace {
+// sqrt(1 - a^2) for ln a = half_q / 2, exact also where a is close to 1 (half_q = 2 ln a <= 0)
+__device__ __forceinline__ float decay_input(float q, float a) {
+    float t = 1.0f - a * a;
+    if (q > -0.25f) {                                          // 1 - e^q = -q (1 + q/2 (1 + q/3 (1 + ...)))
+        float s = fmaf(q, 1.0f / 7.0f, 1.0f);
+        s = fmaf(q * (1.0f / 6.0f), s, 1.0f);
+        s = fmaf(q * (1.0f / 5.0f), s, 1.0f);
+        s = fmaf(q * (1.0f / 4.0f), s, 1.0f);
+        s = fmaf(q * (1.0f / 3.0f), s, 1.0f);
+        s = fmaf(q * (1.0f / 2.0f), s, 1.0f);
+        t = -q * s;
+    }
+    return sqrtf(fmaxf(t, 0.0f));
+}
+__device__ __forceinline__ float softplus_exact(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
+// decay a and input b of one step; sp = softplus(lam), r and i before their sigmoids
+__device__ __forceinline__ void recur_gate(float r, float i, float u, float sp, float& a, float& b) {
+    const float la = -8.0f * sigmoid(r) * sp;
+    a = expf(la);
+    b = decay_input(2.0f * la, a) * sigmoid(i) * u;
+}
+__device__ __forceinline__ uint32_t pack_bf16(float x, float y) {
+    const __nv_bfloat162 b = __floats2bfloat162_rn(x, y);
+    return *(const uint32_t*)&b;
+}
+}  // namespace
+
+// ------------------------------------------------------------------------------------------------ the convolution's memory
+__global__ void __launch_bounds__(256) conv_tail(const ConvTailArgs a) {
+    const int m = a.M - 1 - (int)blockIdx.y, c = blockIdx.x * 256 + threadIdx.x;
+    if (m < 0 || c >= a.n_ch) return;
+    a.conv.ring[((size_t)a.seq * a.conv.taps + a.row_pos[m] % a.conv.taps) * a.conv.ch + c] = a.src[(size_t)m * a.ld + c];
+}
+cudaError_t launch_conv_tail(const ConvTailArgs& a, cudaStream_t st) {
+    if (a.conv.taps <= 0) return cudaSuccess;
+    if (a.M <= 0 || a.n_ch <= 0) return cudaErrorInvalidValue;
+    conv_tail<<<dim3((a.n_ch + 255) / 256, a.conv.taps < a.M ? a.conv.taps : a.M), 256, 0, st>>>(a);
+    return cudaGetLastError();
+}
+
+// ------------------------------------------------------------------------------------------------ one step
+// CTA = (block of the gates, 4 groups of 8 channels: a warp each) x 4 rows.  Lanes are 4 groups of K x 8 channels; the first chunks' weights
+// are asked for before the projection's results are waited for.
+namespace { constexpr int kRsRows = 4, kRsWarps = 4, kRsPre = 4; }
+template <int KIND>
+__global__ void __launch_bounds__(kRsWarps * 32) recur_step(const RecurArgs a) {
+    constexpr int E = KIND == WK_BF16 ? 8 : 4, CK = KIND == WK_BF16 ? 64 : 32;
+    extern __shared__ __align__(16) float rs_u[];             // [rows][kc * CK]
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int rgb = a.bwp / 8, per = (rgb + kRsWarps - 1) / kRsWarps;
+    const int blk = blockIdx.x / per, part = blockIdx.x - blk * per, pg = part * kRsWarps + warp;      // pg: this warp's group of 8 channels
+    const int m0 = blockIdx.y * kRsRows, nr = min(kRsRows, a.M - m0), KL = a.kc * CK;
+    const bool has = pg < rgb;
+    const int rg_r = blk * 2 * rgb + pg, rg_i = rg_r + rgb, RG = a.nt / 8;
+    auto weights = [&](int c, uint4 (&w)[4]) {
+        const uint4* base = (const uint4*)a.w_gate + (size_t)c * RG * 64 + lane;
+        w[0] = __ldg(base + (size_t)rg_r * 64); w[1] = __ldg(base + (size_t)rg_r * 64 + 32);
+        w[2] = __ldg(base + (size_t)rg_i * 64); w[3] = __ldg(base + (size_t)rg_i * 64 + 32);
+    };
+    uint4 pre[kRsPre][4];
+    pdl_launch_dependents();
+    if (has) {
+#pragma unroll
+        for (int c = 0; c < kRsPre; c++) if (c < a.kc) weights(c, pre[c]);
+    }
+    pdl_grid_wait();
+
+    int pos[kRsRows], seq[kRsRows];
+    bool bad = false;
+#pragma unroll
+    for (int r = 0; r < kRsRows; r++) {
+        pos[r] = r < nr ? (a.step ? a.step->pos : a.row_pos[m0 + r]) : 0;
+        seq[r] = r < nr && a.row_seq ? a.row_seq[m0 + r] : a.seq0;
+        bad = bad || pos[r] < 0 || pos[r] >= a.max_seq || seq[r] < 0 || seq[r] >= a.max_batch;
+    }
+    if (bad) {
+        if (tid == 0) atomicOr(a.status, LUM_ST_BAD_POS);
+        return;
+    }
+    // ---- the block's inputs
+#pragma unroll
+    for (int r = 0; r < kRsRows; r++) {
+        if (r >= nr) continue;
+        const float* src = a.yx + (size_t)(m0 + r) * a.ld + a.x_off;
+        float* ring = a.conv.ring + (size_t)seq[r] * a.conv.taps * a.conv.ch;
+        for (int k = tid; k < KL; k += kRsWarps * 32) {
+            float u = 0.0f;
+            if (k < a.bw) {
+                const int c = blk * a.bw + k;
+                u = conv_at(a.conv, ring, src, 0, 0, pos[r], c) + (a.conv_b ? a.conv_b[c] : 0.0f);
+                // (the row of the ring that no step of this position reads)
+                if (part == 0 && a.conv.taps > 0) ring[(size_t)(pos[r] % a.conv.taps) * a.conv.ch + c] = src[c];
+            }
+            rs_u[r * KL + k] = u;
+        }
+    }
+    __syncthreads();
+    if (!has) return;
+    // ---- gates
+    float ar[kRsRows], ai[kRsRows];
+#pragma unroll
+    for (int r = 0; r < kRsRows; r++) ar[r] = ai[r] = 0.0f;
+    const int grp = lane >> 3;
+    auto take = [&](int c, const uint4 (&w)[4]) {
+#pragma unroll
+        for (int h = 0; h < 2; h++) {
+            float wr[E], wi[E];
+            const uint32_t rv[4] = {w[h].x, w[h].y, w[h].z, w[h].w}, iv[4] = {w[2 + h].x, w[2 + h].y, w[2 + h].z, w[2 + h].w};
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                if (KIND == WK_BF16) {
+                    wr[(2 * i) % E] = __uint_as_float(rv[i] << 16); wr[(2 * i + 1) % E] = __uint_as_float(rv[i] & 0xffff0000u);
+                    wi[(2 * i) % E] = __uint_as_float(iv[i] << 16); wi[(2 * i + 1) % E] = __uint_as_float(iv[i] & 0xffff0000u);
+                } else {
+                    wr[i % E] = __uint_as_float(rv[i]); wi[i % E] = __uint_as_float(iv[i]);
+                }
+            }
+#pragma unroll
+            for (int r = 0; r < kRsRows; r++) {
+                if (r < nr) {
+                    const float* x = rs_u + r * KL + c * CK + h * 4 * E + grp * E;
+#pragma unroll
+                    for (int i = 0; i < E; i += 4) {
+                        const float4 v = *(const float4*)(x + i);
+                        ar[r] = fmaf(wr[i], v.x, ar[r]); ar[r] = fmaf(wr[i + 1], v.y, ar[r]); ar[r] = fmaf(wr[i + 2], v.z, ar[r]); ar[r] = fmaf(wr[i + 3], v.w, ar[r]);
+                        ai[r] = fmaf(wi[i], v.x, ai[r]); ai[r] = fmaf(wi[i + 1], v.y, ai[r]); ai[r] = fmaf(wi[i + 2], v.z, ai[r]); ai[r] = fmaf(wi[i + 3], v.w, ai[r]);
+                    }
+                }
+            }
+        }
+    };
+#pragma unroll
+    for (int c = 0; c < kRsPre; c++) if (c < a.kc) take(c, pre[c]);
+    for (int c = kRsPre; c < a.kc; c++) {
+        uint4 w[4];
+        weights(c, w);
+        take(c, w);
+    }
+    // ---- every lane has the sums of channel lane % 8 after two shuffles; lane group r finishes row r
+    float vr = 0.0f, vi = 0.0f;
+    int my_pos = 0, my_seq = 0;
+#pragma unroll
+    for (int r = 0; r < kRsRows; r++) {
+        ar[r] += __shfl_xor_sync(0xffffffffu, ar[r], 8); ar[r] += __shfl_xor_sync(0xffffffffu, ar[r], 16);
+        ai[r] += __shfl_xor_sync(0xffffffffu, ai[r], 8); ai[r] += __shfl_xor_sync(0xffffffffu, ai[r], 16);
+        if (grp == r) { vr = ar[r]; vi = ai[r]; my_pos = pos[r]; my_seq = seq[r]; }
+    }
+    const int kb = pg * 8 + (lane & 7), c = blk * a.bw + kb, m = m0 + grp;
+    if (grp >= nr || kb >= a.bw) return;
+    float da, db;
+    recur_gate(vr + a.r_b[c], vi + a.i_b[c], rs_u[grp * KL + kb], softplus_exact(a.lam[c]), da, db);
+    float* S = a.state + (size_t)my_seq * a.width + c;
+    const float s = my_pos > 0 ? fmaf(da, *S, db) : db;
+    *S = s;
+    const float v = s * a.yx[(size_t)m * a.ld + c];
+    if (a.out_x) { a.out_x[c] = v; return; }
+    unsigned char* o = (unsigned char*)a.out.p + row_operand_off(a.out_kind, a.out.chunks, m, c);
+    if (a.out_kind == WK_BF16) *(__nv_bfloat16*)o = __float2bfloat16_rn(v);
+    else *(float*)o = v;
+}
+cudaError_t launch_recur_step(const RecurArgs& a_in, cudaStream_t st) {
+    RecurArgs a = a_in;
+    const int CK = chunk_elems(a.kind), per = (a.bwp / 8 + kRsWarps - 1) / kRsWarps;
+    const size_t smem = (size_t)kRsRows * a.kc * CK * 4;
+    if (a.M <= 0 || a.bwp % 8 || a.bw > a.bwp || a.bw > a.kc * CK || a.nt != a.blocks * 2 * a.bwp || smem > 200 * 1024) return cudaErrorInvalidValue;
+    const void* fn = a.kind == WK_BF16 ? (const void*)recur_step<WK_BF16> : (const void*)recur_step<WK_F32>;
+    if (smem > 48 * 1024) {
+        const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        if (e != cudaSuccess) return e;
+    }
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(a.blocks * per, (a.M + kRsRows - 1) / kRsRows); cfg.blockDim = dim3(kRsWarps * 32); cfg.dynamicSmemBytes = smem; cfg.stream = st;
+    cudaLaunchAttribute at[1];
+    at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization; at[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = at; cfg.numAttrs = a.use_pdl ? 1 : 0;
+    void* params[] = {&a};
+    return cudaLaunchKernelExC(&cfg, fn, params);
+}
+
+// ------------------------------------------------------------------------------------------------ many rows of one sequence
+// Thread = row x 8 channels of a block (16 bytes of a bf16 operand); lanes are 8 rows x 4 groups of channels.
+template <int KIND>
+__global__ void __launch_bounds__(256) recur_conv(const RecurArgs a) {
+    const int gpb = a.bwp / 8, groups = a.blocks * gpb;
+    const int lane = threadIdx.x & 31, g = (blockIdx.x * 8 + (threadIdx.x >> 5)) * 4 + (lane >> 3), m = blockIdx.y * 8 + (lane & 7);
+    if (g >= groups || m >= a.M) return;
+    const int blk = g / gpb, k0 = (g - blk * gpb) * 8, c0 = blk * a.bw + k0;
+    const int pos = a.row_pos[m];
+    const float* src = a.yx + (size_t)m * a.ld + a.x_off;
+    float u[8];
+    if (a.conv.taps == 4 && m >= 3 && k0 + 8 <= a.bw && ((c0 | a.ld | a.x_off) & 3) == 0) {
+        float4 x[4][2];
+#pragma unroll
+        for (int d = 0; d < 4; d++) {
+            const float* r = src + c0 - (ptrdiff_t)d * a.ld;
+            x[d][0] = *(const float4*)r; x[d][1] = *(const float4*)(r + 4);
+        }
+#pragma unroll
+        for (int i = 0; i < 8; i++) {
+            const float4 w = *(const float4*)(a.conv.w + (size_t)(c0 + i) * 4);
+            const float* x0 = (const float*)&x[0][0] + i; const float* x1 = (const float*)&x[1][0] + i;
+            const float* x2 = (const float*)&x[2][0] + i; const float* x3 = (const float*)&x[3][0] + i;
+            u[i] = fmaf(w.w, *x0, fmaf(w.z, *x1, fmaf(w.y, *x2, w.x * *x3))) + (a.conv_b ? a.conv_b[c0 + i] : 0.0f);
+        }
+    } else {
+        const float* ring = a.conv.ring + (size_t)a.seq0 * a.conv.taps * a.conv.ch;
+#pragma unroll
+        for (int i = 0; i < 8; i++) u[i] = k0 + i < a.bw ? conv_at(a.conv, ring, src, a.ld, m, pos, c0 + i) + (a.conv_b ? a.conv_b[c0 + i] : 0.0f) : 0.0f;
+    }
+    float* uo = a.u + (size_t)m * a.ldu + c0;
+    if (k0 + 8 <= a.bw && ((a.ldu | c0) & 3) == 0) {
+        ((float4*)uo)[0] = make_float4(u[0], u[1], u[2], u[3]);
+        ((float4*)uo)[1] = make_float4(u[4], u[5], u[6], u[7]);
+    } else {
+#pragma unroll
+        for (int i = 0; i < 8; i++) if (k0 + i < a.bw) uo[i] = u[i];
+    }
+    const int kcol = blk * a.kc * (KIND == WK_BF16 ? 64 : 32) + k0;
+    const size_t o = row_operand_off(KIND, a.hi.chunks, m, kcol);
+    if (KIND == WK_BF16) {
+        uint32_t h[4], l[4];
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            h[i] = pack_bf16(u[2 * i], u[2 * i + 1]);
+            l[i] = pack_bf16(u[2 * i] - __uint_as_float(h[i] << 16), u[2 * i + 1] - __uint_as_float(h[i] & 0xffff0000u));
+        }
+        *(uint4*)((unsigned char*)a.hi.p + o) = make_uint4(h[0], h[1], h[2], h[3]);
+        *(uint4*)((unsigned char*)a.lo.p + o) = make_uint4(l[0], l[1], l[2], l[3]);
+    } else {
+        float4* f = (float4*)((unsigned char*)a.hi.p + o);
+        f[0] = make_float4(u[0], u[1], u[2], u[3]);
+        f[1] = make_float4(u[4], u[5], u[6], u[7]);
+    }
+}
+cudaError_t launch_recur_conv(const RecurArgs& a, cudaStream_t st) {
+    const int groups = a.blocks * a.bwp / 8;
+    if (a.M <= 0 || a.row_seq || a.hi.chunks != a.blocks * a.kc || (a.kind == WK_BF16 && (!a.lo.p || a.lo.chunks != a.hi.chunks))) return cudaErrorInvalidValue;
+    const dim3 grid((groups + 31) / 32, (a.M + 7) / 8);
+    if (a.kind == WK_BF16) recur_conv<WK_BF16><<<grid, 256, 0, st>>>(a);
+    else recur_conv<WK_F32><<<grid, 256, 0, st>>>(a);
+    return cudaGetLastError();
+}
+
+// CTA = 16 channels; thread = channel x 8 consecutive rows, 32 such pieces = a tile of 256 rows.  A piece is (product of decays, sum); one
+// warp per channel scans the 32 pieces, then every thread goes through its rows again from the right start.
+namespace { constexpr int kScCh = 16, kScSeg = 32, kScT = 8, kScThreads = kScCh * kScSeg, kScTile = kScSeg * kScT; }
+__global__ void __launch_bounds__(kScThreads, 2) recur_scan(const RecurArgs a) {
+    __shared__ float ag_a[kScCh][kScSeg + 1], ag_b[kScCh][kScSeg + 1], out[kScTile][kScCh + 1];
+    const int tid = threadIdx.x, ch = tid % kScCh, seg = tid / kScCh, warp = tid >> 5, lane = tid & 31;
+    const int c = blockIdx.x * kScCh + ch, cl = min(c, a.width - 1);
+    const int blk = cl / a.bw, gr = blk * 2 * a.bwp + (cl - blk * a.bw), gi = gr + a.bwp;
+    const float rb = a.r_b[cl], ib = a.i_b[cl], sp = softplus_exact(a.lam[cl]);
+    const int pos0 = a.row_pos[0];
+    float carry = 0.0f;                                        // of channel `warp`, in every lane of the warp
+    const int cw = blockIdx.x * kScCh + warp;
+    if (pos0 > 0 && cw < a.width) carry = a.state[(size_t)a.seq0 * a.width + cw];
+    for (int t0 = 0; t0 < a.M; t0 += kScTile) {
+        const int r0 = t0 + seg * kScT;
+        float da[kScT], db[kScT], y[kScT];
+#pragma unroll
+        for (int k = 0; k < kScT; k++) {
+            const size_t m = min(r0 + k, a.M - 1);
+            da[k] = a.gates[m * a.ldg + gr]; db[k] = a.gates[m * a.ldg + gi]; y[k] = a.u[m * a.ldu + cl];
+        }
+#pragma unroll
+        for (int k = 0; k < kScT; k++) {
+            float x, v;
+            recur_gate(da[k] + rb, db[k] + ib, y[k], sp, x, v);
+            const bool in = r0 + k < a.M;
+            da[k] = in ? x : 1.0f;
+            db[k] = in ? v : 0.0f;
+        }
+        float A = 1.0f, B = 0.0f;
+#pragma unroll
+        for (int k = 0; k < kScT; k++) { A *= da[k]; B = fmaf(da[k], B, db[k]); }
+        ag_a[ch][seg] = A;
+        ag_b[ch][seg] = B;
+#pragma unroll
+        for (int k = 0; k < kScT; k++) y[k] = a.yx[(size_t)min(r0 + k, a.M - 1) * a.ld + cl];
+        __syncthreads();
+        {
+            float pa = ag_a[warp][lane], pb = ag_b[warp][lane];
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const float qa = __shfl_up_sync(0xffffffffu, pa, o), qb = __shfl_up_sync(0xffffffffu, pb, o);
+                if (lane >= o) { pb = fmaf(pa, qb, pb); pa *= qa; }
+            }
+            const float end = fmaf(pa, carry, pb);             // state after piece `lane`
+            const float before = __shfl_up_sync(0xffffffffu, end, 1);
+            ag_b[warp][lane] = lane ? before : carry;
+            carry = __shfl_sync(0xffffffffu, end, 31);
+        }
+        __syncthreads();
+        float s = ag_b[ch][seg];
+#pragma unroll
+        for (int k = 0; k < kScT; k++) {
+            s = fmaf(da[k], s, db[k]);
+            out[seg * kScT + k][ch] = s * y[k];
+        }
+        __syncthreads();
+        {   // 8 channels of a row per thread: 16 bytes of the operand
+            const int m = tid % kScTile, h = tid / kScTile, k0 = blockIdx.x * kScCh + h * 8;
+            if (t0 + m < a.M && k0 < a.width) {
+                float f[8];
+#pragma unroll
+                for (int i = 0; i < 8; i++) f[i] = k0 + i < a.width ? out[m][h * 8 + i] : 0.0f;
+                unsigned char* o = (unsigned char*)a.out.p + row_operand_off(a.out_kind, a.out.chunks, t0 + m, k0);
+                if (a.out_kind == WK_BF16) *(uint4*)o = make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
+                else { ((float4*)o)[0] = make_float4(f[0], f[1], f[2], f[3]); ((float4*)o)[1] = make_float4(f[4], f[5], f[6], f[7]); }
+            }
+        }
+    }
+    if (lane == 0 && cw < a.width) a.state[(size_t)a.seq0 * a.width + cw] = carry;
+}
+cudaError_t launch_recur_scan(const RecurArgs& a, cudaStream_t st) {
+    if (a.M <= 0 || a.row_seq) return cudaErrorInvalidValue;
+    recur_scan<<<(a.width + kScCh - 1) / kScCh, kScThreads, 0, st>>>(a);
+    return cudaGetLastError();
+}
+
+}  // namespace lum

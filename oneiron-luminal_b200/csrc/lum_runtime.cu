@@ -112,7 +112,7 @@ struct Tensor {
     size_t row0 = 0, col0 = 0;          // shard origin in the full tensor
     size_t full_rows = 0, full_cols = 0;
     int nt = 0;                         // chunked layout (kc == kLayoutChunked): padded rows of the container this tensor is a row range of
-    size_t crow0 = 0;                   // ... and the tensor's first row in it
+    RowMap rm{};                        // ... and the tensor's rows in it
     size_t bytes() const {
         const size_t n = rows * cols;
         return kind == WK_Q8 ? n + n / 16 : kind == WK_BF16 ? n * 2 : n * 4;
@@ -134,6 +134,18 @@ struct LayerW {
     int o_chunks = 0, dn_chunks = 0;
     int mix = 0;                                              // 0 none, 1 the first mixing layer, 2 a later one
     Tensor attn_norm_b, v_mix, temp, dist_r1, dist_r2, act_par;
+    // block_kind 2 (w_in: q | k | v, or y | x of a recurrence; w_ff: gate and up rows in turn, 8 at a time)
+    int index = 0;                                            // the layer this run is of (a loop runs a layer several times)
+    void *w_ff = nullptr, *w_rec = nullptr;                   // w_rec: per block the rows of r, then those of i
+    int nt_ff = 0, bwp = 0, rec_kc = 0, nt_rec = 0;
+    float *in_bias = nullptr, *in_conv = nullptr;             // over the rows of w_in
+    const float2* rot = nullptr;
+    Tensor q_conv, k_conv, v_conv, lq1, lk1, lq2, lk2, hc_in[2], hc_out[2], hc_mix[2];
+    Tensor rec_y, rec_y_b, rec_x, rec_x_b, rec_conv, rec_conv_b, rec_ra, rec_ra_b, rec_ri, rec_ri_b, rec_lam;
+    float *ring = nullptr, *state = nullptr;                  // of this run: [sequence][taps][ring_ch], [sequence][rec_width]
+    int ring_ch = 0;
+    size_t ring_floats() const { return (size_t)g.conv_taps * ring_ch; }
+    size_t state_floats() const { return g.mixer == 1 ? (size_t)g.rec_width : 0; }
 };
 
 }  // namespace
@@ -157,6 +169,11 @@ struct lum_rt {
     int h_chunks = 0, ldx = 0, ldq = 0, q_floats = 0, attn_chunks = 0, act_chunks = 0, vf_floats = 0, head_nt = 0;
     float* v_first = nullptr;
     double* pos_freq = nullptr;
+    // block_kind 2: streams of the residual (x holds them side by side), the input of the next sublayer, tokens every sequence has seen
+    int n_streams = 0, u_floats = 0, gate_floats = 0, rec_chunks = 0;
+    float* u = nullptr;
+    size_t seq_state_bytes = 0;
+    std::vector<int> seq_pos;
     size_t qkv_floats = 0, attn_floats = 0, h_floats = 0;     // sizes of qkv, attn, h below
     // rows whose logits the next execute keeps (lum_want_logits), and what the last one kept
     std::vector<int32_t> want;
@@ -201,8 +218,10 @@ struct lum_rt {
         float *qkv = nullptr, *o = nullptr, *gu = nullptr, *down = nullptr, *logits = nullptr;   // K-split partial planes of the products
         int8_t* xq = nullptr; float* sx = nullptr;                   // quantised activation rows of the product in flight
         std::vector<int32_t> h_tok, h_pos, h_slot;
-        RowOperand in{}, att{}, act{};                               // block_kind 1: operands of the three products
+        RowOperand in{}, att{}, act{};                               // block_kind 1 and 2: operands of the products
         float* v_first = nullptr;
+        RowOperand rec_hi{}, rec_lo{};                               // block_kind 2: operands of a recurrence's gates
+        float *sub = nullptr, *u = nullptr, *rec_u = nullptr, *gates = nullptr;      // a sublayer's output, sum of the streams, convolved inputs, gates
     } rows;
     float* yarn_inv = nullptr;        // rope_style 2: inverse-frequency table [head_dim / 2] on the device
     float yarn_factor_cs = 1.0f;      // ... and the factor on cos / sin
@@ -341,7 +360,7 @@ void free_model(lum_rt* rt) {
     rt->g_batch = nullptr; rt->g_batch_n = 0; rt->batch_n = 0; rt->cur_seq = 0;
     rt->rows = lum_rt::Rows();
     rt->b_step = nullptr; rt->b_log = nullptr;
-    rt->v_first = nullptr; rt->pos_freq = nullptr;
+    rt->v_first = nullptr; rt->pos_freq = nullptr; rt->u = nullptr; rt->n_streams = 0; rt->seq_state_bytes = 0; rt->seq_pos.clear();
     rt->want.clear(); rt->want_n = 0; rt->want_logits = nullptr; rt->want_cap = 0; rt->want_idx = nullptr; rt->want_idx_cap = 0;
     rt->attn_cnt = nullptr; rt->am_cnt = nullptr; rt->d_sample = nullptr;
     rt->d_page_table = nullptr; rt->page_rows = 0; rt->h_page_table.clear(); rt->page_ref.clear(); rt->page_free.clear();
@@ -352,16 +371,73 @@ void free_model(lum_rt* rt) {
     rt->has_model = false;
 }
 
+// Layer runs of a model: its layers in order, those of the loop several times.
+int n_runs(const lum_model_desc& d) { return d.n_layers + (d.loop_times > 1 ? (d.loop_times - 1) * (d.loop_stop - d.loop_start) : 0); }
+int first_run(const lum_model_desc& d, int layer) { return d.loop_times > 1 && layer >= d.loop_stop ? layer + (d.loop_times - 1) * (d.loop_stop - d.loop_start) : layer; }
+int layer_of_run(const lum_model_desc& d, int run) {
+    if (d.loop_times <= 1 || run < d.loop_stop) return run;
+    const int n = d.loop_stop - d.loop_start, end = d.loop_start + n * d.loop_times;
+    return run < end ? d.loop_start + (run - d.loop_start) % n : run - (d.loop_times - 1) * n;
+}
+
+Tensor* sequential_slot(lum_rt* rt, int slot, LayerW& l) {
+    const lum_layer_desc& g = l.g;
+    const bool att = g.mixer == 0, rec = g.mixer == 1, conv = g.conv_taps > 0, ff = g.ffn > 0;
+    auto when = [](bool have, Tensor& t) { return have ? &t : nullptr; };
+    switch (slot) {
+        case LUM_S_ATTN_NORM: return &l.attn_norm;
+        case LUM_S_MLP_NORM: return when(ff, l.mlp_norm);
+        case LUM_S_GATE: return when(ff, l.gate);
+        case LUM_S_UP: return when(ff, l.up);
+        case LUM_S_DOWN: return when(ff, l.down);
+        case LUM_S_O: return &l.o;
+        case LUM_S_Q: return when(att, l.q);
+        case LUM_S_K: return when(att, l.k);
+        case LUM_S_V: return when(att, l.v);
+        case LUM_S_Q_BIAS: return when(att && g.qkv_bias, l.q_b);
+        case LUM_S_K_BIAS: return when(att && g.qkv_bias, l.k_b);
+        case LUM_S_V_BIAS: return when(att && g.qkv_bias, l.v_b);
+        case LUM_S_Q_NORM: return when(att && g.head_norm, l.q_norm);
+        case LUM_S_K_NORM: return when(att && g.head_norm, l.k_norm);
+        case LUM_S_Q_CONV: return when(att && conv, l.q_conv);
+        case LUM_S_K_CONV: return when(att && conv, l.k_conv);
+        case LUM_S_V_CONV: return when(att && conv, l.v_conv);
+        case LUM_S_LQ1: return when(att && g.maps == 2, l.lq1);
+        case LUM_S_LK1: return when(att && g.maps == 2, l.lk1);
+        case LUM_S_LQ2: return when(att && g.maps == 2, l.lq2);
+        case LUM_S_LK2: return when(att && g.maps == 2, l.lk2);
+        case LUM_S_HC1_IN: return when(rt->d.streams > 0, l.hc_in[0]);
+        case LUM_S_HC1_OUT: return when(rt->d.streams > 0, l.hc_out[0]);
+        case LUM_S_HC1_MIX: return when(rt->d.streams > 0, l.hc_mix[0]);
+        case LUM_S_HC2_IN: return when(ff && rt->d.streams > 0, l.hc_in[1]);
+        case LUM_S_HC2_OUT: return when(ff && rt->d.streams > 0, l.hc_out[1]);
+        case LUM_S_HC2_MIX: return when(ff && rt->d.streams > 0, l.hc_mix[1]);
+        case LUM_S_REC_Y: return when(rec, l.rec_y);
+        case LUM_S_REC_Y_BIAS: return when(rec, l.rec_y_b);
+        case LUM_S_REC_X: return when(rec, l.rec_x);
+        case LUM_S_REC_X_BIAS: return when(rec, l.rec_x_b);
+        case LUM_S_REC_CONV: return when(rec && conv, l.rec_conv);
+        case LUM_S_REC_CONV_BIAS: return when(rec && conv, l.rec_conv_b);
+        case LUM_S_REC_RA: return when(rec, l.rec_ra);
+        case LUM_S_REC_RA_BIAS: return when(rec, l.rec_ra_b);
+        case LUM_S_REC_RI: return when(rec, l.rec_ri);
+        case LUM_S_REC_RI_BIAS: return when(rec, l.rec_ri_b);
+        case LUM_S_REC_LAM: return when(rec, l.rec_lam);
+        default: return nullptr;
+    }
+}
+
 // slot -> tensor of this runtime (null if the slot does not exist for this model)
 Tensor* slot_tensor(lum_rt* rt, int slot, int layer) {
     switch (slot) {
         case LUM_S_EMBED: return &rt->embed;
         case LUM_S_FINAL_NORM: return &rt->final_norm;
         case LUM_S_LM_HEAD: return rt->d.tied_head ? nullptr : &rt->lm_head;
-        case LUM_S_FINAL_NORM_BIAS: return rt->d.block_kind == 1 && rt->d.norm_kind == 1 ? &rt->final_norm_b : nullptr;
+        case LUM_S_FINAL_NORM_BIAS: return rt->d.block_kind != 0 && rt->d.norm_kind == 1 ? &rt->final_norm_b : nullptr;
         default: break;
     }
     if (layer < 0 || layer >= rt->d.n_layers) return nullptr;
+    if (rt->d.block_kind == 2) return sequential_slot(rt, slot, rt->L[(size_t)first_run(rt->d, layer)]);
     LayerW& l = rt->L[(size_t)layer];
     if (rt->d.block_kind == 1) {
         switch (slot) {
@@ -411,7 +487,10 @@ Tensor* slot_tensor(lum_rt* rt, int slot, int layer) {
 }
 // generator id of a slot: shared with the CPU oracle's own statement of the generator
 // (slots 14 and up — the gpt_oss-style tensors — have a range of their own, so the ids of the first 14 never moved)
-uint64_t tensor_id(int slot, int layer) { return slot < 14 ? (uint64_t)layer * 16u + (uint64_t)slot : (1ull << 21) + (uint64_t)layer * 32u + (uint64_t)slot; }
+uint64_t tensor_id(int slot, int layer) {
+    if (slot >= 32) return (1ull << 22) + (uint64_t)layer * 64u + (uint64_t)slot;
+    return slot < 14 ? (uint64_t)layer * 16u + (uint64_t)slot : (1ull << 21) + (uint64_t)layer * 32u + (uint64_t)slot;
+}
 int slot_layer_for_id(const lum_rt* rt, int slot, int layer) {
     return (slot == LUM_S_EMBED || slot == LUM_S_FINAL_NORM || slot == LUM_S_LM_HEAD || slot == LUM_S_FINAL_NORM_BIAS) ? rt->d.n_layers : layer;
 }
@@ -729,6 +808,7 @@ int issue_step(lum_rt* rt, bool with_head, bool pdl, int* n_launch) {
 NormArgs block_norm(const lum_rt* rt, const Tensor& gain, const Tensor& bias) {
     NormArgs n{};
     n.mode = rt->d.norm_kind == 1 ? NORM_LAYER : NORM_RMS;
+    n.gain0 = rt->d.norm_kind == 2 ? 1.0f : 0.0f;
     n.gain = (const float*)gain.w; n.bias = rt->d.norm_kind == 1 ? (const float*)bias.w : nullptr;
     n.eps = rt->d.rms_eps; n.width = rt->d.hidden;
     return n;
@@ -761,6 +841,7 @@ BandArgs block_band(const lum_rt* rt, const LayerW& w) {
     if (d.qk_norm) { t.p.q_gain = (const float*)w.q_norm.w; t.p.k_gain = (const float*)w.k_norm.w; }
     t.p.eps = d.rms_eps; t.p.scale = w.g.scale; t.p.temp = d.dist_bias ? (const float*)w.temp.w : nullptr;
     t.p.n_q = w.g.n_q_heads; t.p.n_kv = w.g.n_kv_heads; t.p.dk = w.g.qk_dim; t.p.dv = w.g.v_dim; t.p.dkp = w.dkp; t.p.dvp = w.dvp;
+    t.p.maps = w.g.maps > 1 ? w.g.maps : 1;
     t.p.mix = w.mix; t.p.lambda = (const float*)w.v_mix.w; t.p.ld_vfirst = rt->vf_floats;
     t.k_cache = w.kc; t.v_cache = w.vc; t.kv_bf16 = d.kv_dtype == LUM_BF16;
     t.window = w.g.window; t.max_seq = d.max_seq; t.max_batch = rt->max_batch;
@@ -812,10 +893,116 @@ int issue_step_blocks(lum_rt* rt, bool with_head, bool pdl, int* n_launch) {
     return 0;
 }
 
+// ---- one sublayer after the other, over residual streams (block_kind 2)
+// A decode step: the embedding starts the streams; then every sublayer is [norm + first products] -> [its middle] -> [last product, whose
+// epilogue takes the result into the streams and mixes the next sublayer's input u].  The middle of attention is one kernel, that of a
+// recurrence is one kernel, that of a feed-forward is the first product's epilogue.
+NormArgs sequential_norm(const lum_rt* rt, const Tensor& gain) { return block_norm(rt, gain, Tensor()); }
+// what a sublayer does to the streams and what the one behind it reads: sublayer q (0 mixer, 1 feed-forward) of run i; i < 0: the embedding
+StreamArgs sequential_streams(const lum_rt* rt, int i, int q) {
+    StreamArgs h{};
+    h.n = rt->n_streams; h.ldx = rt->ldx;
+    const bool hc = rt->d.streams > 0;
+    if (i >= 0 && hc) { h.mix = (const float*)rt->L[(size_t)i].hc_mix[q].w; h.out = (const float*)rt->L[(size_t)i].hc_out[q].w; }
+    const int ni = i < 0 ? 0 : q == 0 && rt->L[(size_t)i].g.ffn > 0 ? i : i + 1, nq = i >= 0 && ni == i ? 1 : 0;
+    if (hc && ni < (int)rt->L.size()) h.next = (const float*)rt->L[(size_t)ni].hc_in[nq].w;
+    return h;
+}
+// norm of the sublayer behind sublayer q of run i; null: the last one (the final norm follows)
+const Tensor* sequential_next_norm(const lum_rt* rt, int i, int q) {
+    if (i >= 0 && q == 0 && rt->L[(size_t)i].g.ffn > 0) return &rt->L[(size_t)i].mlp_norm;
+    return i + 1 < (int)rt->L.size() ? &rt->L[(size_t)(i + 1)].attn_norm : nullptr;
+}
+DenseArgs sequential_in(const lum_rt* rt, const LayerW& w) {
+    DenseArgs g = block_in(rt, w);
+    g.act_row0 = g.nt; g.bias = w.in_bias; g.gelu_rows = w.g.mixer == 1 ? w.k_off : 0;
+    return g;
+}
+DenseArgs sequential_ff(const lum_rt* rt, const LayerW& w) {
+    DenseArgs g{};
+    g.nk = 1; g.kind = kind_of(rt->d.weight_dtype); g.nt = g.n_real = g.act_row0 = w.nt_ff; g.epi = DENSE_STORE; g.mult = 1.0f; g.norm.mode = NORM_NONE;
+    g.seg[0].w = w.w_ff; g.seg[0].chunks = rt->h_chunks; g.pair = 1; g.limit = w.g.ffn_limit; g.status = rt->status;
+    return g;
+}
+DenseArgs sequential_out(const lum_rt* rt, const void* weights, int chunks) {
+    DenseArgs g{};
+    g.nk = 1; g.kind = kind_of(rt->d.weight_dtype); g.nt = g.act_row0 = (rt->d.hidden + 7) / 8 * 8; g.n_real = rt->d.hidden; g.mult = 1.0f;
+    g.seg[0].w = weights; g.seg[0].chunks = chunks; g.norm.mode = NORM_NONE; g.status = rt->status;
+    return g;
+}
+BandArgs sequential_band(const lum_rt* rt, const LayerW& w) {
+    BandArgs t = block_band(rt, w);
+    t.p.per_head = 1; t.p.ld = w.nt_in; t.chunk = w.g.chunk;
+    if (!w.g.head_norm) t.p.q_gain = t.p.k_gain = nullptr;
+    else { t.p.q_gain = (const float*)w.q_norm.w; t.p.k_gain = (const float*)w.k_norm.w; }
+    t.p.conv.w = w.in_conv; t.p.conv.taps = w.g.conv_taps; t.p.conv.ring = w.ring; t.p.conv.ch = w.ring_ch;
+    t.p.rot = w.rot; t.p.rot_dims = w.g.rot_dims;
+    t.lq1 = (const float*)w.lq1.w; t.lk1 = (const float*)w.lk1.w; t.lq2 = (const float*)w.lq2.w; t.lk2 = (const float*)w.lk2.w; t.diff = w.g.diff;
+    return t;
+}
+RecurArgs sequential_recur(const lum_rt* rt, const LayerW& w) {
+    RecurArgs r{};
+    r.ld = w.nt_in; r.x_off = w.k_off; r.width = w.g.rec_width; r.blocks = w.g.rec_blocks; r.bw = w.g.rec_width / w.g.rec_blocks; r.bwp = w.bwp;
+    r.w_gate = w.w_rec; r.kind = kind_of(rt->d.weight_dtype); r.kc = w.rec_kc; r.nt = w.nt_rec;
+    r.conv_b = w.g.conv_taps > 0 ? (const float*)w.rec_conv_b.w : nullptr;
+    r.r_b = (const float*)w.rec_ra_b.w; r.i_b = (const float*)w.rec_ri_b.w; r.lam = (const float*)w.rec_lam.w;
+    r.conv.w = (const float*)w.rec_conv.w; r.conv.taps = w.g.conv_taps; r.conv.ring = w.ring; r.conv.ch = w.ring_ch;
+    r.state = w.state; r.max_batch = rt->max_batch; r.max_seq = rt->d.max_seq; r.status = rt->status;
+    return r;
+}
+int issue_step_sequential(lum_rt* rt, bool with_head, bool pdl, int* n_launch) {
+    const lum_model_desc& d = rt->d;
+    cudaStream_t st = rt->stream;
+    int n = 0;
+    StreamRowsArgs e{};
+    e.hc = sequential_streams(rt, -1, 0); e.hc.x = rt->x; e.hc.u = rt->u;
+    e.table = rt->embed.w; e.table_kind = rt->embed.kind; e.vocab = d.vocab; e.state = rt->state; e.scale = d.embed_scale; e.max_seq = d.max_seq; e.M = 1; e.width = d.hidden;
+    e.status = rt->status;      // first kernel of the step: ordinary stream order behind the previous step
+    CU(rt, launch_stream_rows(e, st)); n++;
+    for (int i = 0; i < (int)rt->L.size(); i++) {
+        const LayerW& w = rt->L[(size_t)i];
+        auto out = [&](const void* weights, int chunks, const float* x, int q) -> int {
+            DenseArgs o = sequential_out(rt, weights, chunks);
+            o.epi = DENSE_STREAMS; o.hc = sequential_streams(rt, i, q); o.hc.x = rt->x; o.hc.u = rt->u; o.seg[0].x = x; o.use_pdl = pdl;
+            CU(rt, launch_dense_gemv(o, rt->sm_count, st)); n++;
+            return 0;
+        };
+        DenseArgs g = sequential_in(rt, w);
+        g.seg[0].x = rt->u; g.y = rt->qkv; g.norm = sequential_norm(rt, w.attn_norm); g.use_pdl = pdl;
+        CU(rt, launch_dense_gemv(g, rt->sm_count, st)); n++;
+        if (w.g.mixer == 1) {
+            RecurArgs r = sequential_recur(rt, w);
+            r.yx = rt->qkv; r.M = 1; r.step = rt->state; r.seq0 = rt->cur_seq; r.out_x = rt->attn; r.use_pdl = pdl;
+            CU(rt, launch_recur_step(r, st)); n++;
+        } else {
+            BandArgs t = sequential_band(rt, w);
+            t.p.qkv = rt->qkv; t.M = 1; t.state = rt->state; t.seq0 = rt->cur_seq; t.out_x = rt->attn; t.use_pdl = pdl;
+            if (rt->page_rows) t.pg = KvPages{rt->d_page_table + (size_t)rt->cur_seq * rt->pages_per_seq, rt->page_lg, rt->pages_per_seq};
+            else {
+                const size_t esz = t.kv_bf16 ? 2 : 4, row0 = (size_t)rt->cur_seq * d.max_seq;
+                t.k_cache = (char*)t.k_cache + row0 * w.k_elems * esz; t.v_cache = (char*)t.v_cache + row0 * w.v_elems * esz;
+            }
+            CU(rt, launch_band_decode(t, rt->sm_count, st)); n++;
+        }
+        if (int r = out(w.w_o, w.o_chunks, rt->attn, 0)) return r;
+        if (w.g.ffn > 0) {
+            DenseArgs f = sequential_ff(rt, w);
+            f.seg[0].x = rt->u; f.act_x = rt->h; f.norm = sequential_norm(rt, w.mlp_norm); f.use_pdl = pdl;
+            CU(rt, launch_dense_gemv(f, rt->sm_count, st)); n++;
+            if (int r = out(w.w_dn, w.dn_chunks, rt->h, 1)) return r;
+        }
+    }
+    if (with_head) if (int r = block_head_sample(rt, rt->u, pdl, &n)) return r;
+    if (n_launch) *n_launch = n;
+    return 0;
+}
+
 int capture_graph(lum_rt* rt, bool with_head, bool pdl, cudaGraphExec_t* out, int* n_launch) {
     cudaGraph_t g = nullptr;
     CU(rt, cudaStreamBeginCapture(rt->stream, cudaStreamCaptureModeThreadLocal));
-    int r = rt->d.block_kind == 1 ? issue_step_blocks(rt, with_head, pdl, n_launch) : issue_step(rt, with_head, pdl, n_launch);
+    int r = rt->d.block_kind == 1   ? issue_step_blocks(rt, with_head, pdl, n_launch)
+            : rt->d.block_kind == 2 ? issue_step_sequential(rt, with_head, pdl, n_launch)
+                                    : issue_step(rt, with_head, pdl, n_launch);
     cudaError_t e = cudaStreamEndCapture(rt->stream, &g);
     if (r) { if (g) cudaGraphDestroy(g); return r; }
     if (e != cudaSuccess) return fail(rt, LUM_E_CUDA, "cudaStreamEndCapture: %s", cudaGetErrorString(e));
@@ -847,6 +1034,7 @@ int run_step(lum_rt* rt, bool with_head) {
         return 0;
     }
     if (rt->d.block_kind == 1) return issue_step_blocks(rt, with_head, rt->cfg.use_pdl != 0, with_head ? &rt->launches_full : nullptr);
+    if (rt->d.block_kind == 2) return issue_step_sequential(rt, with_head, rt->cfg.use_pdl != 0, with_head ? &rt->launches_full : nullptr);
     return issue_step(rt, with_head, rt->cfg.use_pdl != 0, with_head ? &rt->launches_full : nullptr);
 }
 
@@ -921,7 +1109,7 @@ int kv_for_spans(lum_rt* rt, int seq, int layer, int kind, int rows, const char*
 // Every linear of the model in the packed tile stream, one GPU: the tensor-core products can take the model's rows.
 bool rows_supported(const lum_rt* rt) {
     const lum_model_desc& d = rt->d;
-    if (rt->has_model && d.block_kind == 1) return true;
+    if (rt->has_model && d.block_kind != 0) return true;
     if (!rt->has_model || d.weight_dtype != LUM_Q8_0 || d.tp_size > 1 || (d.head_dim != 64 && d.head_dim != 128)) return false;
     if (d.n_experts > 0 || d.proj_bias || d.attn_sinks || d.sliding_window > 0 || d.rope_style == 2) return false;     // per-token path only
     if (d.n_q_heads / d.n_kv_heads > (d.head_dim == 128 ? 4 : 8)) return false;
@@ -961,7 +1149,7 @@ int ensure_rows(lum_rt* rt, int want_rows) {
     std::vector<int32_t> iota((size_t)cap);
     for (int i = 0; i < cap; i++) iota[(size_t)i] = i;
     CU(rt, cudaMemcpyAsync(b.seq, iota.data(), (size_t)cap * 4, cudaMemcpyHostToDevice, rt->stream));
-    if (d.block_kind == 1) {
+    if (d.block_kind != 0) {
         const int kind = kind_of(d.weight_dtype);
         auto zeroed = [&](void** p, size_t bytes) -> int {          // padding columns of rows and operands stay zero
             if (int r = dev_alloc(rt, p, bytes)) return r;
@@ -969,9 +1157,19 @@ int ensure_rows(lum_rt* rt, int want_rows) {
             return 0;
         };
         auto operand = [&](RowOperand& o, int chunks) -> int { o.chunks = chunks; return zeroed(&o.p, row_operand_bytes(kind, chunks, cap)); };
-        if (int r = zeroed((void**)&b.xr, (size_t)cap * rt->ldx * 4)) return r;
+        if (int r = zeroed((void**)&b.xr, (size_t)cap * (rt->n_streams ? rt->n_streams : 1) * rt->ldx * 4)) return r;
+        if (d.block_kind == 2) {
+            if (int r = zeroed((void**)&b.sub, (size_t)cap * rt->ldx * 4)) return r;
+            if (int r = zeroed((void**)&b.u, (size_t)cap * rt->ldx * 4)) return r;
+            if (rt->rec_chunks) {
+                if (int r = zeroed((void**)&b.rec_u, (size_t)cap * rt->u_floats * 4)) return r;
+                if (int r = zeroed((void**)&b.gates, (size_t)cap * rt->gate_floats * 4)) return r;
+                if (int r = operand(b.rec_hi, rt->rec_chunks)) return r;
+                if (kind == WK_BF16) if (int r = operand(b.rec_lo, rt->rec_chunks)) return r;
+            }
+        }
         if (int r = dev_alloc(rt, (void**)&b.qkv, (size_t)cap * rt->ldq * 4)) return r;
-        if (int r = dev_alloc(rt, (void**)&b.q_rot, (size_t)cap * rt->q_floats * 4)) return r;
+        if (rt->q_floats) if (int r = dev_alloc(rt, (void**)&b.q_rot, (size_t)cap * rt->q_floats * 4)) return r;
         if (rt->vf_floats) if (int r = dev_alloc(rt, (void**)&b.v_first, (size_t)cap * rt->vf_floats * 4)) return r;
         if (int r = operand(b.in, rt->h_chunks)) return r;
         if (int r = operand(b.att, rt->attn_chunks)) return r;
@@ -1030,7 +1228,7 @@ int block_want_rows(lum_rt* rt, size_t w0, int n, int c0) {
     for (int i = 0; i < n; i++) idx[(size_t)i] = rt->want[w0 + i] - c0;
     CU(rt, cudaMemcpyAsync(rt->want_idx, idx.data(), (size_t)n * 4, cudaMemcpyHostToDevice, rt->stream));     // pageable source: staged before the call returns
     NormRowsArgs nr{};
-    nr.x = b.xr; nr.ldx = rt->ldx; nr.row_index = rt->want_idx; nr.M = n; nr.norm = block_norm(rt, rt->final_norm, rt->final_norm_b);
+    nr.x = rt->d.block_kind == 2 ? b.u : b.xr; nr.ldx = rt->ldx; nr.row_index = rt->want_idx; nr.M = n; nr.norm = block_norm(rt, rt->final_norm, rt->final_norm_b);
     nr.kind = kind_of(rt->d.weight_dtype); nr.out = b.in;
     CU(rt, launch_norm_rows(nr, rt->stream));
     DenseArgs g = block_head(rt);
@@ -1090,11 +1288,107 @@ int run_rows_blocks(lum_rt* rt, int M, int* d_tok, int* d_pos, const int* d_seq,
     return 0;
 }
 
+// run_rows for one sublayer after the other: the last products store, and stream_rows takes them into the streams row by row, with the next
+// sublayer's input mixed, normalised and laid out as an operand on the way.
+int run_rows_sequential(lum_rt* rt, int M, int* d_tok, int* d_pos, const int* d_seq, int seq0, int head) {
+    const lum_model_desc& d = rt->d;
+    lum_rt::Rows& b = rt->rows;
+    cudaStream_t st = rt->stream;
+    const int kind = kind_of(d.weight_dtype);
+    uint64_t launches = 0;
+    const bool one_each = d_seq != nullptr || M == 1;          // every row is the only one of its sequence
+    auto streams = [&](int i, int q) -> cudaError_t {
+        StreamRowsArgs s{};
+        s.hc = sequential_streams(rt, i, q); s.hc.x = b.xr;
+        if (i >= 0) { s.y = b.sub; s.ldy = rt->ldx; }
+        s.table = rt->embed.w; s.table_kind = rt->embed.kind; s.vocab = d.vocab; s.row_tok = d_tok; s.row_pos = d_pos; s.scale = d.embed_scale; s.max_seq = d.max_seq;
+        s.M = M; s.width = d.hidden; s.kind = kind; s.out = b.in; s.status = rt->status;
+        if (const Tensor* gain = sequential_next_norm(rt, i, q)) s.norm = sequential_norm(rt, *gain);
+        else if (head == 2) s.norm = sequential_norm(rt, rt->final_norm);
+        else s.hc.u = b.u;                                     // the plain sum: rows of it are normalised where they are needed
+        launches++;
+        return launch_stream_rows(s, st);
+    };
+    auto product = [&](DenseArgs& g) -> cudaError_t { g.M = M; launches++; return launch_dense_gemm(g, rt->sm_count, st); };
+    auto out = [&](const void* weights, RowOperand x) -> cudaError_t {
+        DenseArgs o = sequential_out(rt, weights, x.chunks);
+        o.epi = DENSE_STORE; o.seg[0].a = x.p; o.y = b.sub; o.ldy = rt->ldx;
+        return product(o);
+    };
+    auto tail = [&](const LayerW& w, const float* src, int ld) -> cudaError_t {
+        if (one_each || w.g.conv_taps == 0) return cudaSuccess;
+        ConvTailArgs t{};
+        t.conv.taps = w.g.conv_taps; t.conv.ring = w.ring; t.conv.ch = w.ring_ch;
+        t.src = src; t.ld = ld; t.n_ch = w.ring_ch; t.M = M; t.row_pos = d_pos; t.seq = seq0;
+        launches++;
+        return launch_conv_tail(t, st);
+    };
+    CU(rt, streams(-1, 0));
+    for (int i = 0; i < (int)rt->L.size(); i++) {
+        const LayerW& w = rt->L[(size_t)i];
+        RowOperand att = b.att, act = b.act;
+        att.chunks = w.o_chunks; act.chunks = w.dn_chunks;
+        DenseArgs g = sequential_in(rt, w);
+        g.seg[0].a = b.in.p; g.y = b.qkv; g.ldy = w.nt_in;
+        CU(rt, product(g));
+        if (w.g.mixer == 1) {
+            RecurArgs r = sequential_recur(rt, w);
+            r.yx = b.qkv; r.M = M; r.row_pos = d_pos; r.row_seq = d_seq; r.seq0 = seq0; r.out_kind = kind; r.out = att;
+            if (one_each) { CU(rt, launch_recur_step(r, st)); launches++; }
+            else {
+                r.u = b.rec_u; r.ldu = rt->u_floats; r.hi = b.rec_hi; r.lo = b.rec_lo; r.hi.chunks = r.lo.chunks = r.blocks * r.kc;
+                CU(rt, launch_recur_conv(r, st));
+                CU(rt, tail(w, b.qkv + r.x_off, r.ld));
+                DenseArgs p{};                                 // the gates: one group of rows and chunks per block, both terms of u
+                p.nk = kind == WK_BF16 ? 2 : 1; p.kind = kind; p.nt = p.n_real = p.act_row0 = r.nt; p.epi = DENSE_STORE; p.mult = 1.0f; p.norm.mode = NORM_NONE;
+                p.seg[0].w = p.seg[1].w = w.w_rec; p.seg[0].chunks = p.seg[1].chunks = r.kc; p.seg[0].a_chunks = p.seg[1].a_chunks = r.hi.chunks;
+                p.seg[0].a = r.hi.p; p.seg[1].a = r.lo.p; p.grp_rows = 2 * r.bwp; p.grp_chunks = r.kc; p.y = b.gates; p.ldy = r.nt; p.status = rt->status;
+                CU(rt, product(p));
+                r.gates = b.gates; r.ldg = r.nt;
+                CU(rt, launch_recur_scan(r, st));
+                launches += 2;
+            }
+        } else {
+            BandArgs t = sequential_band(rt, w);
+            t.p.qkv = b.qkv; t.M = M; t.pg = kv_pages(rt);
+            t.row_pos = d_pos; t.row_seq = d_seq; t.seq0 = seq0; t.q_out = b.q_rot; t.q = b.q_rot; t.out_kind = kind; t.out = att;
+            CU(rt, launch_qkv_head_rows(t, st));
+            CU(rt, tail(w, b.qkv, w.nt_in));
+            static const int env_tc = [] { const char* e = getenv("LUM_ATTN_TC"); return e ? atoi(e) : 1; }();
+            if (env_tc && M >= 16 && band_prompt_tc_supported(t)) CU(rt, launch_band_prompt_tc(t, st));
+            else CU(rt, launch_band_rows(t, rt->sm_count, st));
+            launches += 2;
+        }
+        CU(rt, out(w.w_o, att));
+        CU(rt, streams(i, 0));
+        if (w.g.ffn > 0) {
+            DenseArgs f = sequential_ff(rt, w);
+            f.seg[0].a = b.in.p; f.act = act;
+            CU(rt, product(f));
+            CU(rt, out(w.w_dn, act));
+            CU(rt, streams(i, 1));
+        }
+    }
+    if (head == 1) {
+        int n = 0;
+        if (int r = block_head_sample(rt, b.u + (size_t)(M - 1) * rt->ldx, false, &n)) return r;
+        launches += n;
+    } else if (head == 2) {
+        DenseArgs g = block_head(rt);
+        g.epi = DENSE_STORE; g.seg[0].a = b.in.p; g.y = b.logits; g.ldy = d.vocab;
+        CU(rt, product(g));
+        if (int r = batch_sample(rt, M, d_tok, d_pos, d_seq, 1, &launches)) return r;
+    }
+    rt->n_launches += launches;
+    return 0;
+}
+
 // One pass of M rows through every layer.  d_tok / d_pos: device arrays [M]; d_seq: device array [M], or null when every row
 // belongs to sequence seq0.  head: 0 none (the rows only fill the cache), 1 vocabulary projection + greedy sample of the LAST row
 // into the decode state (the end of a prompt), 2 of every row into the batch state (batched decode).
 int run_rows(lum_rt* rt, int M, int* d_tok, int* d_pos, const int* d_seq, int seq0, int head) {
     if (rt->d.block_kind == 1) return run_rows_blocks(rt, M, d_tok, d_pos, d_seq, seq0, head);
+    if (rt->d.block_kind == 2) return run_rows_sequential(rt, M, d_tok, d_pos, d_seq, seq0, head);
     const lum_model_desc& d = rt->d;
     lum_rt::Rows& b = rt->rows;
     const int H = d.hidden, hd = d.head_dim, qd = rt->nq_l * hd, kvd = rt->nkv_l * hd, W = qd + 2 * kvd, F = rt->ffn_l;
@@ -1250,7 +1544,7 @@ int run_prompt_rows(lum_rt* rt, int n, const int32_t* forced, int pos0) {
         size_t w1 = want0;
         while (w1 < rt->want.size() && rt->want[w1] < c0 + M) w1++;
         if (w1 > want0) {
-            if (rt->d.block_kind == 1) { if (int r = block_want_rows(rt, want0, (int)(w1 - want0), c0)) return r; }
+            if (rt->d.block_kind != 0) { if (int r = block_want_rows(rt, want0, (int)(w1 - want0), c0)) return r; }
             else for (size_t i = want0; i < w1; i++) if (int r = want_row(rt, rt->want[i] - c0, M, i)) return r;
             want0 = w1;
         }
@@ -1259,6 +1553,7 @@ int run_prompt_rows(lum_rt* rt, int n, const int32_t* forced, int pos0) {
     return 0;
 }
 
+int check_seq_pos(lum_rt* rt, int seq, int from, const char* who);
 // n tokens in one go.  forced: host token ids (prompt processing: sample only after the last) or null (feed
 // every sample back in).  The persistent kernel takes them all in one launch; otherwise one step per token.
 int run_tokens(lum_rt* rt, int n, const int32_t* forced, int pos0) {
@@ -1268,9 +1563,11 @@ int run_tokens(lum_rt* rt, int n, const int32_t* forced, int pos0) {
         const int from = forced ? pos0 : len;
         if (rt->page_rows) {      // (a contiguous cache lets the kernels flag a position beyond the capacity)
             if (from + n > rt->d.max_seq) return fail(rt, LUM_E_INVALID, "%d tokens from position %d pass the cache capacity %d", n, from, rt->d.max_seq);
-            if (int r = kv_ensure(rt, rt->cur_seq, from, from + n)) return r;
         }
+        if (int r = check_seq_pos(rt, rt->cur_seq, from, "execute")) return r;
+        if (rt->page_rows) if (int r = kv_ensure(rt, rt->cur_seq, from, from + n)) return r;
         len = from + n;
+        if (!rt->seq_pos.empty()) rt->seq_pos[(size_t)rt->cur_seq] = len;
     }
     if (forced && !rt->body_only && n >= rt->prefill_min_rows && !(rt->mega_ok && rt->use_mega) && rows_supported(rt))
         return run_prompt_rows(rt, n, forced, pos0);
@@ -1376,7 +1673,7 @@ int init_blocks(lum_rt* rt, lum_model_desc d, const lum_layer_desc* layers) {
     if (d.ep_size <= 0) { d.ep_size = 1; d.ep_rank = 0; }
     if (d.max_batch <= 0) d.max_batch = 1;
     if (d.max_new_tokens <= 0) d.max_new_tokens = 4096;
-    if (d.block_kind != 1) return fail(rt, LUM_E_INVALID, "model_init_layers: block_kind %d (1: parallel sublayers)", d.block_kind);
+    if (d.block_kind != 1) return fail(rt, LUM_E_INVALID, "model_init_layers: block_kind %d (1: parallel sublayers, 2: one after the other)", d.block_kind);
     if (d.tp_size != 1 || d.ep_size != 1 || rt->tp_size > 1) return fail(rt, LUM_E_UNSUPPORTED, "block_kind 1 runs on one GPU");
     if (d.max_batch > 1024) return fail(rt, LUM_E_INVALID, "max_batch %d (at most 1024 sequences)", d.max_batch);
     if (d.n_layers <= 0 || d.hidden <= 0 || d.vocab <= 0 || d.max_seq <= 0) return fail(rt, LUM_E_INVALID, "model dimensions must be positive");
@@ -1384,7 +1681,7 @@ int init_blocks(lum_rt* rt, lum_model_desc d, const lum_layer_desc* layers) {
     if (d.embed_dtype != LUM_F32 && d.embed_dtype != LUM_BF16) return fail(rt, LUM_E_UNSUPPORTED, "embedding dtype must be F32 or BF16");
     if (d.kv_dtype != LUM_F32 && d.kv_dtype != LUM_BF16) return fail(rt, LUM_E_UNSUPPORTED, "KV dtype must be F32 or BF16");
     if (d.norm_kind < 0 || d.norm_kind > 1 || d.pos_kind < 0 || d.pos_kind > 1 || (d.qk_norm != 0 && d.qk_norm != 2) || d.dist_bias < 0 || d.dist_bias > 1 || d.tied_head ||
-        d.n_experts || d.attn_sinks || d.proj_bias || d.rope_style)
+        d.n_experts || d.attn_sinks || d.proj_bias || d.rope_style || d.streams || d.loop_times > 1)
         return fail(rt, LUM_E_UNSUPPORTED, "block_kind 1: norm_kind 0 / 1, pos_kind 0 / 1, qk_norm 0 / 2, dist_bias 0 / 1; no tied head, experts, sinks, biases or rotation");
     const int kind = kind_of(d.weight_dtype), ek = kind_of(d.embed_dtype), CK = chunk_elems(kind), H = d.hidden;
     auto up = [](int n, int to) { return (n + to - 1) / to * to; };
@@ -1415,7 +1712,7 @@ int init_blocks(lum_rt* rt, lum_model_desc d, const lum_layer_desc* layers) {
     };
     auto part = [&](Tensor& t, void* base, int nt, int row0, int rows, int cols) {
         t = Tensor();
-        t.w = base; t.kind = kind; t.kc = kLayoutChunked; t.nt = nt; t.crow0 = (size_t)row0;
+        t.w = base; t.kind = kind; t.kc = kLayoutChunked; t.nt = nt; t.rm.row0 = (size_t)row0;
         t.rows = t.full_rows = (size_t)rows; t.cols = t.full_cols = t.kdev = (size_t)cols;
     };
     auto vec = [&](Tensor& t, int n) { return alloc_tensor(rt, t, WK_F32, 1, n, 1, n, 0, 0); };
@@ -1487,6 +1784,192 @@ int init_blocks(lum_rt* rt, lum_model_desc d, const lum_layer_desc* layers) {
     return 0;
 }
 
+// A decoder with one sublayer after the other (block_kind 2).
+int init_sequential(lum_rt* rt, lum_model_desc d, const lum_layer_desc* layers) {
+    if (d.tp_size <= 0) { d.tp_size = 1; d.tp_rank = 0; }
+    if (d.ep_size <= 0) { d.ep_size = 1; d.ep_rank = 0; }
+    if (d.max_batch <= 0) d.max_batch = 1;
+    if (d.max_new_tokens <= 0) d.max_new_tokens = 4096;
+    if (d.loop_times < 1) d.loop_times = 1;
+    if (d.tp_size != 1 || d.ep_size != 1 || rt->tp_size > 1) return fail(rt, LUM_E_UNSUPPORTED, "block_kind 2 runs on one GPU");
+    if (d.max_batch > 1024) return fail(rt, LUM_E_INVALID, "max_batch %d (at most 1024 sequences)", d.max_batch);
+    if (d.n_layers <= 0 || d.hidden <= 0 || d.vocab <= 0 || d.max_seq <= 0) return fail(rt, LUM_E_INVALID, "model dimensions must be positive");
+    auto dense = [](uint32_t t) { return t == LUM_F32 || t == LUM_BF16; };
+    if (!dense(d.weight_dtype) || !dense(d.embed_dtype) || !dense(d.kv_dtype)) return fail(rt, LUM_E_UNSUPPORTED, "block_kind 2: weights, embedding and cache must be F32 or BF16");
+    if ((d.norm_kind != 0 && d.norm_kind != 2) || d.pos_kind || d.qk_norm || d.dist_bias || d.tied_head || d.n_experts || d.attn_sinks || d.proj_bias || d.rope_style)
+        return fail(rt, LUM_E_UNSUPPORTED, "block_kind 2: norm_kind 0 / 2; positions, q / k norms and biases are chosen layer by layer; no tied head, experts or sinks");
+    if (d.streams < 0 || d.streams > kMaxStreams) return fail(rt, LUM_E_UNSUPPORTED, "%d residual streams (at most %d)", d.streams, kMaxStreams);
+    if (d.loop_times > 1 && (d.loop_start < 0 || d.loop_start > d.loop_stop || d.loop_stop > d.n_layers || (long long)d.loop_times * d.n_layers > 65536))
+        return fail(rt, LUM_E_INVALID, "layers %d .. %d of %d run %d times", d.loop_start, d.loop_stop, d.n_layers, d.loop_times);
+    const int kind = kind_of(d.weight_dtype), ek = kind_of(d.embed_dtype), CK = chunk_elems(kind), H = d.hidden;
+    auto up = [](int n, int to) { return (n + to - 1) / to * to; };
+    for (int l = 0; l < d.n_layers; l++) {
+        const lum_layer_desc& g = layers[l];
+        if (g.conv_taps < 0 || g.conv_taps > 64 || g.ffn < 0 || g.chunk < 0 || g.window < 0) return fail(rt, LUM_E_INVALID, "layer %d: negative sizes, or more than 64 taps", l);
+        if (g.ffn > 0 && g.ffn_kind != 1) return fail(rt, LUM_E_UNSUPPORTED, "layer %d: feed-forward kind %d (block_kind 2 has 1, the clamped gate)", l, g.ffn_kind);
+        if (g.mixer == 1) {
+            if (g.rec_width <= 0 || g.rec_blocks <= 0 || g.rec_width % g.rec_blocks) return fail(rt, LUM_E_INVALID, "layer %d: recurrence of width %d in %d blocks", l, g.rec_width, g.rec_blocks);
+            if (g.rec_width / g.rec_blocks > 3072) return fail(rt, LUM_E_UNSUPPORTED, "layer %d: a recurrence's block of %d channels is too large", l, g.rec_width / g.rec_blocks);
+        } else if (g.mixer == 0) {
+            if (g.n_q_heads <= 0 || g.n_kv_heads <= 0 || g.qk_dim <= 0 || g.v_dim <= 0 || g.n_q_heads % g.n_kv_heads)
+                return fail(rt, LUM_E_INVALID, "layer %d: sizes must be positive and the query heads a multiple of the K/V heads", l);
+            if (g.maps < 0 || g.maps > 2 || (g.chunk && g.window) || g.v_mix || g.rot_dims < 0 || g.rot_dims % 2 || g.rot_dims > g.qk_dim)
+                return fail(rt, LUM_E_UNSUPPORTED, "layer %d: at most two maps, chunk or window, no value mixing, an even number of rotated dimensions of the head", l);
+            if (!band_supported(g.n_q_heads, g.n_kv_heads, head_pad(g.qk_dim), head_pad(g.v_dim))) return fail(rt, LUM_E_UNSUPPORTED, "layer %d: head sizes %d / %d are too large", l, g.qk_dim, g.v_dim);
+        } else {
+            return fail(rt, LUM_E_UNSUPPORTED, "layer %d: mixer %d", l, g.mixer);
+        }
+    }
+    if (int r = setup_pages(rt, d)) return r;
+#define TRY(x) do { if (int r_ = (x)) { free_model(rt); return r_; } } while (0)
+    rt->nq_l = layers[0].n_q_heads; rt->nkv_l = layers[0].n_kv_heads; rt->ffn_l = layers[0].ffn; rt->vocab_l = d.vocab;
+    rt->ep_size = 1; rt->ep_rank = 0;
+    rt->h_chunks = up(H, CK) / CK; rt->ldx = up(H, 8); rt->head_nt = up(d.vocab, 8); rt->n_streams = d.streams > 0 ? d.streams : 1;
+    rt->ldq = rt->q_floats = rt->attn_chunks = rt->act_chunks = rt->vf_floats = rt->u_floats = rt->gate_floats = rt->rec_chunks = 0;
+    rt->x2 = rt->part = nullptr; rt->attn_part = nullptr;
+    auto zeroed = [&](void** p, size_t bytes) -> int {
+        if (int r = dev_alloc(rt, p, bytes)) return r;
+        cudaMemsetAsync(*p, 0, bytes ? bytes : 16, rt->stream);
+        return 0;
+    };
+    auto container = [&](void** p, int nt, int chunks) -> int { return zeroed(p, chunked_bytes((size_t)nt, (size_t)chunks)); };
+    auto part = [&](Tensor& t, void* base, int nt, RowMap rm, int rows, int cols) {
+        t = Tensor();
+        t.w = base; t.kind = kind; t.kc = kLayoutChunked; t.nt = nt; t.rm = rm;
+        t.rows = t.full_rows = (size_t)rows; t.cols = t.full_cols = t.kdev = (size_t)cols;
+    };
+    auto vec = [&](Tensor& t, int n) { return alloc_tensor(rt, t, WK_F32, 1, n, 1, n, 0, 0); };
+    auto range = [&](Tensor& t, float* base, size_t n) {       // a vector inside a larger one
+        t = Tensor();
+        t.w = base; t.kind = WK_F32; t.rows = t.full_rows = 1; t.cols = t.full_cols = t.kdev = n;
+    };
+    auto at = [](int row0) { return RowMap{(size_t)row0}; };
+    TRY(alloc_tensor(rt, rt->embed, ek, d.vocab, H, d.vocab, H, 0, 0));
+    TRY(vec(rt->final_norm, H));
+    {
+        void* base = nullptr;
+        TRY(container(&base, rt->head_nt, rt->h_chunks));
+        part(rt->lm_head, base, rt->head_nt, at(0), d.vocab, H);
+    }
+    auto most = [](int& a, int b) { if (b > a) a = b; };
+    struct Rot { int dims; float base; const float2* table; };
+    std::vector<Rot> rots;
+    const int runs = n_runs(d), HT = up(H, 8);
+    const size_t kv_elem = d.kv_dtype == LUM_BF16 ? 2 : 4;
+    rt->L.resize((size_t)runs);
+    for (int i = 0; i < runs; i++) {
+        LayerW& w = rt->L[(size_t)i];
+        const int li = layer_of_run(d, i);
+        if (first_run(d, li) != i) w = rt->L[(size_t)first_run(d, li)];      // the same weights again; caches and states of its own below
+        else {
+            w.g = layers[li];
+            w.index = li;
+            const lum_layer_desc& g = w.g;
+            const int F = g.ffn, taps = g.conv_taps;
+            if (g.mixer == 1) {
+                const int W = g.rec_width, B = g.rec_blocks, bw = W / B;
+                w.k_off = up(W, 8); w.nt_in = 2 * w.k_off; w.o_chunks = up(W, CK) / CK; w.ring_ch = W;
+                w.bwp = up(bw, 8); w.rec_kc = up(bw, CK) / CK; w.nt_rec = B * 2 * w.bwp;
+                TRY(container(&w.w_in, w.nt_in, rt->h_chunks));
+                part(w.rec_y, w.w_in, w.nt_in, at(0), W, H); part(w.rec_x, w.w_in, w.nt_in, at(w.k_off), W, H);
+                TRY(zeroed((void**)&w.in_bias, (size_t)w.nt_in * 4));
+                range(w.rec_y_b, w.in_bias, W); range(w.rec_x_b, w.in_bias + w.k_off, W);
+                TRY(container(&w.w_rec, w.nt_rec, w.rec_kc));
+                part(w.rec_ra, w.w_rec, w.nt_rec, RowMap{0, (size_t)bw, (size_t)(2 * w.bwp), 1}, W, bw);
+                part(w.rec_ri, w.w_rec, w.nt_rec, RowMap{(size_t)w.bwp, (size_t)bw, (size_t)(2 * w.bwp), 1}, W, bw);
+                TRY(vec(w.rec_ra_b, W)); TRY(vec(w.rec_ri_b, W)); TRY(vec(w.rec_lam, W));
+                if (taps) { TRY(vec(w.rec_conv, W * taps)); TRY(vec(w.rec_conv_b, W)); }
+                most(rt->u_floats, up(W, 8)); most(rt->gate_floats, w.nt_rec); most(rt->rec_chunks, B * w.rec_kc);
+            } else {
+                const int maps = g.maps > 1 ? g.maps : 1, qd = g.n_q_heads * maps * g.qk_dim, kd = g.n_kv_heads * maps * g.qk_dim, vd = g.n_kv_heads * g.v_dim, od = g.n_q_heads * g.v_dim;
+                w.dkp = head_pad(g.qk_dim); w.dvp = head_pad(g.v_dim);
+                w.k_off = up(qd, 8); w.v_off = w.k_off + up(kd, 8); w.nt_in = w.v_off + up(vd, 8); w.o_chunks = up(od, CK) / CK; w.ring_ch = w.nt_in;
+                TRY(container(&w.w_in, w.nt_in, rt->h_chunks));
+                part(w.q, w.w_in, w.nt_in, at(0), qd, H); part(w.k, w.w_in, w.nt_in, at(w.k_off), kd, H); part(w.v, w.w_in, w.nt_in, at(w.v_off), vd, H);
+                if (g.qkv_bias) {
+                    TRY(zeroed((void**)&w.in_bias, (size_t)w.nt_in * 4));
+                    range(w.q_b, w.in_bias, qd); range(w.k_b, w.in_bias + w.k_off, kd); range(w.v_b, w.in_bias + w.v_off, vd);
+                }
+                if (taps) {
+                    TRY(zeroed((void**)&w.in_conv, (size_t)w.nt_in * taps * 4));
+                    range(w.q_conv, w.in_conv, (size_t)qd * taps); range(w.k_conv, w.in_conv + (size_t)w.k_off * taps, (size_t)kd * taps);
+                    range(w.v_conv, w.in_conv + (size_t)w.v_off * taps, (size_t)vd * taps);
+                }
+                if (g.head_norm) { TRY(vec(w.q_norm, g.qk_dim)); TRY(vec(w.k_norm, g.qk_dim)); }
+                if (maps == 2) { TRY(vec(w.lq1, g.qk_dim)); TRY(vec(w.lk1, g.qk_dim)); TRY(vec(w.lq2, g.qk_dim)); TRY(vec(w.lk2, g.qk_dim)); }
+                if (g.rot_dims) {                              // cosine and sine of every position, angles in f64
+                    for (const Rot& r : rots) if (r.dims == g.rot_dims && r.base == g.rot_base) w.rot = r.table;
+                    if (!w.rot) {
+                        const int half = g.rot_dims / 2;
+                        std::vector<float2> t((size_t)d.max_seq * half);
+                        for (int k = 0; k < half; k++) {
+                            const double f = std::pow((double)g.rot_base, -2.0 * k / g.rot_dims);
+                            for (int p = 0; p < d.max_seq; p++) t[(size_t)p * half + k] = make_float2((float)std::cos(p * f), (float)std::sin(p * f));
+                        }
+                        TRY(dev_alloc(rt, (void**)&w.rot, t.size() * sizeof(float2)));
+                        cudaMemcpyAsync((void*)w.rot, t.data(), t.size() * sizeof(float2), cudaMemcpyHostToDevice, rt->stream);
+                        cudaStreamSynchronize(rt->stream);
+                        rots.push_back({g.rot_dims, g.rot_base, w.rot});
+                    }
+                }
+                w.k_elems = (size_t)g.n_kv_heads * maps * w.dkp; w.v_elems = (size_t)g.n_kv_heads * w.dvp;
+                most(rt->q_floats, g.n_q_heads * maps * w.dkp);
+            }
+            if (!taps) w.ring_ch = 0;
+            TRY(container(&w.w_o, HT, w.o_chunks));
+            part(w.o, w.w_o, HT, at(0), H, g.mixer == 1 ? g.rec_width : g.n_q_heads * g.v_dim);
+            TRY(vec(w.attn_norm, H));
+            if (F) {
+                w.nt_ff = 2 * up(F, 8); w.dn_chunks = up(F, CK) / CK;
+                TRY(container(&w.w_ff, w.nt_ff, rt->h_chunks));
+                part(w.gate, w.w_ff, w.nt_ff, RowMap{0, 0, 0, 2}, F, H); part(w.up, w.w_ff, w.nt_ff, RowMap{8, 0, 0, 2}, F, H);
+                TRY(container(&w.w_dn, HT, w.dn_chunks));
+                part(w.down, w.w_dn, HT, at(0), H, F);
+                TRY(vec(w.mlp_norm, H));
+            }
+            for (int q = 0; q < (F ? 2 : 1) && d.streams > 0; q++) { TRY(vec(w.hc_in[q], d.streams)); TRY(vec(w.hc_out[q], d.streams)); TRY(vec(w.hc_mix[q], d.streams * d.streams)); }
+            most(rt->ldq, w.nt_in); most(rt->attn_chunks, w.o_chunks); most(rt->act_chunks, w.dn_chunks);
+        }
+        TRY(zeroed(&w.kc, kv_rows_total(rt) * w.k_elems * kv_elem));
+        TRY(zeroed(&w.vc, kv_rows_total(rt) * w.v_elems * kv_elem));
+        w.ring = w.state = nullptr;
+        if (w.ring_floats()) TRY(zeroed((void**)&w.ring, (size_t)d.max_batch * w.ring_floats() * 4));
+        if (w.state_floats()) TRY(zeroed((void**)&w.state, (size_t)d.max_batch * w.state_floats() * 4));
+        rt->seq_state_bytes += (w.ring_floats() + w.state_floats()) * 4;
+    }
+    rt->qkv_floats = (size_t)rt->ldq; rt->attn_floats = (size_t)rt->attn_chunks * CK; rt->h_floats = (size_t)rt->act_chunks * CK;
+    TRY(zeroed((void**)&rt->x, (size_t)rt->n_streams * rt->ldx * 4));
+    TRY(zeroed((void**)&rt->u, (size_t)rt->ldx * 4));
+    TRY(zeroed((void**)&rt->qkv, rt->qkv_floats * 4));
+    TRY(zeroed((void**)&rt->attn, rt->attn_floats * 4));
+    TRY(zeroed((void**)&rt->h, rt->h_floats * 4));
+    TRY(alloc_decode_state(rt));
+#undef TRY
+    if (rt->seq_state_bytes) rt->seq_pos.assign((size_t)d.max_batch, 0);
+    rt->use_mega = 0; rt->mega_ok = false;
+    rt->has_model = true;
+    return 0;
+}
+
+// ---- the recurrent state of a sequence: rings of the short convolutions and states of the recurrences, run by run
+template <typename F>
+int for_seq_state(lum_rt* rt, int seq, F fn) {                 // fn(device pointer, bytes, offset in the saved form)
+    size_t off = 0;
+    for (const LayerW& w : rt->L) {
+        const size_t rb = w.ring_floats() * 4, sb = w.state_floats() * 4;
+        if (rb) if (int r = fn((char*)w.ring + (size_t)seq * rb, rb, off)) return r;
+        off += rb;
+        if (sb) if (int r = fn((char*)w.state + (size_t)seq * sb, sb, off)) return r;
+        off += sb;
+    }
+    return 0;
+}
+// A sequence with a state continues where it stands, or starts anew.
+int check_seq_pos(lum_rt* rt, int seq, int from, const char* who) {
+    if (rt->seq_pos.empty() || from == 0 || from == rt->seq_pos[(size_t)seq]) return 0;
+    return fail(rt, LUM_E_INVALID, "%s: position %d of sequence %d, whose state is at %d (layers with a state continue there, or from 0)", who, from, seq, rt->seq_pos[(size_t)seq]);
+}
+
 // Describe the loaded model to the persistent kernel; mega_ok says whether it can run it.
 int setup_mega(lum_rt* rt) {
     rt->mega_ok = false;
@@ -1551,7 +2034,7 @@ int lum_internal_weight_view(lum_rt* rt, int slot, int layer, lum::WeightView* o
     if (!rt || !rt->has_model) return 1;
     Tensor* t = slot_tensor(rt, slot, layer);
     if (!t || !t->w) return 1;
-    *out = {t->w, t->s, t->kind, t->kc, t->rows, t->cols, t->kdev, t->row0, t->col0, t->full_rows, t->full_cols, rt->cfg.device, rt->stream, t->nt, t->crow0};
+    *out = {t->w, t->s, t->kind, t->kc, t->rows, t->cols, t->kdev, t->row0, t->col0, t->full_rows, t->full_cols, rt->cfg.device, rt->stream, t->nt, t->rm};
     return 0;
 }
 int lum_internal_label_style(lum_rt* rt) { return rt->d.block_kind; }
@@ -1917,7 +2400,7 @@ int32_t lum_profile_llir(lum_rt* rt, const uint8_t* blob, size_t size, uint64_t 
 
 static int kv_check(lum_rt* rt, int32_t layer, int32_t kind, int32_t rows, size_t bytes, const char* who) {
     if (!rt || !rt->has_model) return fail(rt, LUM_E_INVALID, "%s: no model", who);
-    if (layer < 0 || layer >= rt->d.n_layers || rows < 0 || rows > rt->d.max_seq || (kind != 0 && kind != 1)) return fail(rt, LUM_E_INVALID, "%s: bad layer / kind / rows", who);
+    if (layer < 0 || layer >= (int)rt->L.size() || rows < 0 || rows > rt->d.max_seq || (kind != 0 && kind != 1)) return fail(rt, LUM_E_INVALID, "%s: bad layer / kind / rows", who);
     const size_t want = (size_t)rows * kv_row_bytes(rt, rt->L[(size_t)layer], kind);
     if (bytes != want) return fail(rt, LUM_E_INVALID, "%s: %d rows are %zu bytes in the cache's own type, got %zu", who, rows, want, bytes);
     return 0;
@@ -1954,6 +2437,16 @@ int32_t lum_kv_copy(lum_rt* rt, int32_t src_seq, int32_t dst_seq, int32_t rows) 
         return fail(rt, LUM_E_INVALID, "kv_copy: sequences %d -> %d of %d, %d rows of %d", src_seq, dst_seq, rt->max_batch, rows, rt->d.max_seq);
     if (src_seq == dst_seq || rows == 0) return 0;
     CU(rt, cudaSetDevice(rt->cfg.device));
+    if (!rt->seq_pos.empty()) {
+        if (rt->seq_pos[(size_t)src_seq] != rows)
+            return fail(rt, LUM_E_INVALID, "kv_copy: %d rows of sequence %d, whose state is at %d (layers with a state are copied as they stand)", rows, src_seq, rt->seq_pos[(size_t)src_seq]);
+        for (const LayerW& w : rt->L) {
+            const size_t rf = w.ring_floats(), sf = w.state_floats();
+            if (rf) CU(rt, cudaMemcpyAsync(w.ring + dst_seq * rf, w.ring + src_seq * rf, rf * 4, cudaMemcpyDeviceToDevice, rt->stream));
+            if (sf) CU(rt, cudaMemcpyAsync(w.state + dst_seq * sf, w.state + src_seq * sf, sf * 4, cudaMemcpyDeviceToDevice, rt->stream));
+        }
+        rt->seq_pos[(size_t)dst_seq] = rows;
+    }
     if (rt->page_rows) {
         // whole pages of the prefix are shared (whoever writes into one first gets a copy of its own, see kv_ensure); the rows of the
         // last, partial page are copied into a page of dst's own
@@ -1990,7 +2483,38 @@ int32_t lum_kv_copy(lum_rt* rt, int32_t src_seq, int32_t dst_seq, int32_t rows) 
 int32_t lum_kv_release(lum_rt* rt, int32_t seq) {
     if (!rt || !rt->has_model) return fail(rt, LUM_E_INVALID, "kv_release: no model");
     if (seq < 0 || seq >= rt->max_batch) return fail(rt, LUM_E_INVALID, "kv_release: sequence %d outside max_batch %d", seq, rt->max_batch);
+    if (!rt->seq_pos.empty()) rt->seq_pos[(size_t)seq] = 0;      // (a state starts from zero at position 0, whatever the slot holds)
     if (rt->page_rows) kv_release_seq(rt, seq);      // the device table keeps stale entries: nothing reads rows of a sequence that has none
+    return 0;
+}
+
+int32_t lum_state_bytes(const lum_rt* rt, size_t* bytes) {
+    if (!rt || !rt->has_model || !bytes) return LUM_E_INVALID;
+    *bytes = rt->seq_state_bytes;
+    return 0;
+}
+int32_t lum_state_save(lum_rt* rt, void* host_out, size_t bytes, int32_t* position) {
+    if (!rt || !rt->has_model || (!host_out && bytes) || !position) return fail(rt, LUM_E_INVALID, "state_save: no model or null output");
+    if (bytes != rt->seq_state_bytes) return fail(rt, LUM_E_INVALID, "state_save: a sequence's state is %zu bytes, got %zu", rt->seq_state_bytes, bytes);
+    CU(rt, cudaSetDevice(rt->cfg.device));
+    *position = rt->seq_pos.empty() ? 0 : rt->seq_pos[(size_t)rt->cur_seq];
+    if (int r = for_seq_state(rt, rt->cur_seq, [&](char* dev, size_t n, size_t off) -> int {
+            CU(rt, cudaMemcpyAsync((char*)host_out + off, dev, n, cudaMemcpyDeviceToHost, rt->stream));
+            return 0;
+        })) return r;
+    CU(rt, cudaStreamSynchronize(rt->stream));
+    return 0;
+}
+int32_t lum_state_load(lum_rt* rt, const void* host, size_t bytes, int32_t position) {
+    if (!rt || !rt->has_model || (!host && bytes)) return fail(rt, LUM_E_INVALID, "state_load: no model or null input");
+    if (bytes != rt->seq_state_bytes || position < 0 || position > rt->d.max_seq) return fail(rt, LUM_E_INVALID, "state_load: a sequence's state is %zu bytes, got %zu; position %d of %d", rt->seq_state_bytes, bytes, position, rt->d.max_seq);
+    CU(rt, cudaSetDevice(rt->cfg.device));
+    if (int r = for_seq_state(rt, rt->cur_seq, [&](char* dev, size_t n, size_t off) -> int {
+            CU(rt, cudaMemcpyAsync(dev, (const char*)host + off, n, cudaMemcpyHostToDevice, rt->stream));
+            return 0;
+        })) return r;
+    CU(rt, cudaStreamSynchronize(rt->stream));
+    if (!rt->seq_pos.empty()) rt->seq_pos[(size_t)rt->cur_seq] = position;
     return 0;
 }
 
@@ -2086,6 +2610,7 @@ int32_t lum_batch_begin_slots(lum_rt* rt, int32_t n_seq, const int32_t* slots, c
         if (taken[(size_t)sl]) return fail(rt, LUM_E_INVALID, "batch_begin: cache slot %d named twice", sl);
         taken[(size_t)sl] = 1;
         row_slot[(size_t)i] = sl;
+        if (int r = check_seq_pos(rt, sl, positions[i], "batch_begin")) return r;
     }
     CU(rt, cudaSetDevice(rt->cfg.device));
     if (int r = ensure_rows(rt, n_seq)) return r;
@@ -2110,6 +2635,7 @@ int32_t lum_batch_decode(lum_rt* rt, int32_t n_steps) {
     for (int i = 0; i < rt->batch_n; i++) {
         if (int r = kv_ensure(rt, rt->rows.h_slot[(size_t)i], rt->rows.h_pos[(size_t)i], rt->rows.h_pos[(size_t)i] + n_steps)) return r;
         rt->rows.h_pos[(size_t)i] += n_steps;
+        if (!rt->seq_pos.empty()) rt->seq_pos[(size_t)rt->rows.h_slot[(size_t)i]] = rt->rows.h_pos[(size_t)i];
     }
     const int M = rt->batch_n;
     if (rt->cfg.use_graph && (!rt->g_batch || rt->g_batch_n != M)) {
@@ -2452,7 +2978,7 @@ int32_t lum_model_init_layers(lum_rt* rt, const lum_model_desc* dp, const lum_la
     free_model(rt);
     if (rt->generic) { lum_generic_free(rt->generic); rt->generic = nullptr; }
     if (rt->llir) { lum_llir_free_plan(rt->llir); rt->llir = nullptr; }             // no graph stands behind this model
-    return init_blocks(rt, *dp, layers);
+    return dp->block_kind == 2 ? init_sequential(rt, *dp, layers) : init_blocks(rt, *dp, layers);
 }
 
 int32_t lum_model_synth(lum_rt* rt, uint64_t seed) {
@@ -2468,7 +2994,7 @@ int32_t lum_model_synth(lum_rt* rt, uint64_t seed) {
             void* tmp = nullptr;
             if (cudaMalloc(&tmp, t->rows * t->cols * (t->kind == WK_BF16 ? 2 : 4) + 64) != cudaSuccess) return fail(rt, LUM_E_NOMEM, "synth: staging buffer");
             e = launch_synth_normal(seed, tid, tmp, t->kind, t->rows, t->cols, 0, 0, t->cols, ones, rt->stream);
-            if (e == cudaSuccess) e = launch_chunked_pack(tmp, (uint32_t)t->kind, t->rows, t->cols, t->w, t->kind, t->nt, t->crow0, rt->stream);
+            if (e == cudaSuccess) e = launch_chunked_pack(tmp, (uint32_t)t->kind, t->rows, t->cols, t->w, t->kind, t->nt, t->rm, rt->stream);
             cudaStreamSynchronize(rt->stream);
             cudaFree(tmp);
         }
@@ -2484,9 +3010,12 @@ int32_t lum_model_synth(lum_rt* rt, uint64_t seed) {
     for (int l = 0; l < d.n_layers; l++) {
         const int lin[] = {LUM_S_Q, LUM_S_K, LUM_S_V, LUM_S_O, LUM_S_GATE, LUM_S_UP, LUM_S_DOWN, LUM_S_ROUTER, LUM_S_ROUTER_BIAS, LUM_S_EXP_GATE_UP,
                            LUM_S_EXP_GATE_UP_BIAS, LUM_S_EXP_DOWN, LUM_S_EXP_DOWN_BIAS, LUM_S_Q_BIAS, LUM_S_K_BIAS, LUM_S_V_BIAS, LUM_S_O_BIAS, LUM_S_SINKS,
-                           LUM_S_ATTN_NORM_BIAS, LUM_S_V_MIX, LUM_S_ACT};
+                           LUM_S_ATTN_NORM_BIAS, LUM_S_V_MIX, LUM_S_ACT, LUM_S_LQ1, LUM_S_LK1, LUM_S_LQ2, LUM_S_LK2, LUM_S_HC1_MIX, LUM_S_HC2_MIX, LUM_S_Q_CONV, LUM_S_K_CONV,
+                           LUM_S_V_CONV, LUM_S_REC_Y, LUM_S_REC_Y_BIAS, LUM_S_REC_X, LUM_S_REC_X_BIAS, LUM_S_REC_CONV, LUM_S_REC_CONV_BIAS, LUM_S_REC_RA,
+                           LUM_S_REC_RA_BIAS, LUM_S_REC_RI, LUM_S_REC_RI_BIAS, LUM_S_REC_LAM};
         for (int s : lin) if (int r = fill(s, l, 0)) return r;
-        const int nrm[] = {LUM_S_ATTN_NORM, LUM_S_MLP_NORM, LUM_S_Q_NORM, LUM_S_K_NORM, LUM_S_TEMP, LUM_S_DIST_R1, LUM_S_DIST_R2};
+        const int nrm[] = {LUM_S_ATTN_NORM, LUM_S_MLP_NORM, LUM_S_Q_NORM, LUM_S_K_NORM, LUM_S_TEMP, LUM_S_DIST_R1, LUM_S_DIST_R2,
+                           LUM_S_HC1_IN, LUM_S_HC1_OUT, LUM_S_HC2_IN, LUM_S_HC2_OUT};
         for (int s : nrm) if (int r = fill(s, l, 1)) return r;
     }
     CU(rt, cudaStreamSynchronize(rt->stream));
@@ -2505,7 +3034,7 @@ int32_t lum_model_get_weight_f32(lum_rt* rt, int32_t slot, int32_t layer, size_t
     cudaError_t e = cudaMalloc((void**)&tmp, (chunked ? t->rows * t->cols : n) * 4 + 16);
     if (e != cudaSuccess) return fail(rt, LUM_E_NOMEM, "get_weight: %s", cudaGetErrorString(e));
     if (chunked) {
-        e = launch_chunked_unpack(t->w, t->kind, t->nt, t->crow0, t->rows, t->cols, tmp, nullptr, rt->stream);
+        e = launch_chunked_unpack(t->w, t->kind, t->nt, t->rm, t->rows, t->cols, tmp, nullptr, rt->stream);
         if (e == cudaSuccess) e = cudaMemcpyAsync(host_out, tmp + offset, n * 4, cudaMemcpyDeviceToHost, rt->stream);
         if (e == cudaSuccess) e = cudaStreamSynchronize(rt->stream);
         cudaFree(tmp);
@@ -2528,6 +3057,11 @@ int32_t lum_model_weight_bytes(const lum_rt* rt, uint64_t* bytes) {
         b += w.attn_norm.bytes() + w.mlp_norm.bytes();
         if (rt->d.qk_norm) b += w.q_norm.bytes() + w.k_norm.bytes();
         b += w.attn_norm_b.bytes() + w.v_mix.bytes() + w.temp.bytes() + w.dist_r1.bytes() + w.dist_r2.bytes() + w.act_par.bytes();
+        if (rt->d.block_kind == 2) {
+            const Tensor* ts[] = {&w.rec_y, &w.rec_x, &w.rec_ra, &w.rec_ri, &w.rec_y_b, &w.rec_x_b, &w.rec_ra_b, &w.rec_ri_b, &w.rec_conv, &w.rec_conv_b, &w.rec_lam, &w.q_b, &w.k_b, &w.v_b,
+                                  &w.q_conv, &w.k_conv, &w.v_conv, &w.q_norm, &w.k_norm};
+            for (const Tensor* t : ts) b += t->bytes();
+        }
         if (rt->d.n_experts > 0) {
             // a token reads the router and top_k experts (gate_up + down, their biases)
             const uint64_t H = (uint64_t)rt->d.hidden, F = (uint64_t)rt->d.ffn, eb = rt->embed.kind == WK_BF16 ? 2 : 4;
@@ -2547,6 +3081,7 @@ int32_t lum_kv_reset(lum_rt* rt) {
     CU(rt, cudaSetDevice(rt->cfg.device));
     if (rt->page_rows) for (int sq = 0; sq < rt->max_batch; sq++) kv_release_seq(rt, sq);
     rt->h_next_pos = 0;
+    rt->seq_pos.assign(rt->seq_pos.size(), 0);
     for (LayerW& w : rt->L) {       // every sequence
         CU(rt, cudaMemsetAsync(w.kc, 0, kv_rows_total(rt) * kv_row_bytes(rt, w, 0), rt->stream));
         CU(rt, cudaMemsetAsync(w.vc, 0, kv_rows_total(rt) * kv_row_bytes(rt, w, 1), rt->stream));
@@ -2557,7 +3092,7 @@ int32_t lum_kv_reset(lum_rt* rt) {
 
 int32_t lum_kv_read(lum_rt* rt, int32_t layer, int32_t kind, int32_t rows, float* host_out) {
     if (!rt || !rt->has_model || !host_out) return fail(rt, LUM_E_INVALID, "kv_read: no model or null output");
-    if (layer < 0 || layer >= rt->d.n_layers || rows < 0 || rows > rt->d.max_seq || (kind != 0 && kind != 1)) return fail(rt, LUM_E_INVALID, "kv_read: bad layer/kind/rows");
+    if (layer < 0 || layer >= (int)rt->L.size() || rows < 0 || rows > rt->d.max_seq || (kind != 0 && kind != 1)) return fail(rt, LUM_E_INVALID, "kv_read: bad layer/kind/rows");
     CU(rt, cudaSetDevice(rt->cfg.device));
     const size_t row_elems = kv_row_elems(rt->L[(size_t)layer], kind), n = (size_t)rows * row_elems;
     if (!n) return 0;
@@ -2705,6 +3240,9 @@ int32_t lum_profile(lum_rt* rt, int32_t trials, double* usec, char* display, siz
     CU(rt, cudaStreamSynchronize(rt->stream));
     if (saved.pos + trials + 1 > rt->d.max_seq) return fail(rt, LUM_E_INVALID, "profile: not enough cache capacity left for %d trial steps", trials);
     rt->h_next_pos = saved.pos;
+    std::vector<char> seq_state(rt->seq_state_bytes);          // the trial steps move the sequence's state on: put it back afterwards
+    int32_t seq_at = 0;
+    if (!seq_state.empty()) if (int r = lum_state_save(rt, seq_state.data(), seq_state.size(), &seq_at)) return r;
     cudaEvent_t e0, e1;
     CU(rt, cudaEventCreate(&e0));
     CU(rt, cudaEventCreate(&e1));
@@ -2723,12 +3261,13 @@ int32_t lum_profile(lum_rt* rt, int32_t trials, double* usec, char* display, siz
     rt->h_next_pos = saved.pos;
     cudaMemcpyAsync(rt->state, &saved, sizeof saved, cudaMemcpyHostToDevice, rt->stream);
     cudaStreamSynchronize(rt->stream);
+    if (!seq_state.empty()) if (int r2 = lum_state_load(rt, seq_state.data(), seq_state.size(), seq_at)) return r2;
     if (r) return r;
     if (int s = check_status(rt)) return s;
     const double us = (double)ms * 1000.0 / trials;
     rt->last_profile_usec = us;
     if (usec) *usec = us;
-    if (display && display_len && rt->d.block_kind == 1) snprintf(display, display_len, "%.3f ms/token", us / 1000.0);
+    if (display && display_len && rt->d.block_kind != 0) snprintf(display, display_len, "%.3f ms/token", us / 1000.0);
     else if (display && display_len)
         snprintf(display, display_len, "%.3f ms/token; attention: %d splits per KV head, %s merge", us / 1000.0, rt->n_splits,
                  rt->n_splits < 2 ? "no" : rt->attn_cluster ? "cluster" : "ticket");

@@ -51,7 +51,7 @@ public:
     ~B200Runtime() { if (h_) lum_destroy(h_); }
 
     void load_model(const lum_model_desc& d) { ck(lum_model_init(h_, &d)); desc_ = d; }
-    // a decoder whose layers are described one by one (block_kind 1)
+    // a decoder whose layers are described one by one (block_kind 1 or 2)
     void load_model(const lum_model_desc& d, const std::vector<lum_layer_desc>& layers) {
         if ((int)layers.size() != d.n_layers) throw Error(LUM_E_INVALID, "load_model: one descriptor per layer");
         ck(lum_model_init_layers(h_, &d, layers.data()));
@@ -109,6 +109,15 @@ public:
     void seq_select(int seq) { ck(lum_seq_select(h_, seq)); }
     void kv_copy(int src_seq, int dst_seq, int rows) { ck(lum_kv_copy(h_, src_seq, dst_seq, rows)); }
     void kv_release(int seq) { ck(lum_kv_release(h_, seq)); }                       // paged cache: pages back to the pool
+    // layers with a state: the selected sequence's, whole (empty without one), and the tokens it has seen
+    std::vector<uint8_t> state_save(int* position) {
+        size_t n = 0;
+        ck(lum_state_bytes(h_, &n));
+        std::vector<uint8_t> out(n);
+        ck(lum_state_save(h_, out.data(), n, position));
+        return out;
+    }
+    void state_load(const std::vector<uint8_t>& data, int position) { ck(lum_state_load(h_, data.data(), data.size(), position)); }
     struct KvPool { int32_t pages_total, pages_free, page_rows; };
     KvPool kv_pool() const { KvPool p{0, 0, 0}; lum_kv_pool(h_, &p.pages_total, &p.pages_free, &p.page_rows); return p; }
     void batch_begin_slots(const std::vector<int32_t>& slots, const std::vector<int32_t>& tokens, const std::vector<int32_t>& positions) {

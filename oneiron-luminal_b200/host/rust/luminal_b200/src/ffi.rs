@@ -119,6 +119,11 @@ pub struct lum_model_desc {
     pub dist_bias: i32,
     pub residual_mult: f32,
     pub logit_scale: f32,
+    pub streams: i32,
+    pub loop_start: i32,
+    pub loop_stop: i32,
+    pub loop_times: i32,
+    pub embed_scale: f32,
 }
 
 #[repr(C)]
@@ -132,6 +137,19 @@ pub struct lum_layer_desc {
     pub v_mix: i32,
     pub ffn: i32,
     pub scale: f32,
+    pub mixer: i32,
+    pub chunk: i32,
+    pub conv_taps: i32,
+    pub maps: i32,
+    pub head_norm: i32,
+    pub qkv_bias: i32,
+    pub rot_dims: i32,
+    pub rec_width: i32,
+    pub rec_blocks: i32,
+    pub ffn_kind: i32,
+    pub rot_base: f32,
+    pub diff: f32,
+    pub ffn_limit: f32,
 }
 
 #[repr(C)]
@@ -191,6 +209,9 @@ unsafe extern "C" {
     pub fn lum_kv_load(rt: *mut lum_rt, layer: i32, kind: i32, rows: i32, host: *const c_void, bytes: usize) -> i32;
     pub fn lum_kv_copy(rt: *mut lum_rt, src_seq: i32, dst_seq: i32, rows: i32) -> i32;
     pub fn lum_kv_release(rt: *mut lum_rt, seq: i32) -> i32;
+    pub fn lum_state_bytes(rt: *const lum_rt, bytes: *mut usize) -> i32;
+    pub fn lum_state_save(rt: *mut lum_rt, host_out: *mut c_void, bytes: usize, position: *mut i32) -> i32;
+    pub fn lum_state_load(rt: *mut lum_rt, host: *const c_void, bytes: usize, position: i32) -> i32;
     pub fn lum_kv_pool(rt: *const lum_rt, pages_total: *mut i32, pages_free: *mut i32, page_rows: *mut i32) -> i32;
 
     pub fn lum_set_dim(rt: *mut lum_rt, dim: c_char, value: u64) -> i32;

@@ -186,6 +186,17 @@ impl B200Runtime {
     pub fn kv_copy(&mut self, src_seq: usize, dst_seq: usize, rows: usize) {
         self.check(unsafe { lum_kv_copy(self.h, src_seq as i32, dst_seq as i32, rows as i32) })
     }
+    /// Layers with a state: the selected sequence's, whole (empty without one), and the tokens it has seen.
+    pub fn state_save(&mut self) -> (Vec<u8>, i32) {
+        let (mut n, mut pos) = (0usize, 0i32);
+        self.check(unsafe { lum_state_bytes(self.h, &mut n) });
+        let mut out = vec![0u8; n];
+        self.check(unsafe { lum_state_save(self.h, out.as_mut_ptr() as *mut c_void, n, &mut pos) });
+        (out, pos)
+    }
+    pub fn state_load(&mut self, data: &[u8], position: i32) {
+        self.check(unsafe { lum_state_load(self.h, data.as_ptr() as *const c_void, data.len(), position) })
+    }
     /// Paged cache (`kv_page_rows` > 0): a finished sequence's pages go back to the pool; (pages, free pages, rows per page).
     pub fn kv_release(&mut self, seq: usize) { self.check(unsafe { lum_kv_release(self.h, seq as i32) }) }
     pub fn kv_pool(&self) -> (i32, i32, i32) {

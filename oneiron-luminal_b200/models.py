@@ -11,7 +11,7 @@ import os
 from dataclasses import dataclass
 from typing import Callable, Dict, List, Optional, Union
 
-from .runtime import DTYPE, LayerDesc, ModelDesc, _desc
+from .runtime import DTYPE, LayerDesc, ModelDesc, _desc, layer_order
 
 
 @dataclass
@@ -23,6 +23,8 @@ class ModelSpec:
     def tensor_names(self) -> List[str]:
         """Labels of the tensors a checkpoint of this model must hold (models with per-layer descriptors)."""
         d = self.desc
+        if d.block_kind == 2:
+            return self._sequential_names()
         top = ["embed", "final.norm", "head"] + (["final.norm.b"] if d.norm_kind == 1 else [])
         out = list(top)
         for i, g in enumerate(self.layers or []):
@@ -40,9 +42,37 @@ class ModelSpec:
             out += [f"l{i}.{n}" for n in names]
         return out
 
+    def _sequential_names(self) -> List[str]:
+        out = ["embed", "final.norm", "head"]
+        for i, g in enumerate(self.layers or []):
+            if g.mixer == 1:
+                names = ["mix." + n for n in ("y", "y.b", "x", "x.b", "ra", "ra.b", "ri", "ri.b", "lam", "o")]
+                names += ["mix.conv", "mix.conv.b"] if g.conv_taps else []
+            else:
+                names = ["mix." + n for n in ("q", "k", "v", "o")]
+                names += [f"mix.{c}.b" for c in "qkv"] if g.qkv_bias else []
+                names += [f"mix.{c}.conv" for c in "qkv"] if g.conv_taps else []
+                names += ["mix.q.norm", "mix.k.norm"] if g.head_norm else []
+                names += ["mix.lq1", "mix.lk1", "mix.lq2", "mix.lk2"] if g.maps == 2 else []
+            names += ["norm1"] + (["norm2", "mlp.gate", "mlp.up", "mlp.down"] if g.ffn else [])
+            if self.desc.streams:
+                names += [f"hc{q}.{n}" for q in ((1, 2) if g.ffn else (1,)) for n in ("in", "out", "mix")]
+            out += [f"l{i}.{n}" for n in names]
+        return out
+
     def weight_elems_per_token(self) -> int:
         """Elements of the linear weights one decode step streams."""
         d, n = self.desc, self.desc.vocab * self.desc.hidden
+        if d.block_kind == 2:
+            for i in layer_order(d, len(self.layers)):
+                g = self.layers[i]
+                n += 3 * d.hidden * g.ffn
+                if g.mixer == 1:
+                    n += 3 * d.hidden * g.rec_width + 2 * g.rec_width * (g.rec_width // g.rec_blocks)
+                else:
+                    m = max(1, g.maps)
+                    n += d.hidden * (m * g.qk_dim * (g.n_q_heads + g.n_kv_heads) + g.n_kv_heads * g.v_dim + g.n_q_heads * g.v_dim)
+            return n
         for g in self.layers or []:
             n += d.hidden * (g.n_q_heads * g.qk_dim + g.n_kv_heads * (g.qk_dim + g.v_dim) + g.n_q_heads * g.v_dim + 2 * g.ffn)
         return n
@@ -110,3 +140,47 @@ def madipel(cfg: dict, dtype: int) -> ModelSpec:
                  weight_dtype=dtype, embed_dtype=dtype, kv_dtype=dtype, block_kind=1, norm_kind=1, pos_kind=1, dist_bias=1,
                  residual_mult=float(cfg["residual_mult"]), logit_scale=float(cfg["logit_scale"]))
     return ModelSpec("Madipel", desc, layers)
+
+
+@register("Redenex")
+def redenex(cfg: dict, dtype: int) -> ModelSpec:
+    """Sequential sublayers over several residual streams: gated linear recurrences and differential attention in chunks (short
+    convolutions, per-head q / k norms, rotation of part of a head), clamped gated feed-forwards, and a loop over some of the layers."""
+    layers: List[LayerDesc] = []
+    width = _int(cfg, "width", "config")
+    for i, layer in enumerate(cfg["layers"]):
+        where = f"layers[{i}]"
+        mx, mlp = layer["mixer"], layer.get("mlp")
+        g = LayerDesc(conv_taps=_int(mx, "conv", where) if mx.get("conv") else 0)
+        if layer.get("type") == "rglru":
+            g.mixer, g.rec_width, g.rec_blocks = 1, _int(mx, "width", where), _int(mx, "blocks", where)
+            if g.rec_width % g.rec_blocks:
+                raise ValueError(f"{where}: width {g.rec_width} does not divide into {g.rec_blocks} blocks")
+        elif layer.get("type") == "attention":
+            g.n_q_heads, g.n_kv_heads = _int(mx, "heads", where), _int(mx, "kv_heads", where)
+            if g.n_q_heads % g.n_kv_heads:
+                raise ValueError(f"{where}: {g.n_q_heads} query heads are not a multiple of {g.n_kv_heads} K/V heads")
+            g.qk_dim, g.v_dim, g.scale = _int(mx, "dim", where), _int(mx, "vdim", where), float(mx["scale"])
+            g.maps, g.diff, g.head_norm, g.qkv_bias = 2, float(mx["diff"]), 1, 1
+            g.chunk = _int(mx["mask"], "size", where + ".mask") if mx.get("mask") else 0
+            if mx.get("rot"):
+                g.rot_dims, g.rot_base = _int(mx["rot"], "dims", where + ".rot"), float(mx["rot"]["base"])
+                if g.rot_dims % 2 or g.rot_dims > g.qk_dim:
+                    raise ValueError(f"{where}: {g.rot_dims} rotated dimensions of {g.qk_dim}")
+        else:
+            raise ValueError(f"{where}: type {layer.get('type')!r} (this design has attention and rglru layers)")
+        if mlp is not None:
+            if mlp.get("kind") != "dense":
+                raise ValueError(f"{where}: feed-forward kind {mlp.get('kind')!r} (this design has dense ones)")
+            g.ffn, g.ffn_kind, g.ffn_limit = _int(mlp, "ff", where), 1, float(mlp["limit"])
+        layers.append(g)
+    if not layers:
+        raise ValueError("a model needs at least one layer")
+    loop = cfg.get("loop") or {"start": 0, "stop": 0, "times": 1}
+    if not (0 <= loop["start"] <= loop["stop"] <= len(layers)) or loop["times"] < 1:
+        raise ValueError(f"loop {loop!r} over {len(layers)} layers")
+    desc = _desc(n_layers=len(layers), hidden=width, vocab=_int(cfg, "vocab", "config"), rms_eps=float(cfg["norm"]["eps"]), rope_theta=10000.0,
+                 weight_dtype=dtype, embed_dtype=dtype, kv_dtype=dtype, block_kind=2, norm_kind=2, residual_mult=1.0, logit_scale=1.0,
+                 streams=_int(cfg, "streams", "config"), embed_scale=float(cfg["embedding"]["scale"]),
+                 loop_start=loop["start"], loop_stop=loop["stop"], loop_times=loop["times"])
+    return ModelSpec("Redenex", desc, layers)

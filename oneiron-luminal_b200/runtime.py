@@ -34,6 +34,9 @@ SLOT = {
     "q_bias": 14, "k_bias": 15, "v_bias": 16, "o_bias": 17, "sinks": 18, "router": 19, "router_bias": 20,
     "exp_gate_up": 21, "exp_gate_up_bias": 22, "exp_down": 23, "exp_down_bias": 24,
     "attn_norm_bias": 25, "final_norm_bias": 26, "v_mix": 27, "temp": 28, "dist_r1": 29, "dist_r2": 30, "act": 31,
+    "q_conv": 32, "k_conv": 33, "v_conv": 34, "lq1": 35, "lk1": 36, "lq2": 37, "lk2": 38, "hc1_in": 39, "hc1_out": 40, "hc1_mix": 41,
+    "hc2_in": 42, "hc2_out": 43, "hc2_mix": 44, "rec_y": 45, "rec_y_bias": 46, "rec_x": 47, "rec_x_bias": 48, "rec_conv": 49,
+    "rec_conv_bias": 50, "rec_ra": 51, "rec_ra_bias": 52, "rec_ri": 53, "rec_ri_bias": 54, "rec_lam": 55,
 }
 
 
@@ -58,6 +61,7 @@ class ModelDesc(C.Structure):
         ("kv_page_rows", C.c_int32), ("kv_pool_pages", C.c_int32),
         ("block_kind", C.c_int32), ("norm_kind", C.c_int32), ("pos_kind", C.c_int32), ("dist_bias", C.c_int32),
         ("residual_mult", C.c_float), ("logit_scale", C.c_float),
+        ("streams", C.c_int32), ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32), ("embed_scale", C.c_float),
     ]
 
     def copy(self, **kw) -> "ModelDesc":
@@ -72,7 +76,17 @@ class LayerDesc(C.Structure):
     """Mirror of ``lum_layer_desc`` (include/lum_b200.h): one layer of a model whose layers are described one by one."""
 
     _fields_ = [("n_q_heads", C.c_int32), ("n_kv_heads", C.c_int32), ("qk_dim", C.c_int32), ("v_dim", C.c_int32),
-                ("window", C.c_int32), ("v_mix", C.c_int32), ("ffn", C.c_int32), ("scale", C.c_float)]
+                ("window", C.c_int32), ("v_mix", C.c_int32), ("ffn", C.c_int32), ("scale", C.c_float),
+                ("mixer", C.c_int32), ("chunk", C.c_int32), ("conv_taps", C.c_int32), ("maps", C.c_int32), ("head_norm", C.c_int32),
+                ("qkv_bias", C.c_int32), ("rot_dims", C.c_int32), ("rec_width", C.c_int32), ("rec_blocks", C.c_int32), ("ffn_kind", C.c_int32),
+                ("rot_base", C.c_float), ("diff", C.c_float), ("ffn_limit", C.c_float)]
+
+
+def layer_order(d: ModelDesc, n_layers: int) -> List[int]:
+    """The layers in the order they run (a loop of layers runs several times)."""
+    if d.loop_times <= 1:
+        return list(range(n_layers))
+    return list(range(d.loop_stop)) + list(range(d.loop_start, d.loop_stop)) * (d.loop_times - 1) + list(range(d.loop_stop, n_layers))
 
 
 class Stats(C.Structure):
@@ -229,6 +243,9 @@ def load_library() -> C.CDLL:
         "lum_kv_copy": (i32, [vp, i32, i32, i32]),
         "lum_kv_release": (i32, [vp, i32]),
         "lum_kv_pool": (i32, [vp, P(i32), P(i32), P(i32)]),
+        "lum_state_bytes": (i32, [vp, P(sz)]),
+        "lum_state_save": (i32, [vp, vp, sz, P(i32)]),
+        "lum_state_load": (i32, [vp, vp, sz, i32]),
         "lum_set_sampling": (i32, [vp, P(Sampling)]),
         "lum_op_sample_topk": (i32, [vp, i32, i32, P(Sampling), i32, vp, vp, vp]),
         "lum_get_stats": (i32, [vp, P(Stats)]),
@@ -472,7 +489,7 @@ class B200Runtime:
 
     # ---- model -----------------------------------------------------------------------------------
     def load_model(self, desc: ModelDesc, layers: Optional[Sequence[LayerDesc]] = None) -> None:
-        """``layers``: one descriptor per layer for models with ``block_kind`` 1 (see ``models.from_config``)."""
+        """``layers``: one descriptor per layer for models with ``block_kind`` 1 or 2 (see ``models.from_config``)."""
         if layers is None:
             self._ck(self._lib.lum_model_init(self._h, C.byref(desc)))
         else:
@@ -539,8 +556,10 @@ class B200Runtime:
         d = self.desc
         if self.layers is None:
             return (d.n_kv_heads // max(1, d.tp_size)) * d.head_dim
-        g = self.layers[layer]
-        return g.n_kv_heads * (-(-(g.qk_dim if kind == "k" else g.v_dim) // 16) * 16)     # heads padded to multiples of 16
+        g = self.layers[layer_order(d, len(self.layers))[layer]]
+        if g.mixer == 1:
+            return 0
+        return g.n_kv_heads * (max(1, g.maps) if kind == "k" else 1) * (-(-(g.qk_dim if kind == "k" else g.v_dim) // 16) * 16)     # heads padded to multiples of 16
 
     def kv_save(self, layer: int, kind: str, rows: int):
         """Rows [0, rows) of one layer's K or V cache as raw bytes in the cache's own element type."""
@@ -553,6 +572,18 @@ class B200Runtime:
 
     def kv_load(self, layer: int, kind: str, rows: int, data) -> None:
         self._ck(self._lib.lum_kv_load(self._h, layer, 0 if kind == "k" else 1, rows, data.ctypes.data_as(C.c_void_p), data.nbytes))
+
+    def state_save(self):
+        """The selected sequence's recurrent state (raw bytes) and the number of tokens it has seen; empty for models without one."""
+        import numpy as np
+        n, pos = C.c_size_t(), C.c_int32()
+        self._ck(self._lib.lum_state_bytes(self._h, C.byref(n)))
+        out = np.empty(n.value, dtype=np.uint8)
+        self._ck(self._lib.lum_state_save(self._h, out.ctypes.data_as(C.c_void_p), out.nbytes, C.byref(pos)))
+        return out, pos.value
+
+    def state_load(self, data, position: int) -> None:
+        self._ck(self._lib.lum_state_load(self._h, data.ctypes.data_as(C.c_void_p), data.nbytes, position))
 
     def debug_wait_timeout(self) -> None:
         """Test hook: one bounded wait runs out (raises LumError with code LUM_E_DEVICE); the runtime stays usable."""
