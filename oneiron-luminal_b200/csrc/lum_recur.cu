@@ -16,27 +16,15 @@
 namespace lum {
 
 namespace {
-// sqrt(1 - a^2) for ln a = half_q / 2, exact also where a is close to 1 (half_q = 2 ln a <= 0)
-__device__ __forceinline__ float decay_input(float q, float a) {
-    float t = 1.0f - a * a;
-    if (q > -0.25f) {                                          // 1 - e^q = -q (1 + q/2 (1 + q/3 (1 + ...)))
-        float s = fmaf(q, 1.0f / 7.0f, 1.0f);
-        s = fmaf(q * (1.0f / 6.0f), s, 1.0f);
-        s = fmaf(q * (1.0f / 5.0f), s, 1.0f);
-        s = fmaf(q * (1.0f / 4.0f), s, 1.0f);
-        s = fmaf(q * (1.0f / 3.0f), s, 1.0f);
-        s = fmaf(q * (1.0f / 2.0f), s, 1.0f);
-        t = -q * s;
-    }
-    return sqrtf(fmaxf(t, 0.0f));
-}
 __device__ __forceinline__ float softplus_exact(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
-// decay a and input b of one step; sp = softplus(lam), r and i before their sigmoids
-__device__ __forceinline__ void recur_gate(float r, float i, float u, float sp, float& a, float& b) {
-    const float la = -8.0f * sigmoid(r) * sp;
-    a = expf(la);
-    b = decay_input(2.0f * la, a) * sigmoid(i) * u;
+// Decay and input of one step; sp = softplus(lam), r and i before their sigmoids.  Decays are kept as e = a - 1: close to 1, a itself has
+// lost the digits that decide how far back a channel remembers, and 1 - a^2 = -e (2 + e).
+__device__ __forceinline__ void recur_gate(float r, float i, float u, float sp, float& e, float& b) {
+    e = expm1f(-8.0f * sigmoid(r) * sp);
+    b = sqrtf(-e * (2.0f + e)) * sigmoid(i) * u;
 }
+// a s + b
+__device__ __forceinline__ float recur_next(float e, float s, float b) { return s + fmaf(e, s, b); }
 __device__ __forceinline__ uint32_t pack_bf16(float x, float y) {
     const __nv_bfloat162 b = __floats2bfloat162_rn(x, y);
     return *(const uint32_t*)&b;
@@ -168,7 +156,7 @@ __global__ void __launch_bounds__(kRsWarps * 32) recur_step(const RecurArgs a) {
     float da, db;
     recur_gate(vr + a.r_b[c], vi + a.i_b[c], rs_u[grp * KL + kb], softplus_exact(a.lam[c]), da, db);
     float* S = a.state + (size_t)my_seq * a.width + c;
-    const float s = my_pos > 0 ? fmaf(da, *S, db) : db;
+    const float s = my_pos > 0 ? recur_next(da, *S, db) : db;
     *S = s;
     const float v = s * a.yx[(size_t)m * a.ld + c];
     if (a.out_x) { a.out_x[c] = v; return; }
@@ -285,12 +273,12 @@ __global__ void __launch_bounds__(kScThreads, 2) recur_scan(const RecurArgs a) {
             float x, v;
             recur_gate(da[k] + rb, db[k] + ib, y[k], sp, x, v);
             const bool in = r0 + k < a.M;
-            da[k] = in ? x : 1.0f;
+            da[k] = in ? x : 0.0f;
             db[k] = in ? v : 0.0f;
         }
-        float A = 1.0f, B = 0.0f;
+        float A = 0.0f, B = 0.0f;                              // product of the piece's decays, minus one, and its sum from zero
 #pragma unroll
-        for (int k = 0; k < kScT; k++) { A *= da[k]; B = fmaf(da[k], B, db[k]); }
+        for (int k = 0; k < kScT; k++) { A = recur_next(A, da[k], A); B = recur_next(da[k], B, db[k]); }
         ag_a[ch][seg] = A;
         ag_b[ch][seg] = B;
 #pragma unroll
@@ -301,9 +289,9 @@ __global__ void __launch_bounds__(kScThreads, 2) recur_scan(const RecurArgs a) {
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
                 const float qa = __shfl_up_sync(0xffffffffu, pa, o), qb = __shfl_up_sync(0xffffffffu, pb, o);
-                if (lane >= o) { pb = fmaf(pa, qb, pb); pa *= qa; }
+                if (lane >= o) { pb = recur_next(pa, qb, pb); pa = recur_next(pa, qa, pa); }
             }
-            const float end = fmaf(pa, carry, pb);             // state after piece `lane`
+            const float end = recur_next(pa, carry, pb);             // state after piece `lane`
             const float before = __shfl_up_sync(0xffffffffu, end, 1);
             ag_b[warp][lane] = lane ? before : carry;
             carry = __shfl_sync(0xffffffffu, end, 31);
@@ -312,7 +300,7 @@ __global__ void __launch_bounds__(kScThreads, 2) recur_scan(const RecurArgs a) {
         float s = ag_b[ch][seg];
 #pragma unroll
         for (int k = 0; k < kScT; k++) {
-            s = fmaf(da[k], s, db[k]);
+            s = recur_next(da[k], s, db[k]);
             out[seg * kScT + k][ch] = s * y[k];
         }
         __syncthreads();
