@@ -664,34 +664,69 @@ def madipel_spec(pkg, size: dict, n_layers: int, vocab: int, max_seq: int):
     return pkg.models.from_config(cfg, dtype="bfloat16", max_seq=max_seq)
 
 
-def run_madipel(args, pkg):
-    """Prompt and decode throughput of the Madipel design (bf16) beside the Llama family (Q8_0) at equal sizes: a cut of `--layers` layers
-    with a vocabulary of 32768, one prompt of `--prompt-len` tokens as rows, then `--steps` x `--tokens-per-step` decoded tokens.  Timed
-    with CUDA events on the runtime's stream; weights are larger than L2."""
+# The Redenex design at the sizes of real recurrent hybrids: two recurrences for every attention layer, four residual streams; `ff` is the
+# inner width of the clamped gate.  The closest existing model — Madipel, bf16 — at the same hidden size, with as many weights per layer
+# (heads of 128, its inner width chosen for that).
+REDENEX_SIZES = {
+    "4096": dict(width=4096, lru=4096, blocks=16, heads=32, kv=8, dim=64, vdim=128, ff=12288, chunk=2048),
+    "2560": dict(width=2560, lru=2560, blocks=10, heads=20, kv=4, dim=64, vdim=128, ff=7680, chunk=2048),
+    "2048": dict(width=2048, lru=2560, blocks=10, heads=16, kv=2, dim=64, vdim=128, ff=6144, chunk=1024),
+}
+
+
+def redenex_spec(pkg, size: dict, n_layers: int, vocab: int, max_seq: int):
+    mlp = {"kind": "dense", "ff": size["ff"], "limit": 7.0}
+    rec = {"type": "rglru", "mixer": {"width": size["lru"], "blocks": size["blocks"], "conv": 4}, "mlp": mlp}
+    att = {"type": "attention", "mixer": {"heads": size["heads"], "kv_heads": size["kv"], "dim": size["dim"], "vdim": size["vdim"], "conv": 4, "diff": 0.5,
+                                          "scale": size["dim"] ** -0.5, "rot": {"dims": size["dim"], "base": 10000.0}, "mask": {"size": size["chunk"]}}, "mlp": mlp}
+    cfg = {"architecture": "Redenex", "layers": [(rec, rec, att)[i % 3] for i in range(n_layers)], "width": size["width"], "vocab": vocab, "streams": 4,
+           "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}}
+    return pkg.models.from_config(cfg, dtype="bfloat16", max_seq=max_seq)
+
+
+def arm_model(pkg, arm: str, z: dict, L: int, vocab: int, max_seq: int):
+    """(descriptors, linear weights of the layers, bytes per weight, attention layers as (flops per visible pair, cache bytes per row, reach))."""
+    if arm == "llama_q8":
+        ff = z["ff"] * 2 // 3
+        desc = pkg.CONFIGS["llama3_8b_q8"].copy(n_layers=L, hidden=z["width"], n_q_heads=z["heads"], n_kv_heads=z["kv"], head_dim=z["dim"], ffn=ff, vocab=vocab, max_seq=max_seq)
+        weights = L * z["width"] * (2 * z["heads"] * z["dim"] + 2 * z["kv"] * z["dim"] + 3 * ff)
+        return (desc,), weights, 34.0 / 32.0, [(4.0 * z["heads"] * z["dim"], 4.0 * z["kv"] * z["dim"], max_seq)] * L
+    if arm == "redenex":
+        spec = redenex_spec(pkg, z, L, vocab, max_seq)
+        att = [(4.0 * z["heads"] * (z["dim"] + z["vdim"]), 2.0 * z["kv"] * (2 * z["dim"] + z["vdim"]), -z["chunk"])] * sum(g.mixer == 0 for g in spec.layers)
+        return (spec.desc, spec.layers), spec.weight_elems_per_token() - vocab * z["width"], 2.0, att
+    if "lru" in z:                                             # Madipel at a Redenex size
+        per = (redenex_spec(pkg, z, 3, vocab, max_seq).weight_elems_per_token() - vocab * z["width"]) / 3
+        heads = z["width"] // 128
+        kv = max(1, heads // 4)
+        z = dict(width=z["width"], heads=heads, kv=kv, dim=128, ff=int(per / z["width"] - 2 * (heads + kv) * 128) // 128 * 64, window=z["chunk"])
+    spec = madipel_spec(pkg, z, L, vocab, max_seq)
+    att = [(4.0 * z["heads"] * z["dim"], 4.0 * z["kv"] * z["dim"], z["window"])] * L
+    return (spec.desc, spec.layers), spec.weight_elems_per_token() - vocab * z["width"], 2.0, att
+
+
+def run_side_by_side(args, pkg):
+    """Prompt and decode throughput of a design (bf16) beside the closest other models at equal sizes: a cut of `--layers` layers with a
+    vocabulary of 32768, one prompt of `--prompt-len` tokens as rows, then `--steps` x `--tokens-per-step` decoded tokens.  Timed with CUDA
+    events on the runtime's stream; weights are larger than L2."""
     import torch
     torch.cuda.set_device(0)
     peaks, peak_kind = measured_peaks()
     tf_peak = peaks.get("bf16_tflops_sustained", 1383.9)
+    design = args.workload
+    table = MADIPEL_SIZES if design == "madipel" else REDENEX_SIZES
+    arms = (args.arms or ("madipel,llama_q8" if design == "madipel" else "redenex,madipel")).split(",")
     n, vocab, L, sizes = PROMPT_LEN, 32768, args.layers, []
-    new = args.steps * TOKENS_PER_STEP
     total_launches = 0
     sampler = ClockSampler(physical_gpu_index(0))
     sampler.start()
-    for name in (args.size.split(",") if args.size else MADIPEL_SIZES):
-        z, row = MADIPEL_SIZES[name], {"size": name, **MADIPEL_SIZES[name]}
+    for name in (args.size.split(",") if args.size else table):
+        z, row = table[name], {"size": name, **table[name]}
         max_seq = (n + (args.warmup + args.steps + 1) * TOKENS_PER_STEP + 63) // 64 * 64
-        for arm in args.arms.split(","):
+        for arm in arms:
             rt = pkg.B200Runtime.initialize(device=0)
-            if arm == "madipel":
-                spec = madipel_spec(pkg, z, L, vocab, max_seq)
-                rt.load_model(spec.desc, spec.layers)
-                w_layers, ff_mats, wb, window = spec.weight_elems_per_token() - vocab * z["width"], 2, 2.0, z["window"]
-            else:
-                desc = pkg.CONFIGS["llama3_8b_q8"].copy(n_layers=L, hidden=z["width"], n_q_heads=z["heads"], n_kv_heads=z["kv"], head_dim=z["dim"],
-                                                        ffn=z["ff"] * 2 // 3, vocab=vocab, max_seq=max_seq)
-                rt.load_model(desc)
-                w_layers = L * z["width"] * (2 * z["heads"] * z["dim"] + 2 * z["kv"] * z["dim"] + 3 * (z["ff"] * 2 // 3))
-                wb, window = 34.0 / 32.0, max_seq
+            model, w_layers, wb, att = arm_model(pkg, arm, z, L, vocab, max_seq)
+            rt.load_model(*model)
             rt.synth(SEED)
             ids = _prompt_tokens(vocab, n)
             ext = torch.cuda.ExternalStream(rt.stream())
@@ -715,10 +750,11 @@ def run_madipel(args, pkg):
             ms_p = timed(prompt, args.steps, args.warmup)
             prompt()
             ms_d = timed(decode, args.steps, args.warmup) / TOKENS_PER_STEP
-            pairs = sum(min(i + 1, window) for i in range(n))
-            flops = 2.0 * w_layers * n + 2.0 * vocab * z["width"] + L * 4.0 * z["heads"] * z["dim"] * pairs
-            ctx = min(n + (args.warmup + args.steps / 2.0) * TOKENS_PER_STEP, window)
-            bytes_tok = (w_layers + vocab * z["width"]) * wb + L * 2 * 2.0 * z["kv"] * z["dim"] * ctx
+            at = n + (args.warmup + args.steps / 2.0) * TOKENS_PER_STEP
+            flops, bytes_tok = 2.0 * w_layers * n + 2.0 * vocab * z["width"], (w_layers + vocab * z["width"]) * wb
+            for pair_flops, row_bytes, reach in att:           # reach < 0: chunks of that many positions
+                flops += pair_flops * sum((i % -reach if reach < 0 else min(i, reach - 1)) + 1 for i in range(n))
+                bytes_tok += row_bytes * (at % -reach if reach < 0 else min(at, reach))
             row[arm] = {"prompt_tokens_per_s": n / ms_p * 1e3, "prompt_ms": ms_p, "prompt_tflops": flops / ms_p / 1e9, "prompt_frac": flops / ms_p / 1e9 / tf_peak,
                         "decode_tokens_per_s": 1e3 / ms_d, "decode_us": ms_d * 1e3, "decode_gbs": bytes_tok / ms_d / 1e6,
                         "decode_frac": bytes_tok / ms_d / 1e6 / peaks["hbm_gbs"], "launches_per_step": rt.launches_per_step()}
@@ -726,11 +762,11 @@ def run_madipel(args, pkg):
             rt.close()
         sizes.append(row)
     clocks = sampler.stop()
-    first = sizes[0].get("madipel") or sizes[0].get("llama_q8")
-    print(json.dumps({"metric": "madipel_bf16_decode_tokens_per_s", "value": first["decode_tokens_per_s"], "unit": UNIT, "n_gpus": 1, "steps": args.steps,
+    first = next(sizes[0][a] for a in [design] + arms if a in sizes[0])
+    print(json.dumps({"metric": f"{design}_bf16_decode_tokens_per_s", "value": first["decode_tokens_per_s"], "unit": UNIT, "n_gpus": 1, "steps": args.steps,
                       "warmup": args.warmup, "ms_per_step": first["decode_us"] * TOKENS_PER_STEP / 1e3, "higher_is_better": True, "scaling": "strong",
-                      "vs_baseline": None, "dtype": "bf16 x bf16 -> f32 (madipel), Q8_0 (llama_q8)", "data": "synthetic",
-                      "config": {"workload": "madipel", "layers": L, "vocab": vocab, "prompt_len": n, "tokens_per_step": TOKENS_PER_STEP, "seed": SEED,
+                      "vs_baseline": None, "dtype": "bf16 x bf16 -> f32 (madipel, redenex), Q8_0 (llama_q8)", "data": "synthetic",
+                      "config": {"workload": design, "layers": L, "vocab": vocab, "prompt_len": n, "tokens_per_step": TOKENS_PER_STEP, "seed": SEED,
                                  "peak": f"of {peak_kind}: {peaks['hbm_gbs']:.1f} GB/s copy, {tf_peak:.1f} TFLOP/s sustained bf16", "l2": "weights >> 126 MB L2"},
                       "sizes": sizes, "gpu_launches": total_launches, "clocks": clocks}))
 
@@ -935,13 +971,13 @@ def main():
     ap.add_argument("--report", default=None, help="also write the byte / flop counts of the timed step as a metrics JSON in the reference bench crate's format")
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN, help="prompt tokens before the timed decode (profiling runs use a short one)")
     ap.add_argument("--tokens-per-step", type=int, default=TOKENS_PER_STEP)
-    ap.add_argument("--workload", default=WORKLOAD, choices=["llama3_8b_q8", "qwen3_4b_q8", "llama3_8b_q8_bs32", "llama3_8b_q8_prefill4096", "gpt_oss_20b_q8", "madipel"],
+    ap.add_argument("--workload", default=WORKLOAD, choices=["llama3_8b_q8", "qwen3_4b_q8", "llama3_8b_q8_bs32", "llama3_8b_q8_prefill4096", "gpt_oss_20b_q8", "madipel", "redenex"],
                     help="llama3_8b_q8: the configuration the metric is quoted on (default); qwen3_4b_q8: the Qwen3-4B shape; "
                          "llama3_8b_q8_bs32 / llama3_8b_q8_prefill4096: the same model in the tensor-core regime (batched decode / one long prompt); "
-                         "madipel: prompt and decode throughput of the Madipel design beside the Llama family at equal sizes")
-    ap.add_argument("--size", default=None, help="madipel: comma-separated sizes (default: all)")
-    ap.add_argument("--layers", type=int, default=8, help="madipel: layers of the cut")
-    ap.add_argument("--arms", default="madipel,llama_q8", help="madipel: which models to time")
+                         "madipel, redenex: prompt and decode throughput of that design beside the closest other model at equal sizes")
+    ap.add_argument("--size", default=None, help="madipel, redenex: comma-separated sizes (default: all)")
+    ap.add_argument("--layers", type=int, default=None, help="madipel, redenex: layers of the cut (8, 9)")
+    ap.add_argument("--arms", default=None, help="madipel, redenex: which models to time (madipel,llama_q8; redenex,madipel)")
     ap.add_argument("--only", default="all", choices=["all", "kernel", "sweep", "floor", "gemm", "gemm512", "gemm32", "prompt2", "sampler"],
                     help="kernel: time only the dominant kernel alone (small, for ncu captures); sweep: the kernel alone over a range of row counts; "
                          "floor: the decode step with all projections shrunk away; gemm: the tensor-core GEMM alone on the layer's shapes "
@@ -957,13 +993,14 @@ def main():
             return
         run_moe(args, pkg)
         return
-    if args.workload == "madipel":
+    if args.workload in ("madipel", "redenex"):
         if args.impl == "reference":
             print(json.dumps({"impl": "reference", "unavailable": "the reference has no such model"}))
             return
         if args.prompt_len == 512:
             PROMPT_LEN = 4096
-        run_madipel(args, pkg)
+        args.layers = args.layers or (8 if args.workload == "madipel" else 9)
+        run_side_by_side(args, pkg)
         return
     if args.workload in ("llama3_8b_q8_bs32", "llama3_8b_q8_prefill4096"):
         if args.impl == "reference":
