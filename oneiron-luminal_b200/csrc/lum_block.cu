@@ -187,93 +187,150 @@ __device__ __forceinline__ void head_norm_rotate(float* v, int n, const float* g
     }
     __syncwarp();
 }
-// Rows of a pass, RB at a time; the convolved columns of a row lie in shared memory until its heads are done.
-template <int RB>
+// Rows of a pass: a warp takes one head (of a map) of queries or keys, or 32 NJ columns of values, of RB rows.  A lane owns the columns
+// lane + 32 j; the convolution's window slides over the rows in registers, the norms of the rows are summed side by side, and the
+// rotation finds its other half in shared memory.
+template <int NJ, int RB>
 __global__ void __launch_bounds__(256) qkv_head_rows(const BandArgs a) {
     extern __shared__ __align__(16) float qh[];
     const QkvArgs& p = a.p;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int nq = p.n_q * p.maps, nk = p.n_kv * p.maps, half = p.rot_dims / 2;
-    const int m0 = blockIdx.x * RB, nr = min(RB, a.M - m0);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int nq = p.n_q * p.maps, nk = p.n_kv * p.maps, vd = p.n_kv * p.dv, half = p.rot_dims / 2;
+    const int job = blockIdx.x * 8 + warp, m0 = blockIdx.y * RB, nr = min(RB, a.M - m0);
+    if (job >= nq + nk + (vd + 32 * NJ - 1) / (32 * NJ)) return;
+    const bool is_q = job < nq, is_v = job >= nq + nk;
+    const int v0 = (job - nq - nk) * 32 * NJ;                              // first column of a value piece
+    const int n = is_v ? min(32 * NJ, vd - v0) : p.dk;
+    const int c0 = is_q ? p.q_off + job * p.dk : is_v ? p.v_off + v0 : p.k_off + (job - nq) * p.dk;
+    float* buf = qh + warp * RB * 32 * NJ;
+    int pos[RB], seq[RB];
     bool bad = false;
-    for (int r = 0; r < nr; r++) {
-        const int pos = a.row_pos[m0 + r], seq = a.row_seq ? a.row_seq[m0 + r] : a.seq0;
-        bad = bad || pos < 0 || pos >= a.max_seq || seq < 0 || seq >= a.max_batch;
+#pragma unroll
+    for (int r = 0; r < RB; r++) {
+        pos[r] = r < nr ? a.row_pos[m0 + r] : 0;
+        seq[r] = r < nr && a.row_seq ? a.row_seq[m0 + r] : a.seq0;
+        bad = bad || pos[r] < 0 || pos[r] >= a.max_seq || seq[r] < 0 || seq[r] >= a.max_batch;
     }
     if (bad) {
-        if (tid == 0) atomicOr(a.status, LUM_ST_BAD_POS);
+        if (lane == 0) atomicOr(a.status, LUM_ST_BAD_POS);
         return;
     }
-    const size_t ring_seq = (size_t)p.conv.taps * p.conv.ch;
-    if (p.conv.taps == 4 && !a.row_seq && m0 >= 3) {                       // the rows before are in this pass: a sliding window in registers
-        for (int c = tid * 4; c < p.ld; c += 1024) {
-            float4 w[4];                                                   // of one column each
+    float x[RB][NJ];
+    if (p.conv.taps == 4 && !a.row_seq && m0 >= 3) {                       // the rows before are in this pass
+        const float* src = p.qkv + (size_t)(m0 - 3) * p.ld + c0 + lane;
+        float h[3][NJ];
+        float4 w[NJ];
 #pragma unroll
-            for (int i = 0; i < 4; i++) w[i] = *(const float4*)(p.conv.w + (size_t)(c + i) * 4);
-            const float* src = p.qkv + (size_t)(m0 - 3) * p.ld + c;
-            float4 x[RB + 3];
+        for (int j = 0; j < NJ; j++) {
+            const bool in = lane + 32 * j < n;
+            w[j] = in ? *(const float4*)(p.conv.w + (size_t)(c0 + lane + 32 * j) * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-            for (int r = 0; r < RB + 3; r++) if (r < nr + 3) x[r] = *(const float4*)(src + (size_t)r * p.ld);
+            for (int d = 0; d < 3; d++) h[d][j] = in ? src[(size_t)d * p.ld + 32 * j] : 0.0f;
+#pragma unroll
+            for (int r = 0; r < RB; r++) x[r][j] = in && r < nr ? src[(size_t)(r + 3) * p.ld + 32 * j] : 0.0f;
+        }
+#pragma unroll
+        for (int j = 0; j < NJ; j++)
 #pragma unroll
             for (int r = 0; r < RB; r++) {
-                if (r < nr) {
-                    float4 o;
-                    o.x = fmaf(w[0].w, x[r + 3].x, fmaf(w[0].z, x[r + 2].x, fmaf(w[0].y, x[r + 1].x, w[0].x * x[r].x)));
-                    o.y = fmaf(w[1].w, x[r + 3].y, fmaf(w[1].z, x[r + 2].y, fmaf(w[1].y, x[r + 1].y, w[1].x * x[r].y)));
-                    o.z = fmaf(w[2].w, x[r + 3].z, fmaf(w[2].z, x[r + 2].z, fmaf(w[2].y, x[r + 1].z, w[2].x * x[r].z)));
-                    o.w = fmaf(w[3].w, x[r + 3].w, fmaf(w[3].z, x[r + 2].w, fmaf(w[3].y, x[r + 1].w, w[3].x * x[r].w)));
-                    *(float4*)(qh + r * p.ld + c) = o;
+                const float now = x[r][j];
+                x[r][j] = fmaf(w[j].w, now, fmaf(w[j].z, h[2][j], fmaf(w[j].y, h[1][j], w[j].x * h[0][j])));
+                h[0][j] = h[1][j]; h[1][j] = h[2][j]; h[2][j] = now;
+            }
+    } else {
+#pragma unroll
+        for (int r = 0; r < RB; r++) {
+            float* ring = p.conv.ring + (size_t)seq[r] * p.conv.taps * p.conv.ch;
+            const float* src = p.qkv + (size_t)(m0 + r) * p.ld;
+#pragma unroll
+            for (int j = 0; j < NJ; j++) {
+                const int e = lane + 32 * j;
+                x[r][j] = 0.0f;
+                if (r < nr && e < n) {
+                    x[r][j] = conv_at(p.conv, ring, src, p.ld, a.row_seq ? 0 : m0 + r, pos[r], c0 + e);
+                    // one row of its sequence: its value takes the place in the ring that no row of this pass reads
+                    if (p.conv.taps > 0 && (a.row_seq || a.M == 1)) ring[(size_t)(pos[r] % p.conv.taps) * p.conv.ch + c0 + e] = src[c0 + e];
                 }
             }
         }
-    } else {
-        for (int r = 0; r < nr; r++) {
-            const int m = m0 + r, pos = a.row_pos[m], seq = a.row_seq ? a.row_seq[m] : a.seq0;
-            const float* src = p.qkv + (size_t)m * p.ld;
-            float* ring = p.conv.ring + seq * ring_seq;
-            for (int c = tid; c < p.ld; c += 256) {
-                qh[r * p.ld + c] = conv_at(p.conv, ring, src, p.ld, a.row_seq ? 0 : m, pos, c);
-                // one row of its sequence: its value takes the place in the ring that no row of this pass reads
-                if (p.conv.taps > 0 && (a.row_seq || a.M == 1)) ring[(size_t)(pos % p.conv.taps) * p.conv.ch + c] = src[c];
+    }
+    if (is_v) {
+#pragma unroll
+        for (int r = 0; r < RB; r++) {
+            if (r >= nr) continue;
+            const size_t vo = kv_phys_row(a.pg, seq[r], a.max_seq, pos[r]) * p.n_kv * p.dvp;
+#pragma unroll
+            for (int j = 0; j < NJ; j++) {
+                const int c = v0 + lane + 32 * j, h = c / p.dv;
+                if (lane + 32 * j < n) cache_store(a.v_cache, a.kv_bf16, vo + (size_t)h * p.dvp + (c - h * p.dv), x[r][j]);      // (padding stays zero)
             }
         }
+        return;
     }
-    __syncthreads();
-    for (int job = warp; job < nr * (nq + nk); job += 8) {
-        const int r = job / (nq + nk), h = job - r * (nq + nk), m = m0 + r, pos = a.row_pos[m];
-        const bool is_q = h < nq;
-        float* v = qh + r * p.ld + (is_q ? p.q_off + h * p.dk : p.k_off + (h - nq) * p.dk);
-        head_norm_rotate(v, p.dk, is_q ? p.q_gain : p.k_gain, p.eps, p.rot + (size_t)pos * half, p.rot_dims, lane);
-        if (is_q) {
-            float* o = a.q_out + ((size_t)m * nq + h) * p.dkp;
-            for (int e = lane; e < p.dkp; e += 32) o[e] = e < p.dk ? v[e] * p.scale : 0.0f;
-        } else {
-            const size_t ko = kv_phys_row(a.pg, a.row_seq ? a.row_seq[m] : a.seq0, a.max_seq, pos) * nk * p.dkp + (size_t)(h - nq) * p.dkp;
-            for (int e = lane; e < p.dkp; e += 32) cache_store(a.k_cache, a.kv_bf16, ko + e, e < p.dk ? v[e] : 0.0f);
+    const float* gain = is_q ? p.q_gain : p.k_gain;
+    if (gain) {
+        float s[RB];
+#pragma unroll
+        for (int r = 0; r < RB; r++) {
+            s[r] = 0.0f;
+#pragma unroll
+            for (int j = 0; j < NJ; j++) s[r] = fmaf(x[r][j], x[r][j], s[r]);
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+            for (int r = 0; r < RB; r++) s[r] += __shfl_xor_sync(0xffffffffu, s[r], o);
+#pragma unroll
+        for (int j = 0; j < NJ; j++) {
+            const float g = lane + 32 * j < n ? gain[lane + 32 * j] : 0.0f;
+#pragma unroll
+            for (int r = 0; r < RB; r++) x[r][j] *= g / sqrtf(s[r] / (float)n + p.eps);
         }
     }
-    for (int r = 0; r < nr; r++) {
-        const size_t vo = kv_phys_row(a.pg, a.row_seq ? a.row_seq[m0 + r] : a.seq0, a.max_seq, a.row_pos[m0 + r]) * p.n_kv * p.dvp;
-        const float* v = qh + r * p.ld + p.v_off;
-        for (int i = tid; i < p.n_kv * p.dvp; i += 256) {
-            const int h = i / p.dvp, e = i - h * p.dvp;
-            cache_store(a.v_cache, a.kv_bf16, vo + i, e < p.dv ? v[h * p.dv + e] : 0.0f);
+    if (half > 0) {
+#pragma unroll
+        for (int r = 0; r < RB; r++)
+#pragma unroll
+            for (int j = 0; j < NJ; j++) buf[(r * NJ + j) * 32 + lane] = x[r][j];
+        __syncwarp();
+#pragma unroll
+        for (int r = 0; r < RB; r++)
+#pragma unroll
+            for (int j = 0; j < NJ; j++) {
+                const int e = lane + 32 * j, i = e < half ? e : e - half;
+                if (e < 2 * half && r < nr) {
+                    const float2 cs = p.rot[(size_t)pos[r] * half + i];
+                    const float o = buf[r * NJ * 32 + (e < half ? e + half : i)];
+                    x[r][j] = e < half ? x[r][j] * cs.x - o * cs.y : fmaf(x[r][j], cs.x, o * cs.y);
+                }
+            }
+    }
+#pragma unroll
+    for (int r = 0; r < RB; r++) {
+        if (r >= nr) continue;
+        if (is_q) {
+            float* o = a.q_out + ((size_t)(m0 + r) * nq + job) * p.dkp;
+#pragma unroll
+            for (int j = 0; j < NJ; j++) if (lane + 32 * j < p.dkp) o[lane + 32 * j] = x[r][j] * p.scale;
+        } else {
+            const size_t ko = kv_phys_row(a.pg, seq[r], a.max_seq, pos[r]) * nk * p.dkp + (size_t)(job - nq) * p.dkp;
+#pragma unroll
+            for (int j = 0; j < NJ; j++) if (lane + 32 * j < p.dkp) cache_store(a.k_cache, a.kv_bf16, ko + lane + 32 * j, x[r][j]);
         }
     }
 }
 cudaError_t launch_qkv_head_rows(const BandArgs& a, cudaStream_t st) {
-    if (a.M <= 0 || !a.p.per_head || a.p.maps < 1 || a.p.ld % 4) return cudaErrorInvalidValue;
-    const size_t row = (size_t)a.p.ld * 4;
-    const int RB = a.row_seq || a.M < 64 ? 1 : row * 4 <= 100 * 1024 ? 4 : row * 2 <= 200 * 1024 ? 2 : 1;
-    if (row * RB > 200 * 1024) return cudaErrorInvalidValue;
-    const void* fn = RB == 4 ? (const void*)qkv_head_rows<4> : RB == 2 ? (const void*)qkv_head_rows<2> : (const void*)qkv_head_rows<1>;
-    if (row * RB > 48 * 1024) {
-        const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-        if (e != cudaSuccess) return e;
-    }
+    const QkvArgs& p = a.p;
+    if (a.M <= 0 || !p.per_head || p.maps < 1 || p.dkp > 1024 || p.dk > p.dkp) return cudaErrorInvalidValue;
+    const int NJ = p.dkp <= 64 ? 2 : p.dkp <= 128 ? 4 : p.dkp <= 256 ? 8 : 32, RB = NJ == 32 || a.row_seq || a.M < 32 ? 1 : NJ == 8 ? 4 : 8;
+    const void* fn = NJ == 32 ? (const void*)qkv_head_rows<32, 1>
+                     : RB == 1 ? (NJ == 2 ? (const void*)qkv_head_rows<2, 1> : NJ == 4 ? (const void*)qkv_head_rows<4, 1> : (const void*)qkv_head_rows<8, 1>)
+                               : (NJ == 2 ? (const void*)qkv_head_rows<2, 8> : NJ == 4 ? (const void*)qkv_head_rows<4, 8> : (const void*)qkv_head_rows<8, 4>);
+    const int jobs = (p.n_q + p.n_kv) * p.maps + (p.n_kv * p.dv + 32 * NJ - 1) / (32 * NJ);
+    const size_t smem = (size_t)8 * RB * 32 * NJ * 4;                      // at most 32 KB
     BandArgs b = a;
     void* params[] = {&b};
-    return cudaLaunchKernel(fn, dim3((a.M + RB - 1) / RB), dim3(256), params, row * RB, st);
+    return cudaLaunchKernel(fn, dim3((jobs + 7) / 8, (a.M + RB - 1) / RB), dim3(256), params, smem, st);
 }
 
 // ------------------------------------------------------------------------------------------------ residual streams

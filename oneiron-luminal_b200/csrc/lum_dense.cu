@@ -353,6 +353,11 @@ __device__ __forceinline__ void rows_epilogue8(const DenseArgs& a, int m, int n,
         return;
     }
     float* y = a.y + (size_t)m * a.ldy + n;
+    if (a.epi == DENSE_STORE && (a.ldy & 7) == 0 && n + 8 <= a.ldy && ((uintptr_t)y & 31) == 0) {      // a whole sector at once
+        asm volatile("st.global.v8.f32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(y), "f"(a.mult * v[0]), "f"(a.mult * v[1]), "f"(a.mult * v[2]), "f"(a.mult * v[3]),
+                     "f"(a.mult * v[4]), "f"(a.mult * v[5]), "f"(a.mult * v[6]), "f"(a.mult * v[7]) : "memory");
+        return;
+    }
     if ((a.ldy & 3) == 0 && n + 8 <= a.ldy) {                 // rows padded to whole 16-byte groups: columns beyond n_real receive zeros
         float4 r0 = make_float4(0.f, 0.f, 0.f, 0.f), r1 = r0;
         if (a.epi == DENSE_RESID) { r0 = ((const float4*)y)[0]; r1 = ((const float4*)y)[1]; }

@@ -47,7 +47,7 @@ cudaError_t launch_conv_tail(const ConvTailArgs& a, cudaStream_t st) {
 // ------------------------------------------------------------------------------------------------ one step
 // CTA = (block of the gates, 4 groups of 8 channels: a warp each) x 4 rows.  Lanes are 4 groups of K x 8 channels; the first chunks' weights
 // are asked for before the projection's results are waited for.
-namespace { constexpr int kRsRows = 4, kRsWarps = 4, kRsPre = 4; }
+namespace { constexpr int kRsRows = 4, kRsWarps = 4, kRsPre = 4, kRsConv = 4; }
 template <int KIND>
 __global__ void __launch_bounds__(kRsWarps * 32) recur_step(const RecurArgs a) {
     constexpr int E = KIND == WK_BF16 ? 8 : 4, CK = KIND == WK_BF16 ? 64 : 32;
@@ -69,6 +69,22 @@ __global__ void __launch_bounds__(kRsWarps * 32) recur_step(const RecurArgs a) {
 #pragma unroll
         for (int c = 0; c < kRsPre; c++) if (c < a.kc) weights(c, pre[c]);
     }
+    // what else does not depend on the step: this lane's channel (of row lane / 8) in the recurrence, the convolution's weights
+    const int grp = lane >> 3, kb = pg * 8 + (lane & 7), c = blk * a.bw + kb, m = m0 + grp;
+    const bool mine = has && grp < nr && kb < a.bw;
+    const float rb = mine ? a.r_b[c] : 0.0f, ib = mine ? a.i_b[c] : 0.0f, lam = mine ? a.lam[c] : 0.0f;
+    const bool four = a.conv.taps == 4 && KL <= kRsConv * kRsWarps * 32;
+    float4 cw[kRsConv];
+    float cb[kRsConv];
+    if (four) {
+#pragma unroll
+        for (int i = 0; i < kRsConv; i++) {
+            const int k = tid + i * kRsWarps * 32;
+            cw[i] = k < a.bw ? __ldg((const float4*)a.conv.w + blk * a.bw + k) : make_float4(0.f, 0.f, 0.f, 0.f);
+            cb[i] = k < a.bw && a.conv_b ? a.conv_b[blk * a.bw + k] : 0.0f;
+        }
+    }
+    const float sp = softplus_exact(lam);
     pdl_grid_wait();
 
     int pos[kRsRows], seq[kRsRows];
@@ -83,7 +99,33 @@ __global__ void __launch_bounds__(kRsWarps * 32) recur_step(const RecurArgs a) {
         if (tid == 0) atomicOr(a.status, LUM_ST_BAD_POS);
         return;
     }
+    int my_pos = pos[0], my_seq = seq[0];
+#pragma unroll
+    for (int r = 1; r < kRsRows; r++) if (grp == r) { my_pos = pos[r]; my_seq = seq[r]; }
+    float* S = a.state + (size_t)my_seq * a.width + c;
+    const float s_old = mine && my_pos > 0 ? *S : 0.0f, y = mine ? a.yx[(size_t)m * a.ld + c] : 0.0f;
     // ---- the block's inputs
+    if (four) {
+#pragma unroll
+        for (int r = 0; r < kRsRows; r++) {
+            if (r >= nr) continue;
+            const float* src = a.yx + (size_t)(m0 + r) * a.ld + a.x_off + blk * a.bw;
+            float* ring = a.conv.ring + (size_t)seq[r] * 4 * a.conv.ch + blk * a.bw;
+            float x[kRsConv][4];
+#pragma unroll
+            for (int i = 0; i < kRsConv; i++) {
+                const int k = tid + i * kRsWarps * 32;
+#pragma unroll
+                for (int d = 0; d < 4; d++) x[i][d] = k < a.bw && pos[r] >= d ? (d ? ring[(size_t)((pos[r] - d) & 3) * a.conv.ch + k] : src[k]) : 0.0f;
+            }
+#pragma unroll
+            for (int i = 0; i < kRsConv; i++) {
+                const int k = tid + i * kRsWarps * 32;
+                if (k < KL) rs_u[r * KL + k] = fmaf(cw[i].w, x[i][0], fmaf(cw[i].z, x[i][1], fmaf(cw[i].y, x[i][2], cw[i].x * x[i][3]))) + cb[i];
+                if (part == 0 && k < a.bw) ring[(size_t)(pos[r] & 3) * a.conv.ch + k] = x[i][0];       // (the row of the ring that no step of this position reads)
+            }
+        }
+    } else
 #pragma unroll
     for (int r = 0; r < kRsRows; r++) {
         if (r >= nr) continue;
@@ -92,10 +134,9 @@ __global__ void __launch_bounds__(kRsWarps * 32) recur_step(const RecurArgs a) {
         for (int k = tid; k < KL; k += kRsWarps * 32) {
             float u = 0.0f;
             if (k < a.bw) {
-                const int c = blk * a.bw + k;
-                u = conv_at(a.conv, ring, src, 0, 0, pos[r], c) + (a.conv_b ? a.conv_b[c] : 0.0f);
-                // (the row of the ring that no step of this position reads)
-                if (part == 0 && a.conv.taps > 0) ring[(size_t)(pos[r] % a.conv.taps) * a.conv.ch + c] = src[c];
+                const int ck = blk * a.bw + k;
+                u = conv_at(a.conv, ring, src, 0, 0, pos[r], ck) + (a.conv_b ? a.conv_b[ck] : 0.0f);
+                if (part == 0 && a.conv.taps > 0) ring[(size_t)(pos[r] % a.conv.taps) * a.conv.ch + ck] = src[ck];
             }
             rs_u[r * KL + k] = u;
         }
@@ -106,7 +147,6 @@ __global__ void __launch_bounds__(kRsWarps * 32) recur_step(const RecurArgs a) {
     float ar[kRsRows], ai[kRsRows];
 #pragma unroll
     for (int r = 0; r < kRsRows; r++) ar[r] = ai[r] = 0.0f;
-    const int grp = lane >> 3;
     auto take = [&](int c, const uint4 (&w)[4]) {
 #pragma unroll
         for (int h = 0; h < 2; h++) {
@@ -144,21 +184,18 @@ __global__ void __launch_bounds__(kRsWarps * 32) recur_step(const RecurArgs a) {
     }
     // ---- every lane has the sums of channel lane % 8 after two shuffles; lane group r finishes row r
     float vr = 0.0f, vi = 0.0f;
-    int my_pos = 0, my_seq = 0;
 #pragma unroll
     for (int r = 0; r < kRsRows; r++) {
         ar[r] += __shfl_xor_sync(0xffffffffu, ar[r], 8); ar[r] += __shfl_xor_sync(0xffffffffu, ar[r], 16);
         ai[r] += __shfl_xor_sync(0xffffffffu, ai[r], 8); ai[r] += __shfl_xor_sync(0xffffffffu, ai[r], 16);
-        if (grp == r) { vr = ar[r]; vi = ai[r]; my_pos = pos[r]; my_seq = seq[r]; }
+        if (grp == r) { vr = ar[r]; vi = ai[r]; }
     }
-    const int kb = pg * 8 + (lane & 7), c = blk * a.bw + kb, m = m0 + grp;
-    if (grp >= nr || kb >= a.bw) return;
+    if (!mine) return;
     float da, db;
-    recur_gate(vr + a.r_b[c], vi + a.i_b[c], rs_u[grp * KL + kb], softplus_exact(a.lam[c]), da, db);
-    float* S = a.state + (size_t)my_seq * a.width + c;
-    const float s = my_pos > 0 ? recur_next(da, *S, db) : db;
+    recur_gate(vr + rb, vi + ib, rs_u[grp * KL + kb], sp, da, db);
+    const float s = recur_next(da, s_old, db);
     *S = s;
-    const float v = s * a.yx[(size_t)m * a.ld + c];
+    const float v = s * y;
     if (a.out_x) { a.out_x[c] = v; return; }
     unsigned char* o = (unsigned char*)a.out.p + row_operand_off(a.out_kind, a.out.chunks, m, c);
     if (a.out_kind == WK_BF16) *(__nv_bfloat16*)o = __float2bfloat16_rn(v);
@@ -194,21 +231,7 @@ __global__ void __launch_bounds__(256) recur_conv(const RecurArgs a) {
     const int pos = a.row_pos[m];
     const float* src = a.yx + (size_t)m * a.ld + a.x_off;
     float u[8];
-    if (a.conv.taps == 4 && m >= 3 && k0 + 8 <= a.bw && ((c0 | a.ld | a.x_off) & 3) == 0) {
-        float4 x[4][2];
-#pragma unroll
-        for (int d = 0; d < 4; d++) {
-            const float* r = src + c0 - (ptrdiff_t)d * a.ld;
-            x[d][0] = *(const float4*)r; x[d][1] = *(const float4*)(r + 4);
-        }
-#pragma unroll
-        for (int i = 0; i < 8; i++) {
-            const float4 w = *(const float4*)(a.conv.w + (size_t)(c0 + i) * 4);
-            const float* x0 = (const float*)&x[0][0] + i; const float* x1 = (const float*)&x[1][0] + i;
-            const float* x2 = (const float*)&x[2][0] + i; const float* x3 = (const float*)&x[3][0] + i;
-            u[i] = fmaf(w.w, *x0, fmaf(w.z, *x1, fmaf(w.y, *x2, w.x * *x3))) + (a.conv_b ? a.conv_b[c0 + i] : 0.0f);
-        }
-    } else {
+    {
         const float* ring = a.conv.ring + (size_t)a.seq0 * a.conv.taps * a.conv.ch;
 #pragma unroll
         for (int i = 0; i < 8; i++) u[i] = k0 + i < a.bw ? conv_at(a.conv, ring, src, a.ld, m, pos, c0 + i) + (a.conv_b ? a.conv_b[c0 + i] : 0.0f) : 0.0f;
@@ -238,9 +261,54 @@ __global__ void __launch_bounds__(256) recur_conv(const RecurArgs a) {
         f[1] = make_float4(u[4], u[5], u[6], u[7]);
     }
 }
+// The same for four taps and blocks of whole groups of 8 channels: thread = 4 channels x 8 rows, the window slides in registers.
+template <int KIND>
+__global__ void __launch_bounds__(256) recur_conv4(const RecurArgs a) {
+    const int c0 = (blockIdx.x * 256 + threadIdx.x) * 4, m0 = blockIdx.y * 8, nr = min(8, a.M - m0);
+    if (c0 >= a.width) return;
+    const int blk = c0 / a.bw, k0 = blk * a.kc * (KIND == WK_BF16 ? 64 : 32) + (c0 - blk * a.bw), pos0 = a.row_pos[0];
+    const float* src = a.yx + a.x_off + c0;
+    const float* ring = a.conv.ring + (size_t)a.seq0 * 4 * a.conv.ch + c0;
+    float4 w[4], x[11];
+#pragma unroll
+    for (int i = 0; i < 4; i++) w[i] = *(const float4*)(a.conv.w + (size_t)(c0 + i) * 4);
+    const float4 b = a.conv_b ? *(const float4*)(a.conv_b + c0) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int r = 0; r < 11; r++) {
+        const int m = m0 + r - 3;
+        x[r] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (m >= 0) { if (r - 3 < nr) x[r] = *(const float4*)(src + (size_t)m * a.ld); }
+        else if (pos0 + m >= 0) x[r] = *(const float4*)(ring + (size_t)((pos0 + m) & 3) * a.conv.ch);
+    }
+#pragma unroll
+    for (int r = 0; r < 8; r++) {
+        if (r >= nr) continue;
+        float4 u;
+        u.x = fmaf(w[0].w, x[r + 3].x, fmaf(w[0].z, x[r + 2].x, fmaf(w[0].y, x[r + 1].x, w[0].x * x[r].x))) + b.x;
+        u.y = fmaf(w[1].w, x[r + 3].y, fmaf(w[1].z, x[r + 2].y, fmaf(w[1].y, x[r + 1].y, w[1].x * x[r].y))) + b.y;
+        u.z = fmaf(w[2].w, x[r + 3].z, fmaf(w[2].z, x[r + 2].z, fmaf(w[2].y, x[r + 1].z, w[2].x * x[r].z))) + b.z;
+        u.w = fmaf(w[3].w, x[r + 3].w, fmaf(w[3].z, x[r + 2].w, fmaf(w[3].y, x[r + 1].w, w[3].x * x[r].w))) + b.w;
+        *(float4*)(a.u + (size_t)(m0 + r) * a.ldu + c0) = u;
+        const size_t o = row_operand_off(KIND, a.hi.chunks, m0 + r, k0);
+        if (KIND == WK_BF16) {
+            const uint32_t h0 = pack_bf16(u.x, u.y), h1 = pack_bf16(u.z, u.w);
+            *(uint2*)((unsigned char*)a.hi.p + o) = make_uint2(h0, h1);
+            *(uint2*)((unsigned char*)a.lo.p + o) = make_uint2(pack_bf16(u.x - __uint_as_float(h0 << 16), u.y - __uint_as_float(h0 & 0xffff0000u)),
+                                                              pack_bf16(u.z - __uint_as_float(h1 << 16), u.w - __uint_as_float(h1 & 0xffff0000u)));
+        } else {
+            *(float4*)((unsigned char*)a.hi.p + o) = u;
+        }
+    }
+}
 cudaError_t launch_recur_conv(const RecurArgs& a, cudaStream_t st) {
     const int groups = a.blocks * a.bwp / 8;
     if (a.M <= 0 || a.row_seq || a.hi.chunks != a.blocks * a.kc || (a.kind == WK_BF16 && (!a.lo.p || a.lo.chunks != a.hi.chunks))) return cudaErrorInvalidValue;
+    if (a.conv.taps == 4 && a.bw % 8 == 0 && ((a.ld | a.x_off | a.ldu | a.conv.ch) & 3) == 0) {
+        const dim3 g4((a.width / 4 + 255) / 256, (a.M + 7) / 8);
+        if (a.kind == WK_BF16) recur_conv4<WK_BF16><<<g4, 256, 0, st>>>(a);
+        else recur_conv4<WK_F32><<<g4, 256, 0, st>>>(a);
+        return cudaGetLastError();
+    }
     const dim3 grid((groups + 31) / 32, (a.M + 7) / 8);
     if (a.kind == WK_BF16) recur_conv<WK_BF16><<<grid, 256, 0, st>>>(a);
     else recur_conv<WK_F32><<<grid, 256, 0, st>>>(a);
