@@ -281,13 +281,27 @@ __global__ void __launch_bounds__(256) qkv_head_rows(const BandArgs a) {
 #pragma unroll
             for (int r = 0; r < RB; r++) s[r] += __shfl_xor_sync(0xffffffffu, s[r], o);
 #pragma unroll
+        for (int r = 0; r < RB; r++) s[r] = 1.0f / sqrtf(s[r] / (float)n + p.eps);
+#pragma unroll
         for (int j = 0; j < NJ; j++) {
             const float g = lane + 32 * j < n ? gain[lane + 32 * j] : 0.0f;
 #pragma unroll
-            for (int r = 0; r < RB; r++) x[r][j] *= g / sqrtf(s[r] / (float)n + p.eps);
+            for (int r = 0; r < RB; r++) x[r][j] *= s[r] * g;
         }
     }
-    if (half > 0) {
+    if (half == 16 * NJ) {                                     // the whole head turns, and both halves of a pair lie in this lane
+#pragma unroll
+        for (int r = 0; r < RB; r++) {
+            const float2* rot = p.rot + (size_t)pos[r] * half + lane;
+#pragma unroll
+            for (int j = 0; j < NJ / 2; j++) {
+                const float2 cs = rot[32 * j];
+                const float u = x[r][j], v = x[r][j + NJ / 2];
+                x[r][j] = u * cs.x - v * cs.y;
+                x[r][j + NJ / 2] = fmaf(v, cs.x, u * cs.y);
+            }
+        }
+    } else if (half > 0) {
 #pragma unroll
         for (int r = 0; r < RB; r++)
 #pragma unroll
@@ -309,9 +323,9 @@ __global__ void __launch_bounds__(256) qkv_head_rows(const BandArgs a) {
     for (int r = 0; r < RB; r++) {
         if (r >= nr) continue;
         if (is_q) {
-            float* o = a.q_out + ((size_t)(m0 + r) * nq + job) * p.dkp;
+            float* o = a.q_out + ((size_t)(m0 + r) * nq + job) * p.dkp + lane;
 #pragma unroll
-            for (int j = 0; j < NJ; j++) if (lane + 32 * j < p.dkp) o[lane + 32 * j] = x[r][j] * p.scale;
+            for (int j = 0; j < NJ; j++) if (lane + 32 * j < p.dkp) o[32 * j] = x[r][j] * p.scale;
         } else {
             const size_t ko = kv_phys_row(a.pg, seq[r], a.max_seq, pos[r]) * nk * p.dkp + (size_t)(job - nq) * p.dkp;
 #pragma unroll

@@ -19,9 +19,12 @@ namespace {
 __device__ __forceinline__ float softplus_exact(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
 // Decay and input of one step; sp = softplus(lam), r and i before their sigmoids.  Decays are kept as e = a - 1: close to 1, a itself has
 // lost the digits that decide how far back a channel remembers, and 1 - a^2 = -e (2 + e).
-__device__ __forceinline__ void recur_gate(float r, float i, float u, float sp, float& e, float& b) {
-    e = expm1f(-8.0f * sigmoid(r) * sp);
-    b = sqrtf(-e * (2.0f + e)) * sigmoid(i) * u;
+__device__ __forceinline__ void recur_gate(float r, float i, float u, float sp, float& e_out, float& b) {
+    const float e = expm1f(-8.0f * sigmoid(r) * sp);
+    float g;
+    asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(g) : "f"(-e * (2.0f + e)));
+    b = g * sigmoid(i) * u;
+    e_out = e;
 }
 // a s + b
 __device__ __forceinline__ float recur_next(float e, float s, float b) { return s + fmaf(e, s, b); }
@@ -331,18 +334,23 @@ __global__ void __launch_bounds__(kScThreads, 2) recur_scan(const RecurArgs a) {
     for (int t0 = 0; t0 < a.M; t0 += kScTile) {
         const int r0 = t0 + seg * kScT;
         float da[kScT], db[kScT], y[kScT];
+        const bool whole = t0 + kScTile <= a.M;
+        if (whole) {
+            const float *pr = a.gates + (size_t)r0 * a.ldg + gr, *pi = a.gates + (size_t)r0 * a.ldg + gi, *pu = a.u + (size_t)r0 * a.ldu + cl;
 #pragma unroll
-        for (int k = 0; k < kScT; k++) {
-            const size_t m = min(r0 + k, a.M - 1);
-            da[k] = a.gates[m * a.ldg + gr]; db[k] = a.gates[m * a.ldg + gi]; y[k] = a.u[m * a.ldu + cl];
+            for (int k = 0; k < kScT; k++) { da[k] = pr[k * a.ldg]; db[k] = pi[k * a.ldg]; y[k] = pu[k * a.ldu]; }
+        } else {
+#pragma unroll
+            for (int k = 0; k < kScT; k++) {
+                const size_t m = min(r0 + k, a.M - 1);
+                da[k] = a.gates[m * a.ldg + gr]; db[k] = a.gates[m * a.ldg + gi]; y[k] = a.u[m * a.ldu + cl];
+            }
         }
 #pragma unroll
-        for (int k = 0; k < kScT; k++) {
-            float x, v;
-            recur_gate(da[k] + rb, db[k] + ib, y[k], sp, x, v);
-            const bool in = r0 + k < a.M;
-            da[k] = in ? x : 0.0f;
-            db[k] = in ? v : 0.0f;
+        for (int k = 0; k < kScT; k++) recur_gate(da[k] + rb, db[k] + ib, y[k], sp, da[k], db[k]);
+        if (!whole) {
+#pragma unroll
+            for (int k = 0; k < kScT; k++) if (r0 + k >= a.M) da[k] = db[k] = 0.0f;
         }
         float A = 0.0f, B = 0.0f;                              // product of the piece's decays, minus one, and its sum from zero
 #pragma unroll
@@ -350,7 +358,7 @@ __global__ void __launch_bounds__(kScThreads, 2) recur_scan(const RecurArgs a) {
         ag_a[ch][seg] = A;
         ag_b[ch][seg] = B;
 #pragma unroll
-        for (int k = 0; k < kScT; k++) y[k] = a.yx[(size_t)min(r0 + k, a.M - 1) * a.ld + cl];
+        for (int k = 0; k < kScT; k++) y[k] = a.yx[(size_t)(whole ? r0 + k : min(r0 + k, a.M - 1)) * a.ld + cl];
         __syncthreads();
         {
             float pa = ag_a[warp][lane], pb = ag_b[warp][lane];
