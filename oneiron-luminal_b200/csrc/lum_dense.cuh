@@ -106,6 +106,13 @@ struct ConvArgs {
 // channel c of the row at `src` (rows ld floats apart); in_pass: rows before it that belong to the same sequence and pass
 __device__ __forceinline__ float conv_at(const ConvArgs& cv, const float* ring, const float* src, int ld, int in_pass, int pos, int c) {
     if (cv.taps == 0) return src[c];
+    if (cv.taps == 4) {                                        // all loads at once
+        float v[4];
+#pragma unroll
+        for (int d = 0; d < 4; d++) v[d] = d <= in_pass ? src[c - (ptrdiff_t)d * ld] : pos >= d ? ring[(size_t)((pos - d) & 3) * cv.ch + c] : 0.0f;
+        const float4 w = *(const float4*)(cv.w + (size_t)c * 4);
+        return fmaf(w.w, v[0], fmaf(w.z, v[1], fmaf(w.y, v[2], w.x * v[3])));
+    }
     const float* w = cv.w + (size_t)c * cv.taps;
     float s = 0.0f;
     for (int d = cv.taps - 1; d >= 0; d--) {
